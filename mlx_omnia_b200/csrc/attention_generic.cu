@@ -1,4 +1,4 @@
-// Paged causal attention for any batch shape, head sizes (<= 256; keys and values may differ in
+// Paged causal attention for any batch shape, head sizes (<= 512; keys and values may differ in
 // width), page size and element type: the kernel of the 32-bit path, and of sizes the tiled kernels
 // refuse. A window may keep the request's first `keep_first` positions visible for good, and the
 // softmax's denominator may hold one more term exp(sink[head]) that has no key and no value.
@@ -12,7 +12,8 @@
 // the token's own position and window, never on how the batch was cut.
 #include "common.cuh"
 
-template <typename T>
+// MOST: a multiple of 32 that neither width exceeds (a lane holds MOST / 32 of the output's dims).
+template <typename T, int MOST>
 __global__ void paged_attention_generic_kernel(
     const T* __restrict__ q,                // [tokens, nq, d]
     const T* __restrict__ k_pages,          // key row: k_pages + page * page_stride + (kvh * page_size + off) * d
@@ -26,7 +27,8 @@ __global__ void paged_attention_generic_kernel(
     const float* __restrict__ sink,         // [nq] or null
     int num_seqs, int max_pages, int num_pages, int nq, int nkv, int d, int dv, int page_size,
     int window, int keep_first, float scale, int chunk, float softcap, int* err) {
-  __shared__ float qs[4][256];
+  constexpr int ACC = MOST / 32;
+  __shared__ float qs[4][MOST];
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.y * 4 + warp;
@@ -48,9 +50,9 @@ __global__ void paged_attention_generic_kernel(
   __syncwarp();
 
   float m = -INFINITY, l = 0.f;
-  float acc[8];
+  float acc[ACC];
 #pragma unroll
-  for (int k = 0; k < 8; ++k) acc[k] = 0.f;
+  for (int k = 0; k < ACC; ++k) acc[k] = 0.f;
   const int* table = block_table + (size_t)seq * max_pages;
 
   // Two runs of keys: the kept first positions below the window, then the window itself.
@@ -81,7 +83,7 @@ __global__ void paged_attention_generic_kernel(
     l = l * alpha + warp_sum(p);
     m = m_new;
 #pragma unroll
-    for (int k = 0; k < 8; ++k) acc[k] *= alpha;
+    for (int k = 0; k < ACC; ++k) acc[k] *= alpha;
     const int count = min(32, run_hi - base + 1);
     for (int jj = 0; jj < count; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
@@ -89,7 +91,7 @@ __global__ void paged_attention_generic_kernel(
       if (vr < 0) continue;
       const T* vp = v_pages + vr;
 #pragma unroll
-      for (int k = 0; k < 8; ++k) {
+      for (int k = 0; k < ACC; ++k) {
         const int i = lane + 32 * k;
         if (i < dv) acc[k] += pj * to_f32(vp[i]);
       }
@@ -102,12 +104,12 @@ __global__ void paged_attention_generic_kernel(
     const float alpha = m == -INFINITY ? 0.f : expf(m - m_new);
     l = l * alpha + expf(z - m_new);
 #pragma unroll
-    for (int k = 0; k < 8; ++k) acc[k] *= alpha;
+    for (int k = 0; k < ACC; ++k) acc[k] *= alpha;
   }
   const float inv = l > 0.f ? 1.f / l : 0.f;
   T* orow = out + ((size_t)t * nq + head) * dv;
 #pragma unroll
-  for (int k = 0; k < 8; ++k) {
+  for (int k = 0; k < ACC; ++k) {
     const int i = lane + 32 * k;
     if (i >= dv) continue;
     float v = acc[k] * inv;
@@ -125,14 +127,21 @@ extern "C" int omnia_paged_attention_generic(
     int tokens, int num_seqs, int max_pages, int num_pages, int nq, int nkv, int d, int dv, int page_size, int window,
     int keep_first, float scale, int chunk, float softcap, int dtype, int* err, cudaStream_t stream) {
   if (tokens == 0) return 0;
-  if (d > 256 || dv > 256 || nkv <= 0 || nq % nkv != 0 || keep_first < 0 || (keep_first > 0 && window <= 0) ||
+  if (d > 512 || dv > 512 || nkv <= 0 || nq % nkv != 0 || keep_first < 0 || (keep_first > 0 && window <= 0) ||
       chunk < 0 || softcap < 0.f || (chunk > 0 && keep_first > 0))
     return (int)cudaErrorInvalidValue;
   dim3 grid(tokens, (nq + 3) / 4);
-  OMNIA_DISPATCH_DTYPE(dtype, (paged_attention_generic_kernel<T><<<grid, 128, 0, stream>>>(
-                                  (const T*)q, (const T*)k_pages, (const T*)v_pages, page_stride, block_table,
-                                  cu_seqlens, positions, (const T*)gate, gate_stride, (T*)out, sink, num_seqs,
-                                  max_pages, num_pages, nq, nkv, d, dv, page_size, window, keep_first, scale, chunk, softcap,
-                                  err)));
+  OMNIA_DISPATCH_DTYPE(dtype, {
+    if (d <= 256 && dv <= 256)
+      paged_attention_generic_kernel<T, 256><<<grid, 128, 0, stream>>>(
+          (const T*)q, (const T*)k_pages, (const T*)v_pages, page_stride, block_table, cu_seqlens, positions, (const T*)gate,
+          gate_stride, (T*)out, sink, num_seqs, max_pages, num_pages, nq, nkv, d, dv, page_size, window, keep_first, scale,
+          chunk, softcap, err);
+    else
+      paged_attention_generic_kernel<T, 512><<<grid, 128, 0, stream>>>(
+          (const T*)q, (const T*)k_pages, (const T*)v_pages, page_stride, block_table, cu_seqlens, positions, (const T*)gate,
+          gate_stride, (T*)out, sink, num_seqs, max_pages, num_pages, nq, nkv, d, dv, page_size, window, keep_first, scale,
+          chunk, softcap, err);
+  });
   return OMNIA_LAUNCH_RESULT();
 }

@@ -16,14 +16,18 @@
 // ---------------------------------------------------------------------------------
 // Per token: c = rms(down[:rank]) * w -> cache[slot, :rank]; the last `rot` columns of the down
 // projection, rotated, -> cache[slot, rank:]; and the last `rot` of every query head rotated in
-// place in the projected rows. Rotation: the first rot_dims dims in pairs (2i, 2i + 1), angle
-// position * inv_freq[i] in float32; dims beyond rot_dims pass unchanged.
+// place in the projected rows. Rotation: the first rot_dims dims in pairs (2i, 2i + 1), or with
+// `half_pairs` (i, i + rot_dims / 2), angle position * inv_freq[i] in float32, cosine and sine times
+// `amount`; dims beyond rot_dims pass unchanged. With `cq_out` the queries have a latent of their own
+// (columns [cq_col, cq_col + q_rank)): it is RMS-normed with `cq_w` into cq_out [tokens, q_rank], and
+// the queries, which the next product makes of it, are turned by latent_rotate_kernel.
 template <typename T>
 __global__ void latent_prepare_kernel(T* __restrict__ proj, int stride, int q_col, int heads, int q_dim,
                                       int down_col, int rank, int rot, const float* __restrict__ w, float eps,
                                       const float* __restrict__ inv_freq, int rot_dims,
                                       const int* __restrict__ positions, const long long* __restrict__ slot_mapping,
-                                      T* __restrict__ cache, long long total_slots, int* err) {
+                                      T* __restrict__ cache, long long total_slots, int half_pairs, float amount, int cq_col,
+                                      int q_rank, const float* __restrict__ cq_w, T* __restrict__ cq_out, int* err) {
   pdl_wait();
   pdl_launch_dependents();
   __shared__ float scratch[33];
@@ -37,6 +41,16 @@ __global__ void latent_prepare_kernel(T* __restrict__ proj, int stride, int q_co
     return;
   }
   T* to = cache + (size_t)(store ? slot : 0) * (rank + rot);
+  if (cq_out != nullptr) {
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
+      const float v = to_f32(row[cq_col + i]);
+      sq += v * v;
+    }
+    const float r = rsqrtf(block_sum(sq, scratch) / (float)q_rank + eps);
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
+      cq_out[(size_t)t * q_rank + i] = from_f32<T>(to_f32(row[cq_col + i]) * r * cq_w[i]);
+  }
   float ss = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) {
     const float v = to_f32(row[down_col + i]);
@@ -51,13 +65,15 @@ __global__ void latent_prepare_kernel(T* __restrict__ proj, int stride, int q_co
     const int job = item / half, i = item % half;
     float s, c;
     sincosf(pos * inv_freq[i], &s, &c);
+    s *= amount, c *= amount;
+    const int i0 = half_pairs ? i : 2 * i, i1 = half_pairs ? i + half : 2 * i + 1;
     T* at = job == 0 ? row + down_col + rank : row + q_col + (size_t)(job - 1) * q_dim + (q_dim - rot);
-    const float a = to_f32(at[2 * i]), b = to_f32(at[2 * i + 1]);
+    const float a = to_f32(at[i0]), b = to_f32(at[i1]);
     const T ra = from_f32<T>(a * c - b * s), rb = from_f32<T>(b * c + a * s);
     if (job == 0) {
-      if (store) to[rank + 2 * i] = ra, to[rank + 2 * i + 1] = rb;
+      if (store) to[rank + i0] = ra, to[rank + i1] = rb;
     } else {
-      at[2 * i] = ra, at[2 * i + 1] = rb;
+      at[i0] = ra, at[i1] = rb;
     }
   }
   if (store)
@@ -67,12 +83,54 @@ __global__ void latent_prepare_kernel(T* __restrict__ proj, int stride, int q_co
 extern "C" int omnia_latent_prepare(void* proj, int stride, int q_col, int heads, int q_dim, int down_col, int rank,
                                     int rot, const float* w, float eps, const float* inv_freq, int rot_dims,
                                     const int* positions, const long long* slot_mapping, void* cache,
-                                    long long total_slots, int tokens, int dtype, int* err, cudaStream_t stream) {
+                                    long long total_slots, int half_pairs, float amount, int cq_col, int q_rank,
+                                    const float* cq_w, void* cq_out, int tokens, int dtype, int* err,
+                                    cudaStream_t stream) {
   if (tokens == 0) return 0;
-  if (rot_dims % 2 != 0 || rot_dims > rot || rot > q_dim || rank < 1) return (int)cudaErrorInvalidValue;
+  if (cq_out != nullptr && (q_rank < 1 || heads != 0)) return (int)cudaErrorInvalidValue;
+  if (rot_dims % 2 != 0 || rot_dims > rot || (heads > 0 && rot > q_dim) || rank < 1) return (int)cudaErrorInvalidValue;
   OMNIA_DISPATCH_DTYPE(dtype, (launch_pdl(latent_prepare_kernel<T>, tokens, 128, 0, stream, (T*)proj, stride, q_col,
                                           heads, q_dim, down_col, rank, rot, w, eps, inv_freq, rot_dims, positions,
-                                          slot_mapping, (T*)cache, total_slots, err)));
+                                          slot_mapping, (T*)cache, total_slots, half_pairs, amount, cq_col,
+                                          q_rank, cq_w, (T*)cq_out, err)));
+  return OMNIA_LAUNCH_RESULT();
+}
+
+// The last `rot` of every query head (q [tokens, heads * q_dim], rows `stride` apart) turned in place as above:
+// a thread a pair.
+template <typename T>
+__global__ void latent_rotate_kernel(T* __restrict__ q, int stride, int heads, int q_dim, int rot,
+                                     const float* __restrict__ inv_freq, int half, int half_pairs, float amount,
+                                     const int* __restrict__ positions, int tokens) {
+  pdl_wait();
+  pdl_launch_dependents();
+  extern __shared__ float2 turn_s[];  // [half] (cos, sin)
+  const int t = blockIdx.x;
+  const float pos = (float)positions[t];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(pos * inv_freq[i], &s, &c);
+    turn_s[i] = make_float2(c * amount, s * amount);
+  }
+  __syncthreads();
+  for (int item = threadIdx.x; item < heads * half; item += blockDim.x) {
+    const int head = item / half, i = item % half;
+    const int i0 = half_pairs ? i : 2 * i, i1 = half_pairs ? i + half : 2 * i + 1;
+    T* at = q + (size_t)t * stride + (size_t)head * q_dim + (q_dim - rot);
+    const float a = to_f32(at[i0]), b = to_f32(at[i1]);
+    const float2 turn = turn_s[i];
+    at[i0] = from_f32<T>(a * turn.x - b * turn.y), at[i1] = from_f32<T>(b * turn.x + a * turn.y);
+  }
+}
+
+extern "C" int omnia_latent_rotate(void* q, int stride, int heads, int q_dim, int rot, const float* inv_freq, int rot_dims,
+                                   int half_pairs, float amount, const int* positions, int tokens, int dtype,
+                                   cudaStream_t stream) {
+  if (tokens == 0 || rot_dims == 0) return 0;
+  if (rot_dims % 2 != 0 || rot_dims > rot || rot > q_dim || heads < 1) return (int)cudaErrorInvalidValue;
+  const int half = rot_dims / 2;
+  OMNIA_DISPATCH_DTYPE(dtype, (launch_pdl(latent_rotate_kernel<T>, tokens, 256, half * sizeof(float2), stream, (T*)q, stride,
+                                          heads, q_dim, rot, inv_freq, half, half_pairs, amount, positions, tokens)));
   return OMNIA_LAUNCH_RESULT();
 }
 

@@ -46,6 +46,12 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// xIELU: rise z^2 + z / 2 above zero, fall (e^z - 1 - z) + z / 2 below. e^z - 1 is taken whole, so small
+// |z| keep their digits.
+__device__ __forceinline__ float xielu(float z, float rise, float fall) {
+  return z > 0.f ? fmaf(rise * z, z, 0.5f * z) : fmaf(fall, expm1f(z) - z, 0.5f * z);
+}
+
 // Sum over the block; every thread gets the result. `scratch` holds 33 floats.
 // The order of the additions depends only on blockDim, never on the data.
 __device__ __forceinline__ float block_sum(float v, float* scratch) {

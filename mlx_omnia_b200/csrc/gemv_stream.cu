@@ -158,7 +158,7 @@ __host__ __device__ constexpr size_t partial_bytes(int nt) { return sizeof(float
 template <int NT, int EPI, bool PENDING>
 __global__ void __launch_bounds__(THREADS, 1)
 gemv_stream_kernel(const bf16* __restrict__ a, const __grid_constant__ CUtensorMap map_w, void* __restrict__ out,
-                   int m, int n, int k, int inner, int tiles, float multiplier, float cap, const PendingStep pending,
+                   int m, int n, int k, int inner, int tiles, float multiplier, float cap, float second, const PendingStep pending,
                    int* __restrict__ err) {
   extern __shared__ __align__(128) unsigned char smem[];
   unsigned char* ring = smem;
@@ -446,8 +446,8 @@ gemv_stream_kernel(const bf16* __restrict__ a, const __grid_constant__ CUtensorM
             const float z = __bfloat162float(__float2bfloat16_rn(v)) * multiplier;
             reinterpret_cast<float*>(out)[(size_t)token * n + col] = cap > 0.f ? cap * tanhf(z / cap) : z;
           } else {
-            // cap selects an activation of the stored product (0 none, 1 relu^2, 2 tanh-GELU, 3 SiLU),
-            // applied to the product as bfloat16 would hold it, as a separate kernel would read it.
+            // cap selects an activation of the stored product (0 none, 1 relu^2, 2 tanh-GELU, 3 SiLU, 4 xIELU
+            // with the constants `multiplier` and `second`), applied to the product as bfloat16 would hold it, as a separate kernel would read it.
             if (cap != 0.f) {
               const float z = __bfloat162float(__float2bfloat16_rn(v));
               if (cap == 1.f) {
@@ -455,8 +455,10 @@ gemv_stream_kernel(const bf16* __restrict__ a, const __grid_constant__ CUtensorM
                 v = r * r;
               } else if (cap == 2.f) {
                 v = 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-              } else {
+              } else if (cap == 3.f) {
                 v = z / (1.f + expf(-z));
+              } else {
+                v = xielu(z, multiplier, second);
               }
             }
             reinterpret_cast<bf16*>(out)[(size_t)token * n + col] = __float2bfloat16_rn(v);
@@ -509,7 +511,7 @@ constexpr size_t fixed_most() {
 
 template <int NT, int EPI, bool PENDING>
 int launch(const bf16* a, const bf16* w, void* out, int m, int n, int k, int inner, float multiplier, float cap,
-           const PendingStep& pending, int* err, cudaStream_t stream) {
+           float second, const PendingStep& pending, int* err, cudaStream_t stream) {
   const size_t fixed = (size_t)STAGES * STAGE_BYTES + ((partial_bytes(NT) + 15) & ~(size_t)15);
   const size_t smem = fixed + (PENDING ? sizeof(bf16) * NT * 8 * (size_t)(k + PENDING_PAD) + sizeof(float) * 2 * k : 0);
   constexpr size_t most = fixed_most<NT, PENDING>();
@@ -529,24 +531,24 @@ int launch(const bf16* a, const bf16* w, void* out, int m, int n, int k, int inn
   if (!make_map(&map_w, w, n, k)) return (int)cudaErrorInvalidValue;
   const int tiles = EPI == EPI_SWIGLU ? (inner + 7) / 8 : (n + TILE_ROWS - 1) / TILE_ROWS;
   launch_pdl(gemv_stream_kernel<NT, EPI, PENDING>, min(tiles, sms), THREADS, smem, stream, a, map_w, out, m, n, k, inner,
-             tiles, multiplier, cap, pending, err);
+             tiles, multiplier, cap, second, pending, err);
   return OMNIA_LAUNCH_RESULT();
 }
 
 template <int EPI, bool PENDING>
 int launch_rows(const bf16* a, const bf16* w, void* out, int m, int n, int k, int inner, float multiplier, float cap,
-                const PendingStep& pending, int* err, cudaStream_t stream) {
-  if (m <= 8) return launch<1, EPI, PENDING>(a, w, out, m, n, k, inner, multiplier, cap, pending, err, stream);
+                float second, const PendingStep& pending, int* err, cudaStream_t stream) {
+  if (m <= 8) return launch<1, EPI, PENDING>(a, w, out, m, n, k, inner, multiplier, cap, second, pending, err, stream);
   if (PENDING) return (int)cudaErrorInvalidValue;  // sixteen normalised rows and the weights do not fit beside the ring
-  return launch<2, EPI, false>(a, w, out, m, n, k, inner, multiplier, cap, pending, err, stream);
+  return launch<2, EPI, false>(a, w, out, m, n, k, inner, multiplier, cap, second, pending, err, stream);
 }
 
 }  // namespace
 
-// epilogue: 0 store bfloat16 [m, n] (cap 1, 2, 3: relu^2, tanh-GELU or SiLU of the product; 0: as it is); 1 SwiGLU, w = [gate rows | up rows] with n = 2 * inner,
+// epilogue: 0 store bfloat16 [m, n] (cap 1, 2, 3: relu^2, tanh-GELU or SiLU of the product, 4: xIELU with the constants `multiplier` and `second`; 0: as it is); 1 SwiGLU, w = [gate rows | up rows] with n = 2 * inner,
 // out bfloat16 [m, inner] (cap > 0: the clamped unit min(gate, cap) * sigmoid(multiplier * min(gate, cap)) * (clamp(up, +-cap) + 1); cap < 0: relu(gate) * up); 2 soft cap, out float32 [m, n]. err: the device error word.
 extern "C" int omnia_gemv_stream(const void* a, const void* w, void* out, int m, int n, int k, int epilogue,
-                                 float multiplier, float cap, int* err, cudaStream_t stream) {
+                                 float multiplier, float cap, float second, int* err, cudaStream_t stream) {
   if (m == 0 || n == 0) return 0;
   if (m > 16 || k % 8 != 0 || k <= 0) return (int)cudaErrorInvalidValue;
   if (((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(w)) & 15) != 0) return (int)cudaErrorInvalidValue;
@@ -555,12 +557,12 @@ extern "C" int omnia_gemv_stream(const void* a, const void* w, void* out, int m,
   const PendingStep none{};
   if (epilogue == EPI_SWIGLU) {
     if (n % 2) return (int)cudaErrorInvalidValue;
-    return launch_rows<EPI_SWIGLU, false>(ap, wp, out, m, n, k, n / 2, cap > 0.f ? multiplier : 1.f, cap, none, err, stream);
+    return launch_rows<EPI_SWIGLU, false>(ap, wp, out, m, n, k, n / 2, cap > 0.f ? multiplier : 1.f, cap, 0.f, none, err, stream);
   }
   if (epilogue == EPI_SOFTCAP)
-    return launch_rows<EPI_SOFTCAP, false>(ap, wp, out, m, n, k, 0, multiplier, cap, none, err, stream);
-  if (epilogue != EPI_STORE || cap < 0.f || cap > 3.f) return (int)cudaErrorInvalidValue;
-  return launch_rows<EPI_STORE, false>(ap, wp, out, m, n, k, 0, 1.f, cap, none, err, stream);
+    return launch_rows<EPI_SOFTCAP, false>(ap, wp, out, m, n, k, 0, multiplier, cap, 0.f, none, err, stream);
+  if (epilogue != EPI_STORE || cap < 0.f || cap > 4.f) return (int)cudaErrorInvalidValue;
+  return launch_rows<EPI_STORE, false>(ap, wp, out, m, n, k, 0, cap == 4.f ? multiplier : 1.f, cap, second, none, err, stream);
 }
 
 extern "C" int omnia_gemv_stream_pending_max_k(void) { return PENDING_MAX_K; }
@@ -581,8 +583,8 @@ extern "C" int omnia_gemv_stream_pending(const float* x, float* x_out, const voi
   const bf16* wp = (const bf16*)w;
   if (epilogue == EPI_SWIGLU) {
     if (n % 2) return (int)cudaErrorInvalidValue;
-    return launch_rows<EPI_SWIGLU, true>(nullptr, wp, out, m, n, k, n / 2, 1.f, 0.f, pending, err, stream);
+    return launch_rows<EPI_SWIGLU, true>(nullptr, wp, out, m, n, k, n / 2, 1.f, 0.f, 0.f, pending, err, stream);
   }
   if (epilogue != EPI_STORE) return (int)cudaErrorInvalidValue;
-  return launch_rows<EPI_STORE, true>(nullptr, wp, out, m, n, k, 0, 1.f, 0.f, pending, err, stream);
+  return launch_rows<EPI_STORE, true>(nullptr, wp, out, m, n, k, 0, 1.f, 0.f, 0.f, pending, err, stream);
 }

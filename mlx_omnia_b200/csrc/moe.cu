@@ -2,7 +2,9 @@
 // host which token went where:
 //
 //   route     per token: router logits in float32, softmax over all router outputs, choice by
-//             score + correction, the `top` largest; the weights are the scores themselves. Router
+//             score + correction, the `top` largest (optionally only among the experts of the groups
+//             whose two largest choice scores sum highest); the weights are the scores themselves, or
+//             the chosen ones' shares of their sum times a constant. Router
 //             outputs at or beyond `experts` name identity experts (they have no tensors).
 //   plan      one block: where each expert's rows begin in the sorted order, and the list of row
 //             tiles (expert, first row, rows) that the grouped products walk.
@@ -42,8 +44,8 @@ __device__ __forceinline__ float gated_unit(float gate, float up, float alpha, f
 template <typename T, int TOK, int THREADS, int CHUNK>
 __global__ void __launch_bounds__(THREADS)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
-                 int tokens, int outputs, int experts, int hidden, int top, int sigmoid_scores,
-                 int* __restrict__ choice, float* __restrict__ weight, int* __restrict__ counts) {
+                 int tokens, int outputs, int experts, int hidden, int top, int sigmoid_scores, int groups,
+                 int keep_groups, int normalise, float weight_scale, int* __restrict__ choice, float* __restrict__ weight, int* __restrict__ counts) {
   pdl_wait();
   pdl_launch_dependents();
   constexpr int WARPS = THREADS / 32;
@@ -51,7 +53,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
   extern __shared__ __align__(16) float route_s[];
   const int padded = (outputs + 3) / 4 * 4;
   float* hrow = route_s;                           // [TOK][hidden]
-  float* scores = hrow + (size_t)TOK * hidden;     // [TOK][padded] logits, then scores; [TOK][padded] choice scores
+  float* scores = hrow + (size_t)TOK * hidden;     // [TOK][padded] logits, then scores; [TOK][padded] choice scores; [TOK][padded] groups
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t0 = blockIdx.x * TOK, live = min(TOK, tokens - t0);
   for (int tok = 0; tok < TOK; ++tok)
@@ -125,6 +127,31 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
     pick[e] = s + (correction ? correction[e] : 0.f);
   }
   __syncwarp();
+  if (groups > 1 && keep_groups < groups) {
+    // A group of neighbouring outputs scores the sum of its two largest choice scores (its one, if it has
+    // one); outputs outside the `keep_groups` best groups (of equal ones the lowest) are taken out.
+    float* group = scores + (size_t)(2 * TOK + warp) * padded;
+    const int size = outputs / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float first = -INFINITY, second = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        const float v = pick[e];
+        if (v > first) second = first, first = v;
+        else if (v > second) second = v;
+      }
+      group[g] = size > 1 ? first + second : first;
+    }
+    __syncwarp();
+    for (int e = lane; e < outputs; e += 32) {
+      const int mine = e / size;
+      const float v = group[mine];
+      int better = 0;
+      for (int g = 0; g < groups; ++g) better += group[g] > v || (group[g] == v && g < mine);
+      if (better >= keep_groups) pick[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  float chosen_sum = 0.f;
   for (int k = 0; k < top; ++k) {
     // The largest choice score not taken yet; of equal ones the lowest index. A row of NaNs still
     // gets `top` different experts (the lowest indices).
@@ -149,8 +176,14 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
       weight[(size_t)t * top + k] = score[best_e];
       if (best_e < experts) atomicAdd(counts + best_e, 1);
       pick[best_e] = -INFINITY;
+      chosen_sum += score[best_e];
     }
     __syncwarp();
+  }
+  if (normalise || weight_scale != 1.f) {
+    chosen_sum = __shfl_sync(0xffffffffu, chosen_sum, 0);
+    const float factor = normalise ? weight_scale / (chosen_sum + 1e-20f) : weight_scale;
+    for (int k = lane; k < top; k += 32) weight[(size_t)t * top + k] *= factor;
   }
 }
 
@@ -503,36 +536,41 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, const T* __restri
 
 template <typename T, int TOK, int THREADS, int CHUNK>
 int launch_route(const T* h, const float* router, const float* correction, int tokens, int outputs, int experts,
-                 int hidden, int top, int sigmoid_scores, int* choice, float* weight, int* counts, size_t smem,
-                 cudaStream_t stream) {
+                 int hidden, int top, int sigmoid_scores, int groups, int keep_groups, int normalise, float weight_scale,
+                 int* choice, float* weight, int* counts, size_t smem, cudaStream_t stream) {
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(moe_route_kernel<T, TOK, THREADS, CHUNK>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
   launch_pdl(moe_route_kernel<T, TOK, THREADS, CHUNK>, (tokens + TOK - 1) / TOK, THREADS, smem, stream, h, router, correction, tokens,
-             outputs, experts, hidden, top, sigmoid_scores, choice, weight, counts);
+             outputs, experts, hidden, top, sigmoid_scores, groups, keep_groups, normalise, weight_scale, choice, weight, counts);
   return OMNIA_LAUNCH_RESULT();
 }
 
 }  // namespace
 
 extern "C" int omnia_moe_route(const void* h, const float* router, const float* correction, int tokens, int outputs,
-                               int experts, int hidden, int top, int sigmoid_scores, int* choice, float* weight,
-                               int* counts, int dtype, cudaStream_t stream) {
+                               int experts, int hidden, int top, int sigmoid_scores, int groups, int keep_groups,
+                               int normalise, float weight_scale, int* choice, float* weight, int* counts, int dtype,
+                               cudaStream_t stream) {
   if (tokens == 0) return 0;
+  if (groups < 1 || outputs % groups || keep_groups < 1 || keep_groups > groups || top > keep_groups * (outputs / groups))
+    return (int)cudaErrorInvalidValue;
   if (top < 1 || top > outputs || experts < 0 || experts > outputs || outputs > 4096) return (int)cudaErrorInvalidValue;
   const int padded = (outputs + 3) / 4 * 4;
-  auto bytes = [&](int tok) { return ((size_t)tok * hidden + (size_t)2 * tok * padded) * sizeof(float); };
+  auto bytes = [&](int tok) { return ((size_t)tok * hidden + (size_t)(groups > 1 ? 3 : 2) * tok * padded) * sizeof(float); };
   // Eight tokens a block where there are enough tokens to fill the GPU so and their rows fit.
   const bool many = tokens >= 8 * omnia_sm_count() && bytes(8) <= 160 * 1024;
   if (bytes(1) > 200 * 1024) return (int)cudaErrorInvalidValue;
   OMNIA_DISPATCH_DTYPE(dtype, {
     if (many)
       return launch_route<T, 8, 256, 4>((const T*)h, router, correction, tokens, outputs, experts, hidden, top,
-                                        sigmoid_scores, choice, weight, counts, bytes(8), stream);
+                                        sigmoid_scores, groups, keep_groups, normalise, weight_scale, choice, weight, counts,
+                                        bytes(8), stream);
     return launch_route<T, 1, 1024, 1>((const T*)h, router, correction, tokens, outputs, experts, hidden, top,
-                                       sigmoid_scores, choice, weight, counts, bytes(1), stream);
+                                       sigmoid_scores, groups, keep_groups, normalise, weight_scale, choice, weight, counts,
+                                       bytes(1), stream);
   });
   return (int)cudaErrorInvalidValue;
 }

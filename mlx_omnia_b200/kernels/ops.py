@@ -919,11 +919,11 @@ def _library_mm(a: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 
 
 def _gemv_stream(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epilogue: int, multiplier: float = 1.0,
-                 cap: float = 0.0) -> torch.Tensor:
+                 cap: float = 0.0, second: float = 0.0) -> torch.Tensor:
     """The product of up to 16 rows on the weight-streaming kernel (epilogue 0 store, 1 SwiGLU, 2 soft cap)."""
     fn = _function("gemv_stream", "omnia_gemv_stream",
-                   [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p])
-    _check(fn(_ptr(a), _ptr(weight), _ptr(out), a.shape[0], weight.shape[0], a.shape[1], epilogue, multiplier, cap,
+                   [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_void_p])
+    _check(fn(_ptr(a), _ptr(weight), _ptr(out), a.shape[0], weight.shape[0], a.shape[1], epilogue, multiplier, cap, second,
               _ptr(error_word(a.device)), _stream()), "gemv_stream")
     return out
 
@@ -1173,24 +1173,26 @@ def streams_leave(xs: torch.Tensor, branch: torch.Tensor, mix: torch.Tensor | No
     return h
 
 
-ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2}
+ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "xielu": 3}
 
 
-def activation(z: torch.Tensor, kind: str) -> torch.Tensor:
-    """relu(z)^2, the tanh form of GELU, or SiLU, element by element in float32."""
+def activation(z: torch.Tensor, kind: str, constants: tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
+    """relu(z)^2, the tanh form of GELU, SiLU, or xIELU with its two constants (`rise` z^2 + z / 2 above
+    zero, `fall` (e^z - 1 - z) + z / 2 below), element by element in float32."""
     act = torch.empty_like(z)
-    fn = _function("elementwise", "omnia_activation", [c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p])
-    _check(fn(_ptr(z), _ptr(act), z.numel(), ACTIVATIONS[kind], _code(z.dtype), _stream()), "activation")
+    fn = _function("elementwise", "omnia_activation",
+                   [c_void_p, c_void_p, c_longlong, c_int, c_float, c_float, c_int, c_void_p])
+    _check(fn(_ptr(z), _ptr(act), z.numel(), ACTIVATIONS[kind], *constants, _code(z.dtype), _stream()), "activation")
     return act
 
 
-def linear_act(a: torch.Tensor, weight: torch.Tensor, kind: str) -> torch.Tensor:
+def linear_act(a: torch.Tensor, weight: torch.Tensor, kind: str, constants: tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
     """act(a @ weight^T): a few bfloat16 rows run on the weight-streaming kernel with the activation
     in its epilogue; otherwise the library's product and the activation kernel."""
     if _skinny(a, weight):
         out = torch.empty(a.shape[0], weight.shape[0], dtype=a.dtype, device=a.device)
-        return _gemv_stream(a, weight, out, 0, 1.0, float(ACTIVATIONS[kind] + 1))
-    return activation(_library_mm(a, weight), kind)
+        return _gemv_stream(a, weight, out, 0, constants[0], float(ACTIVATIONS[kind] + 1), constants[1])
+    return activation(_library_mm(a, weight), kind, constants)
 
 
 # ------------------------------------------------------------------------------------
@@ -1495,19 +1497,37 @@ LATENT_MAX_RANK = 512
 
 def latent_prepare(proj: torch.Tensor, q_col: int, heads: int, q_dim: int, down_col: int, rank: int, rot: int,
                    weight: torch.Tensor, eps: float, inv_freq: torch.Tensor, positions: torch.Tensor,
-                   kv: KVView) -> None:
+                   kv: KVView, half_pairs: bool = False, amount: float = 1.0, cq_col: int = 0,
+                   cq_weight: torch.Tensor | None = None) -> torch.Tensor | None:
     """Per projected row: the RMS-normed latent (columns [down_col, down_col + rank)) and the rotated
     shared key part (the `rot` columns after it) go to the row's cache slot; the last `rot` dims of
     each of the `heads` query heads (each `q_dim` wide, from `q_col`) are rotated in place. The rotation
-    pairs dims (2i, 2i + 1) over the first 2 * len(inv_freq) of the `rot`."""
+    pairs dims (2i, 2i + 1), or with `half_pairs` (i, i + half), over the first 2 * len(inv_freq) of the
+    `rot`; cosine and sine are multiplied by `amount`. With `cq_weight` (and `heads` 0) the queries have a
+    latent too: columns [cq_col, cq_col + len(cq_weight)), RMS-normed with that weight, are returned."""
     store = kv.writes
+    cq = None if cq_weight is None else torch.empty(proj.shape[0], cq_weight.shape[0], dtype=proj.dtype, device=proj.device)
     fn = _function("attention_latent", "omnia_latent_prepare",
                    [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int,
-                    c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p])
+                    c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int,
+                    c_int, c_void_p, c_void_p])
     _check(fn(_ptr(proj), proj.shape[1], q_col, heads, q_dim, down_col, rank, rot, _ptr(weight), eps, _ptr(inv_freq),
               2 * inv_freq.shape[0], _ptr(positions), _ptr(kv.slot_mapping) if store else None, _ptr(kv.pages),
-              kv.pages.shape[0] * kv.page_size, proj.shape[0], _code(proj.dtype), _ptr(error_word(proj.device)),
+              kv.pages.shape[0] * kv.page_size, int(half_pairs), amount, cq_col, 0 if cq is None else cq.shape[1],
+              _ptr(cq_weight), _ptr(cq), proj.shape[0], _code(proj.dtype), _ptr(error_word(proj.device)),
               _stream()), "latent_prepare")
+    return cq
+
+
+def latent_rotate(q: torch.Tensor, rot: int, inv_freq: torch.Tensor, positions: torch.Tensor, half_pairs: bool,
+                  amount: float) -> None:
+    """In place: the last `rot` dims of every query head of q [tokens, heads, q_dim] turned as
+    `latent_prepare` turns them."""
+    tokens, heads, q_dim = q.shape
+    fn = _function("attention_latent", "omnia_latent_rotate",
+                   [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_int, c_void_p])
+    _check(fn(_ptr(q), q.stride(0), heads, q_dim, rot, _ptr(inv_freq), 2 * inv_freq.shape[0], int(half_pairs), amount,
+              _ptr(positions), tokens, _code(q.dtype), _stream()), "latent_rotate")
 
 
 def latent_tc_supported(q_lat: torch.Tensor, q_rot: torch.Tensor, out: torch.Tensor, scale: float) -> bool:
@@ -1598,11 +1618,14 @@ def batched_mm(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | None, experts: int, top: int,
-              counts: torch.Tensor, scoring: str = "softmax") -> tuple[torch.Tensor, torch.Tensor]:
+              counts: torch.Tensor, scoring: str = "softmax", groups: int = 1, keep_groups: int = 1,
+              normalise: bool = False, weight_scale: float = 1.0) -> tuple[torch.Tensor, torch.Tensor]:
     """Per row of `h`: float32 logits against `router` (float32 [outputs, hidden]), softmax over all
     outputs (or, with `scoring` "sigmoid", every output's own sigmoid), the `top` largest of score +
     correction; -> (choice int32 [rows, top], weight float32
-    [rows, top]: the chosen outputs' scores, not renormalised). Outputs at or beyond `experts` are identity experts; the
+    [rows, top]: the chosen outputs' scores; with `normalise` divided by their sum (+ 1e-20); times
+    `weight_scale`). With `groups` > 1 the outputs form that many equal runs; a run's score is the sum of its
+    two largest choice scores, and only outputs of the `keep_groups` best runs can be chosen. Outputs at or beyond `experts` are identity experts; the
     others are counted into `counts` (int32 [experts], zero before the call)."""
     rows, hidden = h.shape
     choice = torch.empty(rows, top, dtype=torch.int32, device=h.device)
@@ -1610,10 +1633,10 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
     if scoring not in ("softmax", "sigmoid"):
         raise KernelError(f"router scores are a softmax or sigmoids, not {scoring!r}")
     fn = _function("moe", "omnia_moe_route",
-                   [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
-                    c_int, c_void_p])
+                   [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                    c_void_p, c_void_p, c_void_p, c_int, c_void_p])
     _check(fn(_ptr(h), _ptr(router), _ptr(correction), rows, router.shape[0], experts, hidden, top,
-              int(scoring == "sigmoid"), _ptr(choice), _ptr(weight), _ptr(counts), _code(h.dtype), _stream()), "moe_route")
+              int(scoring == "sigmoid"), groups, keep_groups, int(normalise), weight_scale, _ptr(choice), _ptr(weight), _ptr(counts), _code(h.dtype), _stream()), "moe_route")
     return choice, weight
 
 
@@ -1646,7 +1669,8 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
                 tensor_cores: bool | None = None, tcgen05: bool | None = None,
                 table: torch.Tensor | None = None, token_ids: torch.Tensor | None = None,
                 alpha: float = 1.0, limit: float = 0.0, scoring: str = "softmax", weigh: str = "output",
-                extra: torch.Tensor | None = None) -> torch.Tensor:
+                extra: torch.Tensor | None = None, groups: int = 1, keep_groups: int = 1, normalise: bool = False,
+                weight_scale: float = 1.0, combine: bool = True) -> "torch.Tensor | ExpertRows":
     """A routed mixture of gated feed-forward experts over the rows of `h` [rows, hidden]:
     y = sum over a row's `top` choices of score * expert(h), expert e being
     down[e] (silu(gate_e h) * (up_e h)) with gate_up [experts, 2 inner, hidden] (gate rows, then up
@@ -1662,7 +1686,10 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
     `scoring`: the router's scores are a "softmax" over all outputs or every output's own "sigmoid".
     `weigh` "input": y = sum of expert(score * h) instead: a choice's score multiplies what its expert
     is given (the product in float32, rounded once), and the experts' outputs are added as they are.
-    `extra` [rows, hidden]: added to y in the same pass (an expert that every row uses)."""
+    `extra` [rows, hidden]: added to y in the same pass (an expert that every row uses).
+    `groups`, `keep_groups`, `normalise`, `weight_scale`: how the choice is narrowed and weighted (`moe_route`).
+    `combine` False (no `extra`, no identity experts, weights on the outputs): the choices' rows and their
+    weights are returned as they are, for `depth_step` to sum on their way into the residual."""
     if weigh not in ("output", "input"):
         raise KernelError(f"a choice's weight goes on its expert's output or input, not {weigh!r}")
     rows, hidden = h.shape
@@ -1682,7 +1709,8 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
     if table is not None:
         choice, weight = moe_route_table(token_ids[:rows], table, experts, counts)
     else:
-        choice, weight = moe_route(h, router, correction, experts, top, counts, scoring)
+        choice, weight = moe_route(h, router, correction, experts, top, counts, scoring, groups, keep_groups, normalise,
+                                   weight_scale)
     ints = torch.empty(2 * pairs + experts + 1 + 3 * max_tiles + 1, dtype=torch.int32, device=device)
     place, source = ints[:pairs], ints[pairs: 2 * pairs]
     offsets = ints[2 * pairs: 2 * pairs + experts + 1]
@@ -1726,6 +1754,10 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
                        hidden, 1, alpha, limit, _code(h.dtype), int(tensor_cores), _stream()), "moe_product")
         _check(product(_ptr(act), None, _ptr(down), _ptr(out), _ptr(tiles), _ptr(tile_count), max_tiles, hidden, inner, 0,
                        1.0, 0.0, _code(h.dtype), int(tensor_cores), _stream()), "moe_product")
+    if not combine:
+        if extra is not None or weigh != "output" or (router is not None and router.shape[0] != experts):
+            raise KernelError("rows that are summed elsewhere have no extra branch, no identity experts and weigh outputs")
+        return ExpertRows(out, place, weight, top)
     y = torch.empty_like(h)
     fn = _function("moe", "omnia_moe_combine",
                    [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
@@ -1734,6 +1766,162 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
     return y
 
 
+@dataclass
+class ExpertRows:
+    """A routed mixture's outputs before they are summed: y[t] = sum_k weight[t, k] * rows[place[t, k]]."""
+
+    rows: torch.Tensor  # [pairs, hidden], in sorted order
+    place: torch.Tensor  # int32 [tokens * top]
+    weight: torch.Tensor  # float32 [tokens, top]
+    top: int
+
+
 class _NoStep:
     """Stands in for a step where an op is called on its own (tests of single kernels)."""
     workspace = None
+
+
+# ------------------------------------------------------------------------------------
+# Layer norm and the end of a parallel block (csrc/depth.cu)
+
+
+def layernorm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """h = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias, x float32 [rows, hidden] -> `dtype`."""
+    rows, hidden = x.shape
+    h = torch.empty(rows, hidden, dtype=dtype, device=x.device)
+    fn = _function("depth", "omnia_layernorm",
+                   [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(x), _ptr(weight), _ptr(bias), eps, _ptr(h), rows, hidden, _code(dtype), _stream()), "layernorm")
+    return h
+
+
+class DepthHistory:
+    """What a pass's layers leave for the depth averages of later ones: the embedding output and a place
+    for every layer's result."""
+
+    def __init__(self, first: torch.Tensor, layers: int) -> None:
+        self.first = first
+        self.results = torch.empty(layers, *first.shape, dtype=torch.float32, device=first.device)
+
+
+def depth_history(step: StepContext, x: torch.Tensor, layers: int, count: int) -> DepthHistory:
+    """This pass's history; made by the layer that finds only the embedding output ahead of it (`count` 1),
+    whose residual `x` that is."""
+    if step.workspace is None:
+        step.workspace = {}
+    made = step.workspace.setdefault("pass", {})
+    if count == 1:
+        made["depth_history"] = DepthHistory(x, layers)
+    held = made.get("depth_history")
+    if held is None:
+        raise KernelError("a depth average whose first layer has not run in this pass")
+    return held
+
+
+def depth_step(x: torch.Tensor, branch: torch.Tensor, second: "torch.Tensor | ExpertRows | None",
+               history: DepthHistory | None, coef: torch.Tensor | None, norm_weight: torch.Tensor | None,
+               norm_bias: torch.Tensor | None, norm: str | None, eps: float,
+               keep: bool = True) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """r = x + branch + second; with `coef` (float32 [count + 1]) x' = sum_j coef[j] X_j + coef[count] r over the
+    history's `count` entries, and r is kept as the next of them (`keep` False: nobody reads it); without, x' = r.
+    Then h = norm(x') ("layer": with weight and bias; "rms": with weight; None: no h) in the branch's dtype.
+    `second` may be routed experts' rows, which are weighted and summed here. -> (x' float32, a new tensor; h)"""
+    rows, hidden = x.shape
+    x_out = torch.empty_like(x)
+    h = torch.empty(rows, hidden, dtype=branch.dtype, device=x.device) if norm is not None else None
+    experts = second if isinstance(second, ExpertRows) else None
+    count = 0 if coef is None else coef.shape[0] - 1
+    if coef is not None and not 1 <= count <= history.results.shape[0]:
+        raise KernelError(f"a depth average over {count} earlier results of {history.results.shape[0]} layers")
+    fn = _function("depth", "omnia_depth_step",
+                   [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                    c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(x), _ptr(branch), None if experts is not None else _ptr(second),
+              None if experts is None else _ptr(experts.rows), None if experts is None else _ptr(experts.place),
+              None if experts is None else _ptr(experts.weight), 0 if experts is None else experts.top,
+              None if coef is None else _ptr(history.first), None if coef is None else _ptr(history.results), count, int(keep),
+              _ptr(coef), _ptr(x_out), _ptr(norm_weight), _ptr(norm_bias), {None: 0, "layer": 1, "rms": 2}[norm], eps,
+              _ptr(h), rows, hidden, _code(branch.dtype), _stream()), "depth_step")
+    return x_out, h
+
+
+# ------------------------------------------------------------------------------------
+# A gated recurrence whose gates read the current token only (csrc/mingru.cu)
+
+MINGRU_MAX_WARPS = 16
+MINGRU_MAX_CLUSTER = 8
+
+
+def mingru_segments(longest: int, channels: int, requests: int, sms: int) -> tuple[int, int]:
+    """(warps a block, blocks a cluster) that the recurrence kernel cuts a request's portion over: segments of
+    about 16 tokens, more blocks to a cluster only while the SMs are not filled."""
+    warps = max(1, min(MINGRU_MAX_WARPS, longest // 16))
+    cluster = 1
+    while (cluster < MINGRU_MAX_CLUSTER and longest >= 32 * warps * cluster
+           and -(-channels // 32) * requests * cluster < 4 * sms):
+        cluster *= 2
+    return warps, cluster
+
+
+def mingru(proj: torch.Tensor, z_col: int, u_col: int, g_col: int, z_bias: torch.Tensor | None, u_bias: torch.Tensor | None,
+           S: torch.Tensor, step: StepContext, segments: tuple[int, int] | None = None) -> torch.Tensor:
+    """S_t = (1 - z) S_(t-1) + z cand per channel, request by request from `S` [slots, channels] (float32,
+    updated in place), with z = sigmoid(column of z_col + z_bias), u = column of u_col + u_bias, cand = u + 1/2
+    where u >= 0 and sigmoid(u) below. -> S_t * silu(columns of g_col) as [tokens, channels] in proj's type.
+    `segments`: (warps, blocks of a cluster) a portion is cut over (None: the op's choice)."""
+    tokens, C = proj.shape[0], S.shape[1]
+    warps, cluster = segments or mingru_segments(step.max_q_len, C, step.num_seqs, sm_count(proj.device))
+    out = torch.empty(tokens, C, dtype=proj.dtype, device=proj.device)
+    fn = _function("mingru", "omnia_mingru",
+                   [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                    c_int, c_int, c_int, c_void_p, c_int, c_void_p])
+    _check(fn(_ptr(proj), proj.shape[1], z_col, u_col, g_col, _ptr(z_bias), _ptr(u_bias), C, _ptr(S), _ptr(step.cu_seqlens),
+              _ptr(step.state_slots), step.num_seqs, int(step.decode_only), warps, cluster, _ptr(out), _code(proj.dtype),
+              _stream()), "mingru")
+    return out
+
+
+# ------------------------------------------------------------------------------------
+# Convolved projections and heads of several softmax maps (csrc/conv_heads.cu)
+
+CONV_HEADS_MAX_TAPS = 16
+
+
+def conv_heads_prepare(proj: torch.Tensor, col0: int, bias: torch.Tensor | None, taps: torch.Tensor, state: torch.Tensor,
+                       step: StepContext, heads: int, kv_heads: int, maps: int, dk: int, dv: int, d: int,
+                       inv_freq: torch.Tensor | None, half_pairs: bool, amount: float, kv: KVView) -> torch.Tensor:
+    """A step's projected rows (channels q | k | v from column `col0`, `bias` float32 [channels]) behind a causal
+    convolution over time (`taps` float32 [K, channels], the last row the current token's; the request's last
+    K - 1 inputs in `state` [slots, K - 1, channels], moved on), q and k then rotated over the first
+    2 * len(inv_freq) of every map's `dk` dims (neighbours, or with `half_pairs` half-split; cosine and sine
+    times `amount`). Into the cache (`kv_heads` > 0; rows of `d`): a head's `maps` key maps side by side, and
+    its `dv` values, both filled up with zeros. -> queries [tokens, heads * maps, d], each zero but for its
+    own map's dims, so that attention over the cache's rows scores every map by itself."""
+    tokens, stride = proj.shape
+    channels = taps.shape[1]
+    q = torch.empty(tokens, heads * maps, d, dtype=proj.dtype, device=proj.device)
+    k_ptr, v_ptr, page_stride, nkv, kdim, vdim = kv_layout(kv)
+    if kdim != d or vdim != d or (kv_heads and nkv != kv_heads):
+        raise KernelError(f"the cache keeps {nkv} rows of {kdim} and {vdim}, the mixer makes {kv_heads} of {d}")
+    fn = _function("conv_heads", "omnia_conv_heads_prepare",
+                   [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                    c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                    c_longlong, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p])
+    _check(fn(_ptr(proj), stride, col0, _ptr(bias), _ptr(taps), taps.shape[0], channels, _ptr(state), _ptr(step.cu_seqlens),
+              _ptr(step.state_slots), step.num_seqs, heads, kv_heads, maps, dk, dv, d, _ptr(inv_freq),
+              0 if inv_freq is None else 2 * inv_freq.shape[0], int(half_pairs), amount, _ptr(step.positions),
+              _ptr(kv.slot_mapping), _ptr(q), k_ptr, v_ptr, page_stride, kv.page_size, kv.pages.shape[0] * kv.page_size,
+              tokens, int(step.decode_only), _code(proj.dtype), _ptr(error_word(proj.device)), _stream()),
+           "conv_heads_prepare")
+    return q
+
+
+def map_difference(maps: torch.Tensor, heads: int, d: int, dv: int, lam: float, eps: float, factor: float) -> torch.Tensor:
+    """maps [tokens, heads * 2 * d], two rows of `d` a head of which the first `dv` count: o = first - lam * second,
+    divided by its root mean square (eps inside the root), times `factor`. -> [tokens, heads * dv]"""
+    tokens = maps.shape[0]
+    out = torch.empty(tokens, heads * dv, dtype=maps.dtype, device=maps.device)
+    fn = _function("conv_heads", "omnia_map_difference",
+                   [c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_int, c_int, c_void_p])
+    _check(fn(_ptr(maps), heads, d, dv, lam, eps, factor, _ptr(out), tokens, _code(maps.dtype), _stream()), "map_difference")
+    return out

@@ -12,7 +12,13 @@ from __future__ import annotations
 import torch
 
 from mlx_omnia_b200.kernels import ops
-from mlx_omnia_b200.parts.base import POSITIONS, KVSpec, Mixer, PartSpec, TensorSpec, register_mixer
+from mlx_omnia_b200.parts.base import POSITIONS, KVSpec, Mixer, PartSpec, StateSpec, TensorSpec, register_mixer
+
+
+def _no_amount(position, what: str) -> None:
+    """Refuse a position part that wants cosine and sine multiplied by something."""
+    if getattr(position, "amount", 1.0) != 1.0:
+        raise ValueError(f"{what} does not scale cosine and sine")
 
 
 @register_mixer("gqa_attention")
@@ -44,6 +50,7 @@ class GQAAttention(Mixer):
         self.position = POSITIONS.build(position or PartSpec("none"))
         if getattr(self.position, "pairing", "half") != "half":
             raise ValueError("gqa_attention rotates half-split pairs")
+        _no_amount(self.position, "gqa_attention")
 
     def kv_spec(self) -> KVSpec:
         return KVSpec.keys_and_values(self.kv_heads, self.head_dim, self.window)
@@ -119,7 +126,11 @@ class LatentAttention(Mixer):
     is cached, one row per position. This engine never expands the cache: uk is folded into the query
     (q_lat = uk_h^T q_plain) and uv applied to the attention's output in latent space.
     scale:    multiplies the scores
-    position: a rotary part with interleaved pairing over the first `dims` of the rot_dim
+    position: a rotary part over the first `dims` of the rot_dim, of either pairing; its `amount` multiplies
+              cosine and sine
+    q_rank:   None, or the width of a latent of the queries' own: c_q = RMSnorm(dq h) with weight `dq.norm` (eps
+              `norm_eps`), and the query heads are uq c_q (tensors `dq` [q_rank, hidden], `dq.norm`, `uq`
+              [heads * (dim + rot_dim), q_rank] instead of `q`)
     sink:     the softmax's denominator also holds exp(sink_h) (tensor `sink` [heads], unscaled)
     gated:    head h's output is multiplied by sigmoid(g(h))_h (tensor `g` [heads, hidden])
     window:   None, or how many latest positions are visible
@@ -132,14 +143,16 @@ class LatentAttention(Mixer):
 
     def __init__(self, hidden: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float,
                  norm_eps: float, position: PartSpec, sink: bool = True, gated: bool = True,
-                 window: int | None = None) -> None:
+                 window: int | None = None, q_rank: int | None = None) -> None:
         if kv_rank > ops.LATENT_MAX_RANK:
             raise ValueError(f"latent_attention takes a latent of at most {ops.LATENT_MAX_RANK}")
         self.hidden, self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank = hidden, heads, dim, rot_dim, vdim, kv_rank
         self.scale, self.norm_eps, self.sink, self.gated, self.window = float(scale), float(norm_eps), sink, gated, window
         self.position = POSITIONS.build(position)
-        if getattr(self.position, "pairing", None) != "interleaved":
-            raise ValueError("latent_attention rotates interleaved pairs")
+        self.q_rank = q_rank
+        if getattr(self.position, "pairing", None) not in ("interleaved", "half"):
+            raise ValueError("latent_attention needs a rotary position part")
+        self.half_pairs, self.amount = self.position.pairing == "half", self.position.amount
         if self.position.dims > rot_dim:
             raise ValueError(f"{self.position.dims} rotary dims do not fit a rotated part of {rot_dim}")
 
@@ -148,7 +161,12 @@ class LatentAttention(Mixer):
 
     def tensors(self) -> dict[str, TensorSpec]:
         H, qd = self.heads, self.dim + self.rot_dim
-        specs = {"q": TensorSpec((H * qd, self.hidden)), "dkv": TensorSpec((self.kv_rank + self.rot_dim, self.hidden)),
+        if self.q_rank is None:
+            specs = {"q": TensorSpec((H * qd, self.hidden))}
+        else:
+            specs = {"dq": TensorSpec((self.q_rank, self.hidden)), "dq.norm": TensorSpec((self.q_rank,), "vector"),
+                     "uq": TensorSpec((H * qd, self.q_rank))}
+        specs |= {"dkv": TensorSpec((self.kv_rank + self.rot_dim, self.hidden)),
                  "dkv.norm": TensorSpec((self.kv_rank,), "vector"), "uk": TensorSpec((H * self.dim, self.kv_rank)),
                  "uv": TensorSpec((H * self.vdim, self.kv_rank)), "o": TensorSpec((self.hidden, H * self.vdim))}
         if self.sink:
@@ -161,9 +179,12 @@ class LatentAttention(Mixer):
         super().load(tensors, runtime)
         self.position.load({}, runtime)
         H, qd = self.heads, self.dim + self.rot_dim
-        # One operand [q | down | gate] (rows padded to a multiple of 8).
-        rows = [tensors["q"], tensors["dkv"]]
-        self.down_col = H * qd
+        # One operand [q, or the queries' down projection | down | gate] (rows padded to a multiple of 8).
+        rows = [tensors["q" if self.q_rank is None else "dq"], tensors["dkv"]]
+        self.down_col = rows[0].shape[0]
+        self.uq = self.q_norm = None
+        if self.q_rank is not None:
+            self.uq, self.q_norm = tensors["uq"].contiguous(), tensors["dq.norm"].contiguous()
         self.gate_col = self.down_col + self.kv_rank + self.rot_dim
         total = self.gate_col
         if self.gated:
@@ -184,9 +205,15 @@ class LatentAttention(Mixer):
         H, qd, step = self.heads, self.dim + self.rot_dim, ctx.step
         proj = ops.linear(h, self.in_proj)
         tokens = proj.shape[0]
-        ops.latent_prepare(proj, 0, H, qd, self.down_col, self.kv_rank, self.rot_dim, self.down_norm, self.norm_eps,
-                           self.position.table(), step.positions, ctx.kv)
-        q = proj[:, : H * qd].view(tokens, H, qd)
+        table = self.position.table()
+        cq = ops.latent_prepare(proj, 0, H if self.q_rank is None else 0, qd, self.down_col, self.kv_rank, self.rot_dim,
+                                self.down_norm, self.norm_eps, table, step.positions, ctx.kv, self.half_pairs, self.amount,
+                                0, self.q_norm)
+        if cq is None:
+            q = proj[:, : H * qd].view(tokens, H, qd)
+        else:
+            q = ops.linear(cq, self.uq).view(tokens, H, qd)
+            ops.latent_rotate(q, self.rot_dim, table, step.positions, self.half_pairs, self.amount)
         q_lat = ops.batched_mm(q[:, :, : self.dim].transpose(0, 1), self.uk)  # [H, tokens, rank]
         o_lat = torch.empty(H, tokens, self.kv_rank, dtype=proj.dtype, device=proj.device)
         ops.latent_attention(q_lat, q[:, :, self.dim:], ctx.kv, step, self.scale, self.sink_logits,
@@ -264,6 +291,7 @@ class SinkWindowAttention(Mixer):
         self.interleaved = getattr(self.position, "pairing", "half") == "interleaved"
         if getattr(self.position, "dims", 0) > dim:
             raise ValueError(f"{self.position.dims} rotary dims do not fit a head of {dim}")
+        _no_amount(self.position, "sink_window_attention")
 
     def kv_spec(self) -> KVSpec:
         return KVSpec(((self.kv_heads, self.dim), (self.kv_heads, self.vdim)), self.window, keep_first=self.keep_first,
@@ -343,3 +371,99 @@ class SinkWindowAttention(Mixer):
         return ops.paged_attention(q, ctx.kv, ctx.step, self.scale, gate=proj if self.gated else None,
                                    gate_col=col0 + self.gate_col, sink=self.sink_logits, window=self.window,
                                    keep_first=self.keep_first, chunk=self.chunk, softcap=self.softcap)
+
+
+@register_mixer("differential_attention")
+class DifferentialAttention(Mixer):
+    """Grouped-query causal attention whose heads are the difference of two softmax maps over the same values,
+    behind a short causal convolution over time of every projected channel.
+
+    hidden, heads, kv_heads: sizes; dim: width of a map's query and key (a head has 2 * dim of them, laid out
+    [map 1, map 2]); vdim: width of a value head
+    scale:    multiplies q.k in both maps
+    diff:     lambda = exp(lq1.lk1) - exp(lq2.lk2) + diff, one number for the layer; a head's output is
+              a = a_1 - lambda a_2, divided by its own root mean square over vdim (`norm_eps` inside the root),
+              times 1 - diff
+    conv:     taps of the convolution (q, k and v each; the last column is the current token's)
+    position: PartSpec of the rotary encoding over the first `dims` of every map of q and k, after the convolution
+    bias:     q, k and v projections have biases, added ahead of the convolution
+    window:   None, or how many latest positions are visible
+    own_kv:   False for a layer without k and v tensors that reads another layer's cache with its own queries
+
+    The cache's rows: a head's two key maps side by side and its values, both filled up to one width `row`
+    (a multiple of 8), so that what runs over them is ordinary grouped-query attention of 2 * heads query
+    heads, each zero outside its own map's dims, and the two maps of a head share one fetch of keys and values.
+
+    Tensors: q [heads * 2 * dim, hidden], k [kv_heads * 2 * dim, hidden], v [kv_heads * vdim, hidden], each with
+    `.b` and `.conv` [rows, conv]; lq1, lk1, lq2, lk2 [dim]; o [hidden, heads * vdim].
+    State (float32): the projections' last conv - 1 values."""
+
+    graph_safe = True
+    graph_safe_mixed = True
+    MAPS = 2
+
+    def __init__(self, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, diff: float, conv: int,
+                 norm_eps: float, position: PartSpec | None = None, bias: bool = True, window: int | None = None,
+                 own_kv: bool = True) -> None:
+        if kv_heads < 1 or heads % kv_heads:
+            raise ValueError(f"{heads} query heads do not divide into {kv_heads} groups")
+        if not 1 <= conv <= ops.CONV_HEADS_MAX_TAPS:
+            raise ValueError(f"a convolution of {conv} taps (1 to {ops.CONV_HEADS_MAX_TAPS})")
+        self.row = -(-max(self.MAPS * dim, vdim) // 8) * 8
+        if self.row > 512:
+            raise ValueError(f"differential_attention takes two maps of at most 256 and values of at most 512, got {dim} and {vdim}")
+        self.hidden, self.heads, self.kv_heads, self.dim, self.vdim = hidden, heads, kv_heads, dim, vdim
+        self.scale, self.diff, self.conv, self.norm_eps = float(scale), float(diff), conv, float(norm_eps)
+        self.bias, self.window, self.own_kv = bias, window, own_kv
+        self.position = POSITIONS.build(position or PartSpec("none"))
+        if getattr(self.position, "dims", 0) > dim:
+            raise ValueError(f"{self.position.dims} rotary dims do not fit a map of {dim}")
+
+    def kv_spec(self) -> KVSpec:
+        return KVSpec.keys_and_values(self.kv_heads, self.row, self.window)
+
+    def _names(self) -> dict[str, int]:
+        """The projections and their rows."""
+        rows = {"q": self.heads * self.MAPS * self.dim}
+        if self.own_kv:
+            rows |= {"k": self.kv_heads * self.MAPS * self.dim, "v": self.kv_heads * self.vdim}
+        return rows
+
+    def state_spec(self):
+        return {"conv": StateSpec((max(self.conv - 1, 1), sum(self._names().values())))}
+
+    def tensors(self) -> dict[str, TensorSpec]:
+        specs = {"o": TensorSpec((self.hidden, self.heads * self.vdim))}
+        for name, rows in self._names().items():
+            specs[name], specs[name + ".conv"] = TensorSpec((rows, self.hidden)), TensorSpec((rows, self.conv), "vector")
+            if self.bias:
+                specs[name + ".b"] = TensorSpec((rows,), "vector")
+        return specs | {name: TensorSpec((self.dim,), "vector") for name in ("lq1", "lk1", "lq2", "lk2")}
+
+    def load(self, tensors, runtime) -> None:
+        super().load(tensors, runtime)
+        self.position.load({}, runtime)
+        names = self._names()
+        rows = [tensors[name] for name in names]  # one operand [q | k | v] (rows padded to a multiple of 8)
+        pad = -sum(names.values()) % 8
+        if pad:
+            rows.append(torch.zeros(pad, self.hidden, dtype=rows[0].dtype, device=rows[0].device))
+        self.in_proj = torch.cat(rows, dim=0).contiguous()
+        self.channel_bias = torch.cat([tensors[name + ".b"] for name in names]).contiguous() if self.bias else None
+        self.taps = torch.cat([tensors[name + ".conv"] for name in names]).t().contiguous()
+        self.o = tensors["o"].contiguous()
+        a, b, c, d = (tensors[name].double() for name in ("lq1", "lk1", "lq2", "lk2"))
+        self.lam = float(torch.exp((a * b).sum()) - torch.exp((c * d).sum()) + self.diff)
+
+    def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
+        if ctx.kv is None:
+            raise RuntimeError("an attention mixer needs cache pages")
+        if ctx.kv.writes and not self.own_kv:
+            raise RuntimeError("a mixer without k/v projections cannot own a cache entry")
+        q = ops.conv_heads_prepare(ops.linear(h, self.in_proj), 0, self.channel_bias, self.taps, ctx.state["conv"], ctx.step,
+                                   self.heads, self.kv_heads if self.own_kv else 0, self.MAPS, self.dim, self.vdim, self.row,
+                                   self.position.table(), getattr(self.position, "pairing", "half") == "half",
+                                   getattr(self.position, "amount", 1.0), ctx.kv)
+        maps = ops.paged_attention(q, ctx.kv, ctx.step, self.scale, window=self.window)
+        return ops.linear(ops.map_difference(maps, self.heads, self.row, self.vdim, self.lam, self.norm_eps, 1.0 - self.diff),
+                          self.o)

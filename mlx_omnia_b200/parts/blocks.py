@@ -20,7 +20,7 @@ import torch
 from mlx_omnia_b200.kernels import ops
 from mlx_omnia_b200.parts.base import (FEED_FORWARDS, MIXERS, NORMS, Block, Norm, PartSpec, StateSpec, TensorSpec,
                                        register_block)
-from mlx_omnia_b200.parts.norms import RMSNorm
+from mlx_omnia_b200.parts.norms import LayerNorm, RMSNorm
 
 
 def residual_step(x: torch.Tensor, branch: torch.Tensor, branch_norm: Norm | None, out_norm: Norm | None,
@@ -346,3 +346,67 @@ class BranchNormBlock(Block):
             return x, h2
         m = self.feed_forward.forward(h2, ctx)
         return x, self._step(x, m, self.norms["norm2"], exit_norm, True)
+
+
+@register_block("parallel")
+class ParallelBlock(Block):
+    """One norm whose output both branches read: r = x + mixer(norm(x)) + feed_forward(norm(x)). The
+    feed-forward may be missing.
+
+    mixer:        PartSpec of the mixer; feed_forward: PartSpec or None
+    norm:         PartSpec of the norm (tensors under `norm1`)
+    averaged:     None: x' = r. Otherwise the number of earlier results, n: what goes on is the depth average
+                  x' = sum_(j < n) dwa[j] X_j + dwa[n] r, X_0 being the embedding output and X_j the result r of
+                  the j-th layer, so the block must be the n-th one run (tensor `dwa` [n + 1])
+    depth:        with `averaged`, how many layers the model runs (places for their results)
+
+    The residual sum, the experts' weighted sum (where the feed-forward gives its rows), the average and
+    the next reader's norm are one pass over a row."""
+
+    def __init__(self, mixer: PartSpec, feed_forward: PartSpec | None, norm: PartSpec, averaged: int | None = None,
+                 depth: int = 0, mixer_name: str = "mix", feed_forward_name: str = "mlp") -> None:
+        if averaged is not None and not 1 <= averaged <= depth:
+            raise ValueError(f"a depth average over {averaged} earlier results in a model of {depth} layers")
+        self.mixer = MIXERS.build(mixer)
+        self.feed_forward = FEED_FORWARDS.build(feed_forward) if feed_forward is not None else None
+        self.entry_norm = NORMS.build(norm)
+        self.averaged, self.depth = averaged, depth
+        self.mixer_name, self.feed_forward_name = mixer_name, feed_forward_name
+
+    def children(self):
+        yield self.mixer_name, self.mixer
+        if self.feed_forward is not None:
+            yield self.feed_forward_name, self.feed_forward
+        yield "norm1", self.entry_norm
+
+    def tensors(self) -> dict[str, TensorSpec]:
+        specs = {f"{name}.{local}": spec for name, part in self.children() for local, spec in part.tensors().items()}
+        if self.averaged is not None:
+            specs["dwa"] = TensorSpec((self.averaged + 1,), "vector")
+        return specs
+
+    def load(self, tensors, runtime) -> None:
+        super().load(tensors, runtime)
+        for name, part in self.children():
+            prefix = name + "."
+            part.load({k[len(prefix):]: v for k, v in tensors.items() if k.startswith(prefix)}, runtime)
+        self.coef = tensors["dwa"].contiguous() if self.averaged is not None else None
+
+    def forward(self, x, h, ctx, exit_norm):
+        h = ops.settle(h)
+        branch = self.mixer.forward(h, ctx)
+        second = None
+        if self.feed_forward is not None:
+            rows = getattr(self.feed_forward, "gives_rows", False)
+            second = self.feed_forward.forward_rows(h, ctx) if rows else self.feed_forward.forward(h, ctx)
+        history = None
+        if self.coef is not None:
+            history = ops.depth_history(ctx.step, x, self.depth, self.averaged)
+        kind = "layer" if isinstance(exit_norm, LayerNorm) else \
+            "rms" if isinstance(exit_norm, RMSNorm) and exit_norm.groups == 1 else None
+        x, out = ops.depth_step(x, branch, second, history, self.coef, exit_norm.weight if kind else None,
+                                exit_norm.bias if kind == "layer" else None, kind, exit_norm.eps if kind else 0.0,
+                                keep=self.averaged != self.depth)
+        if kind is None and exit_norm is not None:
+            out = exit_norm.forward(x)
+        return x, out

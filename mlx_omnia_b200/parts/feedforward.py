@@ -45,7 +45,9 @@ class GatedMLP(FeedForward):
 class DenseMLP(FeedForward):
     """down(act(up(h))), no biases and no gate.
 
-    hidden, inner: widths; activation: "relu2" (the square of relu), "gelu_tanh" or "silu".
+    hidden, inner: widths; activation: "relu2" (the square of relu), "gelu_tanh", "silu" or "xielu".
+    xielu has two learned numbers p, q (tensor `act` [2]): softplus(p) z^2 + z / 2 for z > 0,
+    (1/2 + softplus(q)) (e^z - 1 - z) + z / 2 for z <= 0.
     Tensors: `up` [inner, hidden], `down` [hidden, inner].
     """
 
@@ -55,14 +57,21 @@ class DenseMLP(FeedForward):
         self.hidden, self.inner, self.activation = hidden, inner, activation
 
     def tensors(self) -> dict[str, TensorSpec]:
-        return {"up": TensorSpec((self.inner, self.hidden)), "down": TensorSpec((self.hidden, self.inner))}
+        specs = {"up": TensorSpec((self.inner, self.hidden)), "down": TensorSpec((self.hidden, self.inner))}
+        if self.activation == "xielu":
+            specs["act"] = TensorSpec((2,), "vector")
+        return specs
 
     def load(self, tensors, runtime) -> None:
         super().load(tensors, runtime)
         self.up, self.down = tensors["up"].contiguous(), tensors["down"].contiguous()
+        self.constants = (0.0, 0.0)
+        if self.activation == "xielu":
+            rise, fall = torch.nn.functional.softplus(tensors["act"].double()).tolist()
+            self.constants = (rise, 0.5 + fall)
 
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
-        return ops.linear(ops.linear_act(h, self.up, self.activation), self.down)
+        return ops.linear(ops.linear_act(h, self.up, self.activation, self.constants), self.down)
 
 
 @register_feed_forward("clamped_glu_mlp")
@@ -172,13 +181,23 @@ class RoutedExperts(FeedForward):
               expert is given the token multiplied by its score and its output counts as it is
     shared_inner: None, or the inner width of one more gated expert (`shared.gate`, `shared.up`,
               `shared.down`) that every token uses unweighted and whose output is added
+    groups, keep_groups: the outputs form `groups` equal runs of neighbours; a run's score is the sum of its two
+              largest choice scores, and only outputs of the `keep_groups` best runs can be chosen
+    normalise: the weights are the chosen scores divided by their sum (+ 1e-20)
+    weight_scale: multiplies the weights
     Tensors: `router` [experts + identity, hidden], `correction` [experts + identity], and per expert i
     `e<i>.gate`, `e<i>.up` [inner, hidden], `e<i>.down` [hidden, inner] (stacked at load).
     """
 
     def __init__(self, hidden: int, inner: int, experts: int, top: int, identity: int = 0,
                  correction: bool = True, scoring: str = "softmax", weigh: str = "output",
-                 shared_inner: int | None = None) -> None:
+                 shared_inner: int | None = None, groups: int = 1, keep_groups: int = 1, normalise: bool = False,
+                 weight_scale: float = 1.0) -> None:
+        outputs = experts + identity
+        if groups < 1 or outputs % groups or not 1 <= keep_groups <= groups or top > keep_groups * (outputs // groups):
+            raise ValueError(f"routed_experts: {top} of {outputs} outputs in {groups} groups of which {keep_groups} are kept")
+        self.groups, self.keep_groups = groups, keep_groups
+        self.normalise, self.weight_scale = bool(normalise), float(weight_scale)
         if experts < 1 or identity < 0 or not 1 <= top <= experts + identity:
             raise ValueError(f"routed_experts of {experts} experts and {identity} identity ones, {top} a token")
         if scoring not in ("softmax", "sigmoid") or weigh not in ("output", "input"):
@@ -217,5 +236,20 @@ class RoutedExperts(FeedForward):
         extra = None
         if self.shared_gate_up is not None:
             extra = ops.linear(ops.linear_swiglu(h, self.shared_gate_up), self.shared_down)
+        return self._experts(h, ctx, extra, True)
+
+    @property
+    def gives_rows(self) -> bool:
+        """Whether `forward_rows` may stand in for `forward`."""
+        return self.shared_inner is None and self.identity == 0 and self.weigh == "output"
+
+    def forward_rows(self, h: torch.Tensor, ctx) -> "ops.ExpertRows":
+        """The chosen experts' outputs and weights, not yet summed (a block that takes them sums them on their
+        way into the residual, in float32)."""
+        return self._experts(h, ctx, None, False)
+
+    def _experts(self, h, ctx, extra, combine: bool):
         return ops.moe_experts(h, self.router, self.correction, self.gate_up, self.down, self.top, ctx.step,
-                               scoring=self.scoring, weigh=self.weigh, extra=extra)
+                               scoring=self.scoring, weigh=self.weigh, extra=extra, groups=self.groups,
+                               keep_groups=self.keep_groups, normalise=self.normalise, weight_scale=self.weight_scale,
+                               combine=combine)

@@ -1,4 +1,4 @@
-"""Norms. `rms_norm` covers the three conventions one trunk can mix: a plain weight,
+"""Norms. `layer_norm` takes the mean off and has a weight and a bias. `rms_norm` covers the three conventions one trunk can mix: a plain weight,
 a centred weight stored as `w` and applied as `1 + w`, and no weight at all.
 
 Reference: the four block norms are centred and folded at load
@@ -48,3 +48,24 @@ class RMSNorm(Norm):
         if self.groups > 1:
             return ops.streams_enter(x, None, 1, self.weight, self.eps, self.groups, self.runtime.dtype)
         return ops.rmsnorm(x, self.weight, self.eps, self.runtime.dtype)
+
+
+@register_norm("layer_norm")
+class LayerNorm(Norm):
+    """h = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias over the last axis, in float32.
+
+    size: length of the normalised axis; eps: added to the mean squared deviation.
+    Tensors: `weight`, `bias` [size]."""
+
+    def __init__(self, size: int, eps: float) -> None:
+        self.size, self.eps, self.weight, self.bias = size, float(eps), None, None
+
+    def tensors(self) -> dict[str, TensorSpec]:
+        return {"weight": TensorSpec((self.size,), "vector"), "bias": TensorSpec((self.size,), "vector")}
+
+    def load(self, tensors, runtime) -> None:
+        super().load(tensors, runtime)
+        self.weight, self.bias = tensors["weight"].contiguous(), tensors["bias"].contiguous()
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.layernorm(x, self.weight, self.bias, self.eps, self.runtime.dtype)

@@ -20,6 +20,9 @@ and a silu or sigmoid gate.
 convolution, gates that are sigmoids of block-diagonal maps, S <- a S + sqrt(1 - a^2) i u with
 a = exp(-c r softplus(lam)), the output multiplied by a tanh-GELU branch.
 
+`min_gru` is a gated recurrence over channels whose gate and candidate read the current token only:
+S <- (1 - z) S + z cand, the output multiplied by silu(g(h)).
+
 `side_by_side` runs two mixers on the same input and adds their outputs with a constant each.
 """
 
@@ -201,6 +204,8 @@ class GatedStateAttention(Mixer):
         self.position = POSITIONS.build(position or PartSpec("none"))
         if getattr(self.position, "pairing", "half") != "half":
             raise ValueError("gated_state_attention rotates half-split pairs")
+        if getattr(self.position, "amount", 1.0) != 1.0:
+            raise ValueError("gated_state_attention does not scale cosine and sine")
         if getattr(self.position, "dims", 0) > dim:
             raise ValueError(f"{self.position.dims} rotary dims do not fit a head of {dim}")
 
@@ -318,6 +323,50 @@ class GatedChannelRecurrence(Mixer):
         return ops.gated_channel_recurrence(proj, col0, col0 + self.width, self.x_bias, self.y_bias, self.taps,
                                             self.conv_bias, self.gates, self.r_bias, self.i_bias, self.lam, self.c_decay,
                                             ctx.state["S"], ctx.state["conv"], ctx.step)
+
+
+@register_mixer("min_gru")
+class MinGRU(Mixer):
+    """hidden: model width; width: channels of the recurrence.
+
+    z = sigmoid(z h + z.b), u = x h + x.b; the candidate is u + 1/2 where u >= 0 and sigmoid(u) below;
+    S <- (1 - z) S + z candidate from S = 0; out = o (S * silu(g h)).
+
+    Tensors: z, x, g [width, hidden]; z.b, x.b [width]; o [hidden, width]. State (float32): S [width]."""
+
+    graph_safe = True
+    graph_safe_mixed = True
+    takes_pending = True  # h goes to the in-projection and nowhere else
+
+    def __init__(self, hidden: int, width: int) -> None:
+        if width < 1:
+            raise ValueError(f"min_gru of {width} channels")
+        self.hidden, self.width = hidden, width
+
+    def state_spec(self):
+        return StateSpec((self.width,), torch.float32)
+
+    def tensors(self) -> dict[str, TensorSpec]:
+        w, d = self.width, self.hidden
+        return {"z": TensorSpec((w, d)), "x": TensorSpec((w, d)), "g": TensorSpec((w, d)), "z.b": TensorSpec((w,), "vector"),
+                "x.b": TensorSpec((w,), "vector"), "o": TensorSpec((d, w))}
+
+    def load(self, tensors, runtime) -> None:
+        super().load(tensors, runtime)
+        rows = [tensors["z"], tensors["x"], tensors["g"]]  # one operand [z | x | g]
+        if 3 * self.width % 8:
+            rows.append(torch.zeros(8 - 3 * self.width % 8, self.hidden, dtype=rows[0].dtype, device=rows[0].device))
+        self.in_proj = torch.cat(rows, dim=0).contiguous()
+        self.z_bias, self.x_bias = tensors["z.b"].contiguous(), tensors["x.b"].contiguous()
+        self.o = tensors["o"].contiguous()
+
+    def forward(self, h, ctx) -> torch.Tensor:
+        return ops.linear(self.forward_heads(ops.linear(h, self.in_proj), 0, ctx), self.o)
+
+    def forward_heads(self, proj: torch.Tensor, col0: int, ctx) -> torch.Tensor:
+        """S * silu(g) for every channel, ahead of the output projection, from projected rows whose columns
+        from `col0` on are this mixer's input projection."""
+        return ops.mingru(proj, col0, col0 + self.width, col0 + 2 * self.width, self.z_bias, self.x_bias, ctx.state, ctx.step)
 
 
 @register_mixer("side_by_side")
