@@ -30,7 +30,10 @@ at equal width, depth, heads, window and experts; its kernels stand beside the l
 for the recurrence, of Fokalorn. `--only narezen` is that record for the Narezen design (attention beside a
 decayed linear-attention state in one mixer, a gated recurrence over channels, sigmoid-routed experts weighted
 on their inputs with a shared expert), beside Bobarax at equal width, depth, heads and experts; its kernels
-stand beside the like kernels of Bobarax.
+stand beside the like kernels of Bobarax. `--only rinirax` is that record for the Rinirax design (parallel blocks
+whose residual is averaged over depth, differential attention behind short convolutions, windowed latent
+attention, a gated recurrence over channels, group-limited experts), beside Narezen at equal width, depth,
+heads and experts; its kernels stand beside the like kernels of Narezen and, for latent attention, of Fokalorn.
 """
 
 from __future__ import annotations
@@ -1524,6 +1527,275 @@ def run_narezen(args) -> dict:
     return record
 
 
+def rinirax_config(size: dict) -> dict:
+    """Layers in fours: differential attention, a gated recurrence over channels, windowed latent attention, and
+    differential attention that reads the first one's cache; group-limited experts everywhere. A head's two maps
+    are half its value width each."""
+    H, G, d, D = size["heads"], size["kv"], size["dim"], size["width"]
+    moe = {"kind": "moe", "expert": {"ff": size["eff"]},
+           "router": {"experts": size["experts"], "top": size["top"], "groups": {"count": 4, "keep": 2}, "scale": 1.5}}
+    layers = []
+    for i in range(size["layers"]):
+        kind = i % 4
+        if kind in (0, 3):
+            mixer = {"heads": H, "kv_heads": G, "dim": d // 2, "vdim": d, "scale": (d // 2) ** -0.5, "diff": 0.4, "conv": 4,
+                     "rot": {"base": 100000.0, "dims": d // 2}}
+            if kind == 3:
+                mixer["kv_from"] = i - 3
+            layers.append({"type": "attention", "mixer": mixer, "mlp": moe})
+        elif kind == 1:
+            layers.append({"type": "mingru", "mixer": {"width": D}, "mlp": moe})
+        else:
+            mixer = {"heads": H, "dim": d, "rot_dim": 64, "vdim": d, "kv_rank": 4 * d, "q_rank": D // 2, "scale": (d + 64) ** -0.5,
+                     "mask": {"size": size["window"]},
+                     "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+            layers.append({"type": "latent_attention", "mixer": mixer, "mlp": moe})
+    return {"architecture": "Rinirax", "vocab": DOLUTAR_VOCAB, "width": D, "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def events_ms(fn, count: int, warm: int = 3) -> float:
+    """Milliseconds a call of `fn`, by CUDA events around `count` calls."""
+    import torch
+
+    for _ in range(warm):
+        fn()
+    torch.cuda.synchronize()
+    start, stop = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    start.record()
+    for _ in range(count):
+        fn()
+    stop.record()
+    torch.cuda.synchronize()
+    return start.elapsed_time(stop) / count
+
+
+def replayed_ms(fn, count: int, warm: int = 2) -> float:
+    """Milliseconds a call of `fn` takes inside a replayed CUDA graph of `count` calls (no launches from Python)."""
+    import torch
+
+    for _ in range(warm):
+        fn()
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for _ in range(count):
+            fn()
+    ms = events_ms(graph.replay, 3, 1) / count
+    del graph
+    return ms
+
+
+def step_alone(lens: list[int], starts: list[int], device):
+    """A step's metadata for kernels that are called on their own: requests that bring `lens` tokens after `starts`."""
+    import types
+
+    import torch
+
+    cu = [0]
+    for n in lens:
+        cu.append(cu[-1] + n)
+    held = [s + n for s, n in zip(starts, lens)]
+    ints = lambda values: torch.tensor(values, dtype=torch.int32, device=device)
+    return types.SimpleNamespace(
+        num_seqs=len(lens), q_lens=list(lens), num_tokens=cu[-1], cu_seqlens=ints(cu), state_slots=ints(list(range(len(lens)))),
+        positions=ints([s + i for s, n in zip(starts, lens) for i in range(n)]), seq_lens=ints(held), seq_lens_host=held,
+        max_q_len=max(lens), max_seq_len=max(held), decode_only=all(n == 1 for n in lens), workspace={"private": True})
+
+
+def whole_model_ms(raw: dict, args, vocab: int, generator) -> dict:
+    """Prefill of one prompt of --prefill-tokens and decode steps of --batch requests that end at --context tokens."""
+    import torch
+
+    from mlx_omnia_b200.engine.engine import Engine, EngineArgs
+    from mlx_omnia_b200.engine.step import StepEntry
+    from mlx_omnia_b200.kernels import ops
+
+    steps, warmup, batch, context, tokens = args.steps, max(args.warmup, 3), args.batch, args.context, args.prefill_tokens
+    engine = Engine.from_random(raw, SEED, EngineArgs(dtype="bfloat16", page_size=16, max_requests=batch + 1,
+                                                      cache_tokens=batch * (context + 16) + tokens + 16))
+    times = []
+    for index in range(warmup + 3):
+        request = engine.cache.open(f"p{index}")
+        ids = torch.randint(0, vocab, (tokens,), generator=generator).tolist()
+        torch.cuda.synchronize()
+        start, stop = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        start.record()
+        engine.runner.run([StepEntry(request, ids, [tokens - 1])])
+        stop.record()
+        torch.cuda.synchronize()
+        engine.cache.close(request.request_id)
+        times.append(start.elapsed_time(stop))
+    prefill_ms = statistics.median(times[warmup:])
+    requests = [engine.cache.open(f"d{i}") for i in range(batch)]
+    length = context - steps - warmup - 1
+    for r in requests:
+        engine.runner.run([StepEntry(r, torch.randint(0, vocab, (length,), generator=generator).tolist(), [])])
+    entries = lambda i: [StepEntry(r, [1 + i], [0]) for r in requests]
+    for i in range(warmup):
+        engine.runner.run(entries(i), copy=False)
+    torch.cuda.synchronize()
+    launches = ops.launches
+    start, stop = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    start.record()
+    for i in range(steps):
+        engine.runner.run(entries(warmup + i), copy=False)
+    stop.record()
+    torch.cuda.synchronize()
+    decode_ms = start.elapsed_time(stop) / steps
+    ops.raise_on_error(engine.runtime.device)
+    out = {"prefill_tokens_per_s": round(tokens * 1000.0 / prefill_ms, 1), "prefill_ms": round(prefill_ms, 3),
+           "decode_tokens_per_s": round(batch * 1000.0 / decode_ms, 1), "decode_ms": round(decode_ms, 4),
+           "launches_per_decode_step": (ops.launches - launches) // steps}
+    for r in requests:
+        engine.cache.close(r.request_id)
+    del engine
+    torch.cuda.empty_cache()
+    return out
+
+
+def run_rinirax(args) -> dict:
+    """Prefill and decode of Rinirax and of Narezen at equal sizes, then the new design's kernels alone (each replayed
+    from a CUDA graph), each beside the like kernel of Narezen, or for latent attention of Fokalorn."""
+    import torch
+
+    from mlx_omnia_b200.kernels import ops
+    from mlx_omnia_b200.parts.base import KVSpec, KVView
+
+    measured, peak_source = peaks()
+    hbm, flops_peak = measured["hbm_gbs"] * 1e9, measured["bf16_tflops"] * 1e12
+    g = torch.Generator().manual_seed(SEED)
+    batch, context, tokens = args.batch, args.context, args.prefill_tokens
+    dev, bf = torch.device("cuda:0"), torch.bfloat16
+
+    def kernels(size: dict) -> dict:
+        H, G, d, D, W = size["heads"], size["kv"], size["dim"], size["width"], size["window"]
+        E, top, F = size["experts"], size["top"], size["eff"]
+        out = {}
+
+        def note(name, fn, count, bytes_=None, flops=None):
+            ms = replayed_ms(fn, count)
+            entry = {"us": round(ms * 1000.0, 2)}
+            if bytes_ is not None:
+                entry.update(gb_s=round(bytes_ / ms / 1e6, 1), frac_hbm=round(bytes_ / (ms / 1e3) / hbm, 4))
+            if flops is not None:
+                entry.update(tflops=round(flops / ms / 1e9, 2), frac_tensor=round(flops / (ms / 1e3) / flops_peak, 4))
+            out[name] = entry
+
+        for mode, lens, starts in (("prefill", [tokens], [0]), ("decode", [1] * batch, [context - 1] * batch)):
+            st = step_alone(lens, starts, dev)
+            T, page, reps = sum(lens), 16, 5 if mode == "prefill" else 20
+            pages = -(-st.max_seq_len // page)
+            table = torch.arange(len(lens) * pages, dtype=torch.int32, device=dev).view(len(lens), pages)
+            slots = torch.cat([table[i].long()[(st.positions[st.cu_seqlens[i]: st.cu_seqlens[i + 1]] // page).long()] * page
+                               + st.positions[st.cu_seqlens[i]: st.cu_seqlens[i + 1]].long() % page for i in range(len(lens))])
+            cache = (torch.randn(len(lens) * pages, 2, G, page, d, device=dev) * 0.3).to(bf)
+            kv = KVView(cache, table, slots, page, None, True, KVSpec(((G, d), (G, d))))
+            # convolved, rotated projections into the cache, beside Narezen's rotated ones
+            cols = (H + 2 * G) * d
+            proj = (torch.randn(T, cols, device=dev) * 0.5).to(bf)
+            bias, taps = torch.zeros(cols, device=dev), torch.randn(4, cols, device=dev)
+            conv_state = torch.zeros(len(lens) + 1, 3, cols, device=dev)
+            inv = torch.tensor([100000.0 ** (-4.0 * i / d) for i in range(d // 4)], device=dev)
+            note(f"conv_heads_prepare_{mode}",
+                 lambda: ops.conv_heads_prepare(proj, 0, bias, taps, conv_state, st, H, G, 2, d // 2, d, d, inv, False, 1.0, kv),
+                 20, bytes_=T * (cols * 2 + (2 * H + 2 * G) * d * 2))
+            note(f"like:qkv_prepare_{mode}",
+                 lambda: ops.qkv_prepare(proj, 0, H * d, (H + G) * d, H, d, None, None, None, None, inv, st.positions, kv, True),
+                 20, bytes_=T * cols * 4)
+            # two maps of half the width a head, beside one map of the whole width with a sink
+            q2 = torch.zeros(T, H, 2, d, device=dev, dtype=bf)
+            q2[:, :, 0, : d // 2], q2[:, :, 1, d // 2:] = torch.randn(2, T, H, d // 2, device=dev).to(bf)
+            q2 = q2.view(T, 2 * H, d)
+            seen = sum(s + i + 1 for s, n in zip(starts, lens) for i in range(n))
+            held = sum(s + n for s, n in zip(starts, lens))
+            difference = ops.MapDifference(0.6, 1e-5, 0.6, d)
+            note(f"differential_attention_{mode}", lambda: ops.paged_attention(q2, kv, st, 0.125, difference=difference), reps,
+                 bytes_=held * 2 * G * d * 2 + 4 * T * H * d, flops=2 * seen * H * (d + 2 * d))
+            q = (torch.randn(T, H, d, device=dev) * 0.3).to(bf)
+            sink = torch.zeros(H, device=dev)
+            note(f"like:sink_attention_{mode}", lambda: ops.paged_attention(q, kv, st, 0.125, sink=sink), reps,
+                 bytes_=held * 2 * G * d * 2 + 4 * T * H * d, flops=4 * seen * H * d)
+            del q, q2, proj
+            # the latent's input step and attention, windowed without sink and gate, beside Fokalorn's over everything
+            rank, rot, qr = 4 * d, 64, D // 2
+            row = rank + rot
+            lcache = (torch.randn(len(lens) * pages, 1, 1, page, row, device=dev) * 0.3).to(bf)
+            low = [max(0, s + n - W) for s, n in zip(starts, lens)]
+            lkv = KVView(lcache, table, slots, page, W, True, KVSpec(((1, row),), W))
+            fkv = KVView(lcache, table, slots, page, None, True, KVSpec(((1, row),)))
+            down = (torch.randn(T, qr + row, device=dev) * 0.5).to(bf)
+            nw, nq = torch.ones(rank, device=dev), torch.ones(qr, device=dev)
+            linv = torch.tensor([10000.0 ** (-2.0 * i / rot) for i in range(rot // 2)], device=dev)
+            lq = (torch.randn(T, H, d + rot, device=dev) * 0.3).to(bf)
+            note(f"latent_inputs_{mode}", lambda: (ops.latent_prepare(down, 0, 0, d + rot, qr, rank, rot, nw, 1e-5, linv, st.positions,
+                                                                      lkv, True, 1.1, 0, nq),
+                                                   ops.latent_rotate(lq, rot, linv, st.positions, True, 1.1)), 20,
+                 bytes_=T * ((qr + row) * 4 + H * rot * 4))
+            fproj = (torch.randn(T, H * (d + rot) + row, device=dev) * 0.3).to(bf)
+            note(f"like:latent_prepare_{mode}", lambda: ops.latent_prepare(fproj, 0, H, d + rot, H * (d + rot), rank, rot, nw, 1e-5, linv,
+                                                                           st.positions, fkv), 20,
+                 bytes_=T * (row * 4 + H * rot * 4))
+            q_lat = (torch.randn(H, T, rank, device=dev) * 0.1).to(bf)
+            o_lat = torch.empty_like(q_lat)
+            wseen = sum(min(s + i + 1, W) for s, n in zip(starts, lens) for i in range(n))
+            wheld = sum(s + n - lo for s, n, lo in zip(starts, lens, low)) if mode == "decode" else held
+            note(f"latent_window_attention_{mode}", lambda: ops.latent_attention(q_lat, lq[:, :, d:], lkv, st, 0.07, None, None, o_lat), reps,
+                 bytes_=wheld * row * 2 + 2 * T * H * (row + rank), flops=2 * wseen * H * (row + rank))
+            gate = torch.zeros(T, H, device=dev, dtype=bf)
+            note(f"like:latent_attention_{mode}", lambda: ops.latent_attention(q_lat, lq[:, :, d:], fkv, st, 0.07, sink, gate, o_lat), reps,
+                 bytes_=held * row * 2 + 2 * T * H * (row + rank), flops=2 * seen * H * (row + rank))
+            del q_lat, o_lat, lcache, fproj, down, lq
+            # the recurrence over channels beside Narezen's
+            C, blocks, K = D, H, 4
+            bw = C // blocks
+            gproj = (torch.randn(T, 3 * C, device=dev) * 0.5).to(bf)
+            zb, S1 = torch.zeros(C, device=dev), torch.zeros(len(lens) + 1, C, device=dev)
+            note(f"mingru_{mode}", lambda: ops.mingru(gproj, 0, C, 2 * C, zb, zb, S1, st), 20, bytes_=T * C * 8 + 8 * len(lens) * C)
+            gates = torch.randn(blocks, bw, 2 * bw, device=dev) * bw ** -0.5
+            rtaps, rstate = torch.randn(C, K, device=dev) * 0.5, torch.zeros(len(lens) + 1, K - 1, C, device=dev)
+            note(f"like:gated_channel_recurrence_{mode}",
+                 lambda: ops.gated_channel_recurrence(gproj, 0, C, zb, zb, rtaps, zb, gates, zb, zb, zb, 8.0, S1, rstate, st), 5,
+                 bytes_=T * C * 6 + blocks * bw * 2 * bw * 4, flops=2 * T * C * 2 * bw)
+            del gproj
+            # the end of a block: both branches, the average over half the model's layers, the next norm
+            a, b = (torch.randn(T, D, device=dev).to(bf) for _ in range(2))
+            x, w = torch.randn(T, D, device=dev), torch.ones(D, device=dev)
+            count = max(size["layers"] // 2, 1)
+            history = ops.DepthHistory(x, size["layers"])
+            history.results.normal_()
+            coef = torch.full((count + 1,), 0.2, device=dev)
+            note(f"depth_step_{count}_earlier_{mode}", lambda: ops.depth_step(x, a, b, history, coef, w, w, "layer", 1e-5), 10,
+                 bytes_=T * D * (4 + 2 + 2 + 4 * count + 4 + 4 + 2))
+            note(f"like:add_rmsnorm_{mode}", lambda: ops.add_rmsnorm(x, a, w, 1e-5, w, 1e-5), 10, bytes_=T * D * (4 + 4 + 2 + 2))
+            del history
+            # experts chosen within the best groups (rows summed elsewhere), beside Narezen's
+            h = (torch.randn(T, D, device=dev) * 0.5).to(bf)
+            egu = (torch.randn(E, 2 * F, D, device=dev) * D ** -0.5).to(bf)
+            edn = (torch.randn(E, D, F, device=dev) * F ** -0.5).to(bf)
+            router, correction = torch.randn(E, D, device=dev) * 0.05, torch.randn(E, device=dev) * 0.1
+            used = E * (1.0 - (1.0 - top / E) ** T)
+            work = dict(bytes_=used * 3 * F * D * 2 + T * D * 4, flops=2 * T * top * 3 * F * D)
+            note(f"group_limited_experts_{mode}",
+                 lambda: ops.moe_experts(h, router, correction, egu, edn, top, st, scoring="sigmoid", groups=4, keep_groups=2,
+                                         normalise=True, weight_scale=1.5, combine=False), 5, **work)
+            note(f"like:sigmoid_input_weighted_experts_{mode}",
+                 lambda: ops.moe_experts(h, router, None, egu, edn, top, st, scoring="sigmoid", weigh="input"), 5, **work)
+            del egu, edn
+        ops.raise_on_error(dev)
+        return out
+
+    record = {"metric": "Rinirax beside Narezen at equal sizes", "unit": "tokens/s", "dtype": "bf16",
+              "data": "synthetic: seeded uniform-random token ids, random weights",
+              "config": {"prefill_tokens": tokens, "decode_batch": batch, "decode_context": context, "vocab": DOLUTAR_VOCAB,
+                         "peaks": peak_source}, "sizes": {}}
+    for name in ([args.size] if args.size else list(BOBARAX_SIZES)):
+        size = BOBARAX_SIZES[name]
+        record["sizes"][name] = {"rinirax": whole_model_ms(rinirax_config(size), args, DOLUTAR_VOCAB, g),
+                                 "narezen": whole_model_ms(narezen_config(size), args, DOLUTAR_VOCAB, g),
+                                 "kernels": kernels(size), "layers": size["layers"]}
+    return record
+
+
 def main() -> int:
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
@@ -1536,7 +1808,7 @@ def main() -> int:
                         help="with --only decode|prefill and OMNIA_TIMELINE=1 in the environment: one step's "
                              "kernels with the time each takes in the stream, on stderr")
     parser.add_argument("--only", choices=["all", "decode", "prefill", "mixed", "portions", "sampling", "products", "elementwise", "fokalorn",
-                                           "dolutar", "bobarax", "narezen"], default="all",
+                                           "dolutar", "bobarax", "narezen", "rinirax"], default="all",
                         help="time one part only (small cases for profilers); prints a short record")
     parser.add_argument("--config", type=int, choices=sorted(CONFIGS), default=2,
                         help="with --only: the sizes of another benchmark configuration (3: 36 layers, hidden 4096, "
@@ -1548,7 +1820,7 @@ def main() -> int:
     parser.add_argument("--portion", type=int, default=256,
                         help="--only mixed: tokens of a prompt that run beside --batch decoding requests")
     parser.add_argument("--size", choices=sorted(FOKALORN_SIZES), default=None,
-                        help="--only fokalorn, dolutar, bobarax or narezen: one size instead of all")
+                        help="--only fokalorn, dolutar, bobarax, narezen or rinirax: one size instead of all")
     args = parser.parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable":
@@ -1570,6 +1842,9 @@ def main() -> int:
         return 0
     if args.only == "narezen":
         print(json.dumps(run_narezen(args)))
+        return 0
+    if args.only == "rinirax":
+        print(json.dumps(run_rinirax(args)))
         return 0
     if args.only == "dolutar":
         print(json.dumps(run_dolutar(args)))

@@ -3,7 +3,8 @@
 // refuse. A window may keep the request's first `keep_first` positions visible for good, and the
 // softmax's denominator may hold one more term exp(sink[head]) that has no key and no value.
 // With `chunk` > 0 a query sees the keys of its own run of `chunk` positions only (runs counted from
-// position 0 of the request); with `softcap` > 0 a scaled score s becomes softcap * tanh(s / softcap).
+// position 0 of the request); with `maps` 2 two neighbouring query heads are the two maps of one head of
+// differential attention, and their difference is written (see MapDifference); with `softcap` > 0 a scaled score s becomes softcap * tanh(s / softcap).
 //
 // One warp per (token, query head). Keys are visited in chunks of 32 starting at the
 // lowest visible position; in a chunk every lane scores one key (a full dot product in
@@ -26,7 +27,8 @@ __global__ void paged_attention_generic_kernel(
     T* __restrict__ out,                    // [tokens, nq * dv]
     const float* __restrict__ sink,         // [nq] or null
     int num_seqs, int max_pages, int num_pages, int nq, int nkv, int d, int dv, int page_size,
-    int window, int keep_first, float scale, int chunk, float softcap, int* err) {
+    int window, int keep_first, float scale, int chunk, float softcap, int maps, const MapDifference difference,
+    int* err) {
   constexpr int ACC = MOST / 32;
   __shared__ float qs[4][MOST];
   const int t = blockIdx.x;
@@ -107,6 +109,26 @@ __global__ void paged_attention_generic_kernel(
     for (int k = 0; k < ACC; ++k) acc[k] *= alpha;
   }
   const float inv = l > 0.f ? 1.f / l : 0.f;
+  if (maps == 2) {
+    // The odd warp of a pair hands its map over (nq is even, so the pair is there or gone together).
+    if (warp & 1)
+#pragma unroll
+      for (int k = 0; k < ACC; ++k) qs[warp][lane + 32 * k] = acc[k] * inv;
+    __syncthreads();
+    if (warp & 1) return;
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < ACC; ++k) {
+      acc[k] = lane + 32 * k < difference.dv ? acc[k] * inv - difference.lambda * qs[warp + 1][lane + 32 * k] : 0.f;
+      ss += acc[k] * acc[k];
+    }
+    const float f = rsqrtf(warp_sum(ss) / (float)difference.dv + difference.eps) * difference.factor;
+    T* drow = out + ((size_t)t * (nq / 2) + head / 2) * difference.dv;
+#pragma unroll
+    for (int k = 0; k < ACC; ++k)
+      if (lane + 32 * k < difference.dv) drow[lane + 32 * k] = from_f32<T>(acc[k] * f);
+    return;
+  }
   T* orow = out + ((size_t)t * nq + head) * dv;
 #pragma unroll
   for (int k = 0; k < ACC; ++k) {
@@ -125,8 +147,12 @@ extern "C" int omnia_paged_attention_generic(
     const void* q, const void* k_pages, const void* v_pages, long long page_stride, const int* block_table,
     const int* cu_seqlens, const int* positions, const void* gate, int gate_stride, void* out, const float* sink,
     int tokens, int num_seqs, int max_pages, int num_pages, int nq, int nkv, int d, int dv, int page_size, int window,
-    int keep_first, float scale, int chunk, float softcap, int dtype, int* err, cudaStream_t stream) {
+    int keep_first, float scale, int chunk, float softcap, int maps, float lambda, float diff_eps, float diff_factor, int out_dv,
+    int dtype, int* err, cudaStream_t stream) {
   if (tokens == 0) return 0;
+  if (maps < 1 || maps > 2 || (maps == 2 && (nq % 2 || gate != nullptr || out_dv < 1 || out_dv > dv)))
+    return (int)cudaErrorInvalidValue;
+  const MapDifference difference{lambda, diff_eps, diff_factor, out_dv};
   if (d > 512 || dv > 512 || nkv <= 0 || nq % nkv != 0 || keep_first < 0 || (keep_first > 0 && window <= 0) ||
       chunk < 0 || softcap < 0.f || (chunk > 0 && keep_first > 0))
     return (int)cudaErrorInvalidValue;
@@ -136,12 +162,12 @@ extern "C" int omnia_paged_attention_generic(
       paged_attention_generic_kernel<T, 256><<<grid, 128, 0, stream>>>(
           (const T*)q, (const T*)k_pages, (const T*)v_pages, page_stride, block_table, cu_seqlens, positions, (const T*)gate,
           gate_stride, (T*)out, sink, num_seqs, max_pages, num_pages, nq, nkv, d, dv, page_size, window, keep_first, scale,
-          chunk, softcap, err);
+          chunk, softcap, maps, difference, err);
     else
       paged_attention_generic_kernel<T, 512><<<grid, 128, 0, stream>>>(
           (const T*)q, (const T*)k_pages, (const T*)v_pages, page_stride, block_table, cu_seqlens, positions, (const T*)gate,
           gate_stride, (T*)out, sink, num_seqs, max_pages, num_pages, nq, nkv, d, dv, page_size, window, keep_first, scale,
-          chunk, softcap, err);
+          chunk, softcap, maps, difference, err);
   });
   return OMNIA_LAUNCH_RESULT();
 }

@@ -26,6 +26,8 @@
 // Two more serve mixers whose queries read only their own run of positions and cap their scores:
 // `run` (a query at position i sees no key below i - i % run) and `softcap` (a scaled score s becomes
 // softcap * tanh(s / softcap) ahead of the softmax).
+// Compiled with -DMAPS=2, two neighbouring query heads are the two maps of one head of differential
+// attention, and what is written is their difference (see MapDifference), [tokens, nq / 2, dv].
 #include "common.cuh"
 
 #ifndef HEAD_DIM
@@ -33,6 +35,9 @@
 #endif
 #ifndef GROUP
 #define GROUP 2
+#endif
+#ifndef MAPS
+#define MAPS 1
 #endif
 
 namespace {
@@ -61,6 +66,7 @@ constexpr float LOG2E = 1.4426950408889634f;
 
 static_assert(D % 8 == 0 && D <= 256, "head size must be a multiple of 8, at most 256");
 static_assert(GROUP >= 1 && GROUP <= 16, "group size must be 1..16");
+static_assert(MAPS == 1 || (MAPS == 2 && GROUP % 2 == 0), "two maps to a head: an even number of query heads");
 
 typedef __nv_bfloat16 bf16;
 
@@ -245,7 +251,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pa
                          const bf16* __restrict__ gate, int gate_stride, bf16* __restrict__ out,
                          int max_pages, int num_pages, int nq, int nkv, int page_size, int window,
                          float scale, int keep_first, const float* __restrict__ sink, int run, float softcap,
-                         int* err) {
+                         const MapDifference difference, int* err) {
   pdl_wait();
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* qs = reinterpret_cast<bf16*>(smem_raw);   // [BM][ROW]
@@ -344,6 +350,45 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pa
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
   }
   const int t = lane & 3;
+  if constexpr (MAPS == 2) {
+    // A head's two maps are neighbouring rows, four lanes apart; both lanes hold the difference and each
+    // stores every other piece of it.
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int row = warp * 16 + (lane >> 2) + 8 * r;
+      const bool second = row & 1;
+      const float inv = l[r] > 0.f ? 1.f / l[r] : 0.f;
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < NT_O; ++j)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float mine = o[j][2 * r + e] * inv, other = __shfl_xor_sync(0xffffffffu, mine, 4);
+          const float d = second ? other - difference.lambda * mine : mine - difference.lambda * other;
+          o[j][2 * r + e] = d;
+          ss += d * d;
+        }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      const float f = rsqrtf(ss / (float)difference.dv + difference.eps) * difference.factor;
+      if (row >= rows) continue;
+      const size_t token = (size_t)(q_begin + tok0 + row / GROUP);
+      bf16* dst = out + (token * (nq / 2) + (kvh * GROUP + row % GROUP) / 2) * difference.dv;
+      const bool even = (difference.dv & 1) == 0;
+#pragma unroll
+      for (int j = 0; j < NT_O; ++j) {
+        const int dim = 8 * j + 2 * t;
+        if ((j & 1) != (int)second || dim >= difference.dv) continue;
+        const float v0 = o[j][2 * r] * f, v1 = o[j][2 * r + 1] * f;
+        if (even) {
+          *reinterpret_cast<__nv_bfloat162*>(dst + dim) = __floats2bfloat162_rn(v0, v1);
+        } else {
+          dst[dim] = __float2bfloat16_rn(v0);
+          if (dim + 1 < difference.dv) dst[dim + 1] = __float2bfloat16_rn(v1);
+        }
+      }
+    }
+  } else {
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int row = warp * 16 + (lane >> 2) + 8 * r;
@@ -366,6 +411,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pa
       *reinterpret_cast<__nv_bfloat162*>(dst + dim) = __floats2bfloat162_rn(v0, v1);
     }
   }
+  }
 }
 
 // Merge chunks c0..c1 of H heads of one token (heads head0 .., whose partials lie max_chunks apart),
@@ -383,7 +429,7 @@ template <int H>
 __device__ __forceinline__ void combine_heads(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                               size_t base, int max_chunks, int c0, int c1, const bf16* gate_row,
                                               bf16* out_row, float* stage, int stage_floats,
-                                              const float* sink = nullptr) {
+                                              const float* sink = nullptr, const MapDifference difference = {}) {
   const int lane = threadIdx.x & 31;
   constexpr int PER_LANE = (D + 31) / 32;
   float gate_v[H][PER_LANE];
@@ -437,6 +483,22 @@ __device__ __forceinline__ void combine_heads(const float* __restrict__ part_o, 
     }
     __syncwarp();  // the stage is read before the next round overwrites it
   }
+  if constexpr (MAPS == 2) {
+    static_assert(H == 2, "a head's two maps are merged together");
+    const float inv0 = total[0] > 0.f ? 1.f / total[0] : 0.f, inv1 = total[H - 1] > 0.f ? 1.f / total[H - 1] : 0.f;
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER_LANE; ++k) {
+      acc[0][k] = acc[0][k] * inv0 - difference.lambda * (acc[H - 1][k] * inv1);
+      if (lane + 32 * k < D) ss += acc[0][k] * acc[0][k];
+    }
+    const float f = rsqrtf(warp_sum(ss) / (float)difference.dv + difference.eps) * difference.factor;
+#pragma unroll
+    for (int k = 0; k < PER_LANE; ++k) {
+      const int dim = lane + 32 * k;
+      if (dim < difference.dv) out_row[dim] = __float2bfloat16_rn(acc[0][k] * f);
+    }
+  } else {
 #pragma unroll
   for (int h = 0; h < H; ++h) {
     if (sink != nullptr && mx[h] != -INFINITY) total[h] += exp2f(sink[h] * LOG2E - mx[h]);  // mx is in log2 units
@@ -449,6 +511,7 @@ __device__ __forceinline__ void combine_heads(const float* __restrict__ part_o, 
       if (gate_row) v *= 1.f / (1.f + expf(-gate_v[h][k]));
       out_row[(size_t)h * D + dim] = __float2bfloat16_rn(v);
     }
+  }
   }
 }
 
@@ -484,7 +547,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pag
                         bf16* __restrict__ out, int chunk_keys, int max_chunks, int max_pages,
                         int num_pages, int nq, int nkv, int page_size, int window, float scale,
                         const FusedQK fused, int keep_first, const float* __restrict__ sink, int run, float softcap,
-                        int* err) {
+                        const MapDifference difference, int* err) {
   // In the fused mode nothing up to the query fragments depends on the kernel before this one
   // (the lengths and tables were copied in before the step began, the keys and values of earlier
   // tokens were written in earlier steps), so the block's start and its first loads of the cache
@@ -809,17 +872,18 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pag
   __threadfence();
   // Two heads at a time (their loads travel together; one at a time where a head's rows would not
   // fit in registers twice), then the odd one.
-  constexpr int TOGETHER = D <= 128 ? 2 : 1;
+  constexpr int TOGETHER = MAPS == 2 || D <= 128 ? 2 : 1;
   // The block's rings are idle by now: the least they hold, in floats, stages the chunks' accumulators.
   constexpr int STAGE_FLOATS = WARPS * STAGES * 2 * DECODE_BN * ROW * (int)sizeof(bf16) / (int)sizeof(float);
 #pragma unroll 1
   for (int r = 0; r + TOGETHER <= GROUP; r += TOGETHER) {
     const int head = kvh * GROUP + r;
     combine_heads<TOGETHER>(part_o, part_ml, ((size_t)blockIdx.z * nq + head) * max_chunks, max_chunks, c0, c1,
-                     gate ? gate + token * gate_stride + (size_t)head * D : nullptr, out + (token * nq + head) * D,
-                     reinterpret_cast<float*>(smem_raw), STAGE_FLOATS, sink ? sink + head : nullptr);
+                     gate ? gate + token * gate_stride + (size_t)head * D : nullptr,
+                     MAPS == 2 ? out + (token * (nq / 2) + head / 2) * difference.dv : out + (token * nq + head) * D,
+                     reinterpret_cast<float*>(smem_raw), STAGE_FLOATS, sink ? sink + head : nullptr, difference);
   }
-  if (GROUP % TOGETHER) {
+  if constexpr (GROUP % TOGETHER != 0) {
     const int head = kvh * GROUP + GROUP - 1;
     combine_heads<1>(part_o, part_ml, ((size_t)blockIdx.z * nq + head) * max_chunks, max_chunks, c0, c1,
                      gate ? gate + token * gate_stride + (size_t)head * D : nullptr, out + (token * nq + head) * D,
@@ -842,9 +906,11 @@ extern "C" int omnia_attention_prefill_tc(const void* q, const void* pages, cons
                                           const int* work, int blocks, const void* gate,
                                           int gate_stride, void* out, int max_pages, int num_pages,
                                           int nq, int nkv, int page_size, int window, float scale,
-                                          int keep_first, const float* sink, int run, float softcap, int* err,
+                                          int keep_first, const float* sink, int run, float softcap, float lambda,
+                                          float diff_eps, float diff_factor, int out_dv, int* err,
                                           cudaStream_t stream) {
   if (blocks == 0) return 0;
+  if (MAPS == 2 && (gate != nullptr || sink != nullptr || out_dv < 1 || out_dv > D)) return (int)cudaErrorInvalidValue;
   if (nq != nkv * GROUP || keep_first < 0 || (keep_first > 0 && window <= 0) || run < 0 || softcap < 0.f ||
       (run > 0 && keep_first > 0))
     return (int)cudaErrorInvalidValue;
@@ -859,7 +925,7 @@ extern "C" int omnia_attention_prefill_tc(const void* q, const void* pages, cons
   launch_pdl(attention_prefill_kernel, dim3(blocks, nkv), 128, smem, stream, 
       (const bf16*)q, (const bf16*)pages, block_table, cu_seqlens, seq_lens, work, (const bf16*)gate,
       gate_stride, (bf16*)out, max_pages, num_pages, nq, nkv, page_size, window, scale, keep_first, sink, run,
-      softcap, err);
+      softcap, MapDifference{lambda, diff_eps, diff_factor, out_dv}, err);
   return OMNIA_LAUNCH_RESULT();
 }
 
@@ -882,8 +948,11 @@ extern "C" int omnia_attention_decode_tc(const void* q, const void* pages, const
                                          const void* proj, int proj_stride, int q_col, int k_col, int v_col,
                                          float eps, const float* inv_freq, const long long* slot_mapping,
                                          int spread, int keep_first, const float* sink, int run, float softcap,
-                                         int* err, cudaStream_t stream) {
+                                         float lambda, float diff_eps, float diff_factor, int out_dv, int* err,
+                                         cudaStream_t stream) {
   if (requests == 0) return 0;
+  if (MAPS == 2 && (gate != nullptr || sink != nullptr || out_dv < 1 || out_dv > D)) return (int)cudaErrorInvalidValue;
+  const MapDifference difference{lambda, diff_eps, diff_factor, out_dv};
   if (keep_first < 0 || (keep_first > 0 && (window <= 0 || proj != nullptr))) return (int)cudaErrorInvalidValue;
   if (run < 0 || softcap < 0.f || (run > 0 && keep_first > 0)) return (int)cudaErrorInvalidValue;
   if (requests < 0 || nkv < 1 || nq != nkv * GROUP || chunk_keys <= 0 || chunk_keys % DECODE_BN != 0 ||
@@ -929,17 +998,17 @@ extern "C" int omnia_attention_decode_tc(const void* q, const void* pages, const
     launch_pdl(attention_decode_kernel<1, DECODE_STAGES>, dim3(max_chunks, nkv, requests), 32, smem, stream,
         (const bf16*)q, (const bf16*)pages, block_table, cu_seqlens, seq_lens, seq_ids, part_o, part_ml,
         tickets, (const bf16*)gate, gate_stride, (bf16*)out, chunk_keys, max_chunks, max_pages,
-        num_pages, nq, nkv, page_size, window, scale, fused, keep_first, sink, run, softcap, err);
+        num_pages, nq, nkv, page_size, window, scale, fused, keep_first, sink, run, softcap, difference, err);
   else if (deep)
     launch_pdl(attention_decode_kernel<4, 2>, dim3(max_chunks, nkv, requests), 128, smem, stream,
         (const bf16*)q, (const bf16*)pages, block_table, cu_seqlens, seq_lens, seq_ids, part_o, part_ml,
         tickets, (const bf16*)gate, gate_stride, (bf16*)out, chunk_keys, max_chunks, max_pages,
-        num_pages, nq, nkv, page_size, window, scale, fused, keep_first, sink, run, softcap, err);
+        num_pages, nq, nkv, page_size, window, scale, fused, keep_first, sink, run, softcap, difference, err);
   else
     launch_pdl(attention_decode_kernel<4, 1>, dim3(max_chunks, nkv, requests), 128, smem, stream,
         (const bf16*)q, (const bf16*)pages, block_table, cu_seqlens, seq_lens, seq_ids, part_o, part_ml,
         tickets, (const bf16*)gate, gate_stride, (bf16*)out, chunk_keys, max_chunks, max_pages,
-        num_pages, nq, nkv, page_size, window, scale, fused, keep_first, sink, run, softcap, err);
+        num_pages, nq, nkv, page_size, window, scale, fused, keep_first, sink, run, softcap, difference, err);
   return OMNIA_LAUNCH_RESULT();
 }
 
@@ -1033,7 +1102,7 @@ extern "C" int omnia_attention_decode_tc_static(const void* q, const void* pages
   launch_pdl(attention_decode_kernel<1, DECODE_STAGES>, dim3(max_chunks, nkv, requests), 32, smem, stream,
       (const bf16*)q, (const bf16*)pages, block_table, cu_seqlens, seq_lens, seq_ids, part_o, part_ml,
       ticket_area, (const bf16*)gate, gate_stride, (bf16*)out, chunk_keys, max_chunks, max_pages,
-      num_pages, nq, nkv, page_size, window, scale, FusedQK{}, 0, nullptr, 0, 0.f, err);
+      num_pages, nq, nkv, page_size, window, scale, FusedQK{}, 0, nullptr, 0, 0.f, MapDifference{}, err);
   e = cudaGetLastError();
   if (e != cudaSuccess) snprintf(static_error, sizeof static_error, "launch: %s", cudaGetErrorString(e));
   return (int)e;

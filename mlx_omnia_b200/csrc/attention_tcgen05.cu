@@ -38,6 +38,10 @@
 // below its own) and `softcap` (a scaled score s becomes softcap * tanh(s / softcap), in float32, in the
 // softmax warps ahead of the maximum: two more special-function operations a score).
 //
+// Compiled with -DMAPS=2, two neighbouring query heads (two neighbouring rows, so two neighbouring lanes) are
+// the two maps of one head of differential attention, and what is written is their difference (see
+// MapDifference), [tokens, nq / 2, dv].
+//
 // Every wait on a barrier is bounded: when the bound is hit the block raises OMNIA_ERR_TIMEOUT
 // in the error word, every role leaves its loop, the producer waits (bounded) for loads in
 // flight, the block frees its tensor memory and returns.
@@ -47,6 +51,9 @@
 #ifndef GROUP
 #define GROUP 2
 #endif
+#ifndef MAPS
+#define MAPS 1
+#endif
 
 #include "attention_tcgen05.cuh"
 
@@ -55,6 +62,7 @@ namespace {
 constexpr int D = HEAD_DIM;
 static_assert(D == 64 || D == 128, "the tcgen05 attention kernel takes head sizes 64 and 128");
 static_assert(GROUP >= 1 && GROUP <= 16, "group size must be 1..16");
+static_assert(MAPS == 1 || (MAPS == 2 && GROUP % 2 == 0), "two maps to a head: an even number of query heads");
 constexpr int DH = D / 64;                 // 64-wide halves of a head
 constexpr int BM = 128, BN = 64;      // rows per block, keys per tile
 constexpr int TOKENS = BM / GROUP;         // tokens per block
@@ -70,6 +78,19 @@ constexpr uint32_t K_BYTES = DH * TILE_HALF, V_BYTES = DH * TILE_HALF;
 constexpr uint32_t GROUP_BYTES = 16 * 128;           // one TMA box: 16 keys x 64 dims
 constexpr uint32_t TMEM_COLS = 256;                  // two blocks share an SM's 512 columns
 constexpr uint32_t S_COL = 0, O_COL = 128;
+
+// Eight dims of a head's difference, from `c` on, of which those below `dv` exist.
+__device__ __forceinline__ void store_difference(bf16* dst, int c, const float* d, int dv, bool wide, bool mine) {
+  if (!mine || c >= dv) return;
+  if (wide) {
+    *reinterpret_cast<uint4*>(dst + c) =
+        make_uint4(pack_bf16(d[0], d[1]), pack_bf16(d[2], d[3]), pack_bf16(d[4], d[5]), pack_bf16(d[6], d[7]));
+  } else {
+#pragma unroll
+    for (int e = 0; e < 8; ++e)
+      if (c + e < dv) dst[c + e] = __float2bfloat16_rn(d[e]);
+  }
+}
 
 // The four softmax warps among themselves.
 __device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
@@ -93,7 +114,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                                  float* __restrict__ partial, int* __restrict__ tickets,
                                  int max_pages, int num_pages, int nq, int nkv, int page_size, int window,
                                  float scale, int keep_first, const float* __restrict__ sink, int run, float softcap,
-                                 int* err) {
+                                 const MapDifference difference, int* err) {
   if (work[WORK_INTS * blockIdx.x] < 0) return;  // a place of the list that this step does not use
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   // The swizzled tiles need a base on 1024 bytes; the dynamic area starts on one (nothing static
@@ -515,7 +536,46 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
         weights[parts * BM + row] = total > 0.f ? 1.f / total : 0.f;
       }
     }
-    if (ok && whole) {
+    if constexpr (MAPS == 2) ok = __all_sync(0xffffffffu, ok);  // a warp's lanes exchange values below
+    if (MAPS == 2 && ok && whole) {
+      // The accumulator is read twice: for the difference's sum of squares, then to be stored, every other 16
+      // bytes by either of the two lanes.
+      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const bool second = row & 1;
+      const uint32_t o_addr = tmem_base + lane_field + O_COL;
+      float ss = 0.f;
+#pragma unroll 1
+      for (int c0 = 0; c0 < D; c0 += 32) {
+        uint32_t acc[32];
+        tmem_load32(o_addr + c0, acc);
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          const float mine = __uint_as_float(acc[i]) * inv, other = __shfl_xor_sync(0xffffffffu, mine, 1);
+          const float d = second ? other - difference.lambda * mine : mine - difference.lambda * other;
+          ss += d * d;
+        }
+      }
+      const float f = rsqrtf(ss / (float)difference.dv + difference.eps) * difference.factor;
+      bf16* dst = out + (token * (nq / 2) + head / 2) * difference.dv;
+      const bool wide = (difference.dv & 7) == 0;
+#pragma unroll 1
+      for (int c0 = 0; c0 < D; c0 += 32) {
+        uint32_t acc[32];
+        tmem_load32(o_addr + c0, acc);
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+        for (int i = 0; i < 32; i += 8) {
+          float d[8];
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            const float mine = __uint_as_float(acc[i + e]) * inv, other = __shfl_xor_sync(0xffffffffu, mine, 1);
+            d[e] = (second ? other - difference.lambda * mine : mine - difference.lambda * other) * f;
+          }
+          store_difference(dst, c0 + i, d, difference.dv, wide, live && ((i >> 3) & 1) == (int)second);
+        }
+      }
+    } else if (ok && whole) {
       // 64 dims of the row's accumulator in one go (two loads side by side; eight dims a turn with the
       // next turn's columns on their way took longer: every turn waited for a load), then eight dims
       // at a time: normalise, gate, 16 bytes stored.
@@ -583,6 +643,47 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     }
     const float* all = partial + (size_t)slot0 * PART_FLOATS;
     const float* weights = reinterpret_cast<const float*>(k_s);
+    if constexpr (MAPS == 2) {
+      // A thread has every other eight dims of one row; the two threads of a row add their sums of squares
+      // through shared memory (Q's place, read for the last time long ago).
+      const int row = threadIdx.x % BM, half = threadIdx.x / BM;
+      const bool second = row & 1;
+      const float inv = weights[parts * BM + row];
+      float d[D / 2], ss = 0.f;
+#pragma unroll
+      for (int k = 0; k < D / 16; ++k) {
+        const int c = (half + 2 * k) * 8;
+        float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+        for (int q = 0; q < parts; ++q) {
+          const float4* src = reinterpret_cast<const float4*>(all + (size_t)q * PART_FLOATS) + (size_t)(c / 4) * BM + row;
+          const float4 a = __ldcg(src), b2 = __ldcg(src + BM);
+          const float w = weights[q * BM + row];
+          acc[0] += w * a.x, acc[1] += w * a.y, acc[2] += w * a.z, acc[3] += w * a.w;
+          acc[4] += w * b2.x, acc[5] += w * b2.y, acc[6] += w * b2.z, acc[7] += w * b2.w;
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const float mine = acc[e] * inv, other = __shfl_xor_sync(0xffffffffu, mine, 1);
+          const float v = second ? other - difference.lambda * mine : mine - difference.lambda * other;
+          d[k * 8 + e] = v;
+          ss += v * v;
+        }
+      }
+      float* squares = reinterpret_cast<float*>(q_s);
+      squares[threadIdx.x] = ss;
+      __syncthreads();
+      const float f = rsqrtf((squares[row] + squares[BM + row]) / (float)difference.dv + difference.eps) * difference.factor;
+      const size_t token = (size_t)(q_begin + tok0 + row / GROUP);
+      bf16* dst = out + (token * (nq / 2) + (kvh * GROUP + row % GROUP) / 2) * difference.dv;
+#pragma unroll
+      for (int k = 0; k < D / 16; ++k) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) d[k * 8 + e] *= f;
+        store_difference(dst, (half + 2 * k) * 8, d + k * 8, difference.dv, (difference.dv & 7) == 0,
+                         row < rows && (k & 1) == (int)second);
+      }
+      merged = false;
+    }
     if (merged) {
 #pragma unroll 2
       for (int item = threadIdx.x; item < BM * (D / 8); item += THREADS) {
@@ -660,8 +761,10 @@ extern "C" int omnia_attention_prefill_tcgen05(const void* q, int tokens, const 
                                                float* partial, int* tickets,
                                                int max_pages, int num_pages, int nq, int nkv, int page_size,
                                                int window, float scale, int keep_first, const float* sink, int run,
-                                               float softcap, int* err, cudaStream_t stream) {
+                                               float softcap, float lambda, float diff_eps, float diff_factor, int out_dv,
+                                               int* err, cudaStream_t stream) {
   if (blocks == 0) return 0;
+  if (MAPS == 2 && (gate != nullptr || sink != nullptr || out_dv < 1 || out_dv > D)) return (int)cudaErrorInvalidValue;
   if (nq != nkv * GROUP || page_size % 16 != 0 || ((uintptr_t)q & 15) || ((uintptr_t)pages & 15) || keep_first < 0 ||
       (keep_first > 0 && window <= 0) || run < 0 || softcap < 0.f || (run > 0 && keep_first > 0))
     return (int)cudaErrorInvalidValue;
@@ -681,6 +784,6 @@ extern "C" int omnia_attention_prefill_tcgen05(const void* q, int tokens, const 
   launch_pdl(attention_prefill_tcgen05_kernel, blocks, THREADS, smem, stream,
              map_q, map_kv, map_gate, gate_tma, block_table, cu_seqlens, seq_lens, work, (const bf16*)gate, gate_stride, (bf16*)out,
              partial, tickets, max_pages, num_pages, nq, nkv, page_size, window, scale, keep_first, sink, run, softcap,
-             err);
+             MapDifference{lambda, diff_eps, diff_factor, out_dv}, err);
   return OMNIA_LAUNCH_RESULT();
 }

@@ -52,6 +52,14 @@ __device__ __forceinline__ float xielu(float z, float rise, float fall) {
   return z > 0.f ? fmaf(rise * z, z, 0.5f * z) : fmaf(fall, expm1f(z) - z, 0.5f * z);
 }
 
+// Attention whose heads are the difference of two softmax maps (query heads 2 h and 2 h + 1): a head's output
+// is a_1 - lambda a_2 over its `dv` values, divided by its own root mean square (eps inside the root), times
+// `factor`. The kernels that finish rows take this in their epilogue, in float32.
+struct MapDifference {
+  float lambda, eps, factor;
+  int dv;
+};
+
 // Sum over the block; every thread gets the result. `scratch` holds 33 floats.
 // The order of the additions depends only on blockDim, never on the data.
 __device__ __forceinline__ float block_sum(float v, float* scratch) {

@@ -1,7 +1,5 @@
-// Attention whose projections pass a short causal convolution over time, and whose heads may be the
-// difference of several softmax maps.
-//
-// What a token's projected row becomes before the attention (conv_heads_prepare): per channel of q, k
+// What a token's projected row becomes before an attention whose projections pass a short causal
+// convolution over time and whose heads may have several softmax maps. Per channel of q, k
 // and v a bias, then y_t = sum_j taps[K - 1 - j] in_(t - j) over the request's inputs (zeros ahead of its
 // start; inputs before this step come from the request's state slot), then on q and k the rotation of
 // the first `rot` dims of every map of every head. A head has `maps` maps of `dk` dims each. A head of
@@ -10,9 +8,6 @@
 // product with a key row is then its own map's score, every map of a head shares one key row and one
 // value row, and the attention kernels see ordinary grouped-query attention: heads * maps query heads
 // of d over kv_heads key/value heads.
-//
-// What becomes of the maps' outputs (map_difference): per head o = a_1 - lambda a_2, divided by its own
-// root mean square, times a constant.
 //
 // Float32 from the projected row on; rounded once where a row is stored.
 #include "common.cuh"
@@ -203,43 +198,6 @@ __global__ void conv_heads_advance_kernel(const ConvArgs p) {
   }
 }
 
-// A warp per (token, head): maps [tokens, heads * 2, d], the first dv of a row being the map's output.
-template <typename T, int V>
-__global__ void __launch_bounds__(128) map_difference_kernel(const T* __restrict__ maps, int heads, int d, int dv, float lambda,
-                                                             float eps, float factor, T* __restrict__ out, int rows) {
-  pdl_wait();
-  pdl_launch_dependents();
-  constexpr int MOST = 512 / 32 / V > 0 ? 512 / 32 / V : 1;  // dv <= 512
-  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (row >= rows) return;
-  struct alignas(sizeof(T) * V) Pack {
-    T v[V];
-  };
-  const T* first = maps + (size_t)row * 2 * d;
-  float o[MOST][V], ss = 0.f;
-#pragma unroll
-  for (int k = 0; k < MOST; ++k) {
-    const int i = (k * 32 + lane) * V;
-    if (i >= dv) break;
-    const Pack a = *reinterpret_cast<const Pack*>(first + i), b = *reinterpret_cast<const Pack*>(first + d + i);
-#pragma unroll
-    for (int e = 0; e < V; ++e) {
-      o[k][e] = to_f32(a.v[e]) - lambda * to_f32(b.v[e]);
-      ss += o[k][e] * o[k][e];
-    }
-  }
-  const float r = rsqrtf(warp_sum(ss) / (float)dv + eps) * factor;
-#pragma unroll
-  for (int k = 0; k < MOST; ++k) {
-    const int i = (k * 32 + lane) * V;
-    if (i >= dv) break;
-    Pack y;
-#pragma unroll
-    for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(o[k][e] * r);
-    *reinterpret_cast<Pack*>(out + (size_t)row * dv + i) = y;
-  }
-}
-
 }  // namespace
 
 extern "C" int omnia_conv_heads_prepare(const void* proj, int stride, int col0, const float* bias, const float* taps, int K,
@@ -281,22 +239,5 @@ extern "C" int omnia_conv_heads_prepare(const void* proj, int stride, int col0, 
     OMNIA_DISPATCH_DTYPE(dtype, (launch_pdl(conv_heads_advance_kernel<T>, dim3((channels + 127) / 128, num_seqs), dim3(128), 0,
                                             stream, p)));
   }
-  return OMNIA_LAUNCH_RESULT();
-}
-
-extern "C" int omnia_map_difference(const void* maps, int heads, int d, int dv, float lambda, float eps, float factor, void* out,
-                                    int tokens, int dtype, cudaStream_t stream) {
-  if (tokens == 0) return 0;
-  if (dv < 1 || dv > 512 || dv > d || heads < 1) return (int)cudaErrorInvalidValue;
-  const int rows = tokens * heads;
-  const bool wide = dv % 4 == 0 && d % 4 == 0 && (((uintptr_t)maps | (uintptr_t)out) & 15) == 0;
-  OMNIA_DISPATCH_DTYPE(dtype, {
-    if (wide)
-      launch_pdl(map_difference_kernel<T, 4>, dim3((rows + 3) / 4), dim3(128), 0, stream, (const T*)maps, heads, d, dv, lambda,
-                 eps, factor, (T*)out, rows);
-    else
-      launch_pdl(map_difference_kernel<T, 1>, dim3((rows + 3) / 4), dim3(128), 0, stream, (const T*)maps, heads, d, dv, lambda,
-                 eps, factor, (T*)out, rows);
-  });
   return OMNIA_LAUNCH_RESULT();
 }

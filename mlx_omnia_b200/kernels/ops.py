@@ -594,12 +594,24 @@ def decode_fusable(proj: torch.Tensor, nq: int, nkv: int, d: int, inv_freq: torc
             and tiled_attention_supported(proj.dtype, nq, nkv, d))
 
 
+@dataclass(frozen=True)
+class MapDifference:
+    """Differential attention's end of a head: of its two softmax maps' outputs (query heads 2 h and 2 h + 1) over
+    the first `dv` of the cache's value width, a_1 - lam a_2, divided by its root mean square (`eps` inside the
+    root), times `factor`; float32 up to the one rounding."""
+
+    lam: float
+    eps: float
+    factor: float
+    dv: int
+
+
 def paged_attention(q: torch.Tensor | None, kv: KVView, step: StepContext, scale: float,
                     gate: torch.Tensor | None = None, gate_col: int = 0,
                     projection: Projection | None = None, wide: bool | None = None,
                     sink: torch.Tensor | None = None, window: int | None = -1,
                     keep_first: int | None = None, chunk: int | None = None,
-                    softcap: float | None = None) -> torch.Tensor:
+                    softcap: float | None = None, difference: MapDifference | None = None) -> torch.Tensor:
     """Causal (windowed) attention of this step's queries over the paged cache, the
     output multiplied by sigmoid(gate) when `gate` (the projected rows; the gate's
     columns start at `gate_col`) is given.  -> [tokens, nq * dv]
@@ -616,6 +628,9 @@ def paged_attention(q: torch.Tensor | None, kv: KVView, step: StepContext, scale
     position 0, wherever a prompt was cut); `softcap` c: a scaled score s becomes c tanh(s / c) ahead of
     the softmax. Both are taken by the generic kernel, by the mma.sync kernels and by the tcgen05 prefill
     kernel that runs two blocks to an SM.
+
+    `difference`: two neighbouring query heads are the two maps of one head, and [tokens, nq / 2 * difference.dv] is
+    what their difference gives; no gate and no sink then. Taken by the same kernels as runs and capped scores.
 
     With `projection` (only where `decode_fusable` holds) q is not given: the kernel makes the
     queries and the new keys and values from the projected rows, and writes the latter to the cache.
@@ -635,7 +650,11 @@ def paged_attention(q: torch.Tensor | None, kv: KVView, step: StepContext, scale
     keep = kv.keep_first if keep_first is None else keep_first
     if not kv.window:
         keep = 0
-    out = torch.empty(tokens, nq * dv, dtype=q.dtype, device=q.device)
+    if difference is not None and (nq % 2 or gate is not None or sink is not None or projection is not None
+                                   or not 1 <= difference.dv <= dv):
+        raise KernelError("a difference of maps takes pairs of query heads, no gate, no sink and no projected rows")
+    last = (0.0, 0.0, 0.0, 0) if difference is None else (difference.lam, difference.eps, difference.factor, difference.dv)
+    out = torch.empty(tokens, nq * dv if difference is None else nq // 2 * difference.dv, dtype=q.dtype, device=q.device)
     gate_ptr = None if gate is None else gate.data_ptr() + gate_col * gate.element_size()
     gate_stride = 0 if gate is None else gate.shape[1]
     err = _ptr(error_word(q.device))
@@ -649,13 +668,13 @@ def paged_attention(q: torch.Tensor | None, kv: KVView, step: StepContext, scale
         fn = _function("attention_generic", "omnia_paged_attention_generic",
                        [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                        c_int, c_float, c_int, c_float, c_int, c_void_p, c_void_p])
+                        c_int, c_float, c_int, c_float, c_int, c_float, c_float, c_float, c_int, c_int, c_void_p, c_void_p])
         _check(fn(_ptr(q), k_ptr, v_ptr, page_stride, _ptr(kv.block_table), _ptr(step.cu_seqlens),
                   _ptr(step.positions), gate_ptr, gate_stride, _ptr(out), _ptr(sink), tokens, step.num_seqs, max_pages,
                   num_pages, nq, nkv, d, dv, kv.page_size, kv.window or 0, keep, scale, run, softcap,
-                  _code(q.dtype), err, _stream()), "paged_attention")
+                  1 if difference is None else 2, *last, _code(q.dtype), err, _stream()), "paged_attention")
         return out
-    defines = {"HEAD_DIM": d, "GROUP": nq // nkv}
+    defines = {"HEAD_DIM": d, "GROUP": nq // nkv} | ({} if difference is None else {"MAPS": 2})
     # Requests that bring a single token take the split-key decode kernel, in a decode-only step
     # (all of them, no index list: the shape a captured graph replays) and in a mixed step alike.
     single, longest = (None, step.max_seq_len) if step.decode_only else _single_token_requests(step, q.device)
@@ -672,7 +691,7 @@ def paged_attention(q: torch.Tensor | None, kv: KVView, step: StepContext, scale
                        [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                         c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                         c_float, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p,
-                        c_int, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p], defines)
+                        c_int, c_int, c_void_p, c_int, c_float, c_float, c_float, c_float, c_int, c_void_p, c_void_p], defines)
         p = projection
         fused = (None, 0, 0, 0, 0, -1.0, None, None) if p is None else (
             _ptr(p.rows), p.rows.shape[1], p.q_col, p.k_col, p.v_col, -1.0 if p.eps is None else p.eps,
@@ -680,7 +699,7 @@ def paged_attention(q: torch.Tensor | None, kv: KVView, step: StepContext, scale
         _check(fn(None if p is not None else _ptr(q), _ptr(kv.pages), _ptr(kv.block_table), _ptr(step.cu_seqlens),
                   _ptr(step.seq_lens), _ptr(single), count, _ptr(part_o), _ptr(part_ml), _ptr(tickets), chunk,
                   max_chunks, gate_ptr, gate_stride, _ptr(out), max_pages, num_pages, nq, nkv, kv.page_size,
-                  kv.window or 0, scale, warps, *fused, 1, keep, _ptr(sink), run, softcap, err, _stream()),
+                  kv.window or 0, scale, warps, *fused, 1, keep, _ptr(sink), run, softcap, *last, err, _stream()),
                "attention_decode")
         if step.decode_only or all(n == 1 for n in step.q_lens):
             return out
@@ -688,12 +707,12 @@ def paged_attention(q: torch.Tensor | None, kv: KVView, step: StepContext, scale
         per_block = 128 // (nq // nkv)
         sms = sm_count(q.device)
         plain = sink is None and not keep  # a sink or kept first positions: the two-to-an-SM kernel, every block whole
-        narrow = bool(run or softcap)  # runs and capped scores: the two-to-an-SM kernel, blocks cut as ever
+        narrow = bool(run or softcap or difference)  # runs, capped scores, differences of maps: the two-to-an-SM kernel, blocks cut as ever
         if wide is None:
             wide = plain and not narrow and wide_prefill_pays(step.q_lens, step.seq_lens_host, per_block, nkv,
                                                               kv.window or 0, sms)
         elif wide and (not plain or narrow):
-            raise KernelError("the kernel that gives a block its SM takes no sink, kept first positions, runs or cap")
+            raise KernelError("the kernel that gives a block its SM takes no sink, kept first positions, runs, cap or difference")
         if wide:
             # Every block whole (no places to share tiles over), an SM to a block.
             work = _prefill_work_flat(step, per_block, 64, nkv, kv.window or 0, q.device, 0)
@@ -716,21 +735,21 @@ def paged_attention(q: torch.Tensor | None, kv: KVView, step: StepContext, scale
         fn = _function("attention_tcgen05", "omnia_attention_prefill_tcgen05",
                        [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
                         c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
-                        c_int, c_float, c_void_p, c_void_p], defines)
+                        c_int, c_float, c_float, c_float, c_float, c_int, c_void_p, c_void_p], defines)
         _check(fn(_ptr(q), tokens, _ptr(kv.pages), _ptr(kv.block_table), _ptr(step.cu_seqlens), _ptr(step.seq_lens),
                   _ptr(work), work.shape[0], gate_ptr, gate_stride, _ptr(out), _ptr(partial), _ptr(tickets), max_pages,
-                  num_pages, nq, nkv, kv.page_size, kv.window or 0, scale, keep, _ptr(sink), run, softcap, err, _stream()),
+                  num_pages, nq, nkv, kv.page_size, kv.window or 0, scale, keep, _ptr(sink), run, softcap, *last, err, _stream()),
                "attention_prefill_tcgen05")
         return out
     tokens_per_block = 64 // (nq // nkv)
     work = _prefill_work(step, tokens_per_block, q.device)
     fn = _function("attention_tc", "omnia_attention_prefill_tc",
                    [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p,
-                    c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_float, c_void_p,
-                    c_void_p], defines)
+                    c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_float, c_float, c_float,
+                    c_float, c_int, c_void_p, c_void_p], defines)
     _check(fn(_ptr(q), _ptr(kv.pages), _ptr(kv.block_table), _ptr(step.cu_seqlens), _ptr(step.seq_lens), _ptr(work),
               work.shape[0], gate_ptr, gate_stride, _ptr(out), max_pages, num_pages, nq, nkv, kv.page_size,
-              kv.window or 0, scale, keep, _ptr(sink), run, softcap, err, _stream()), "attention_prefill")
+              kv.window or 0, scale, keep, _ptr(sink), run, softcap, *last, err, _stream()), "attention_prefill")
     return out
 
 
@@ -1882,7 +1901,7 @@ def mingru(proj: torch.Tensor, z_col: int, u_col: int, g_col: int, z_bias: torch
 
 
 # ------------------------------------------------------------------------------------
-# Convolved projections and heads of several softmax maps (csrc/conv_heads.cu)
+# Convolved projections of heads with several softmax maps (csrc/conv_heads.cu)
 
 CONV_HEADS_MAX_TAPS = 16
 
@@ -1914,14 +1933,3 @@ def conv_heads_prepare(proj: torch.Tensor, col0: int, bias: torch.Tensor | None,
               tokens, int(step.decode_only), _code(proj.dtype), _ptr(error_word(proj.device)), _stream()),
            "conv_heads_prepare")
     return q
-
-
-def map_difference(maps: torch.Tensor, heads: int, d: int, dv: int, lam: float, eps: float, factor: float) -> torch.Tensor:
-    """maps [tokens, heads * 2 * d], two rows of `d` a head of which the first `dv` count: o = first - lam * second,
-    divided by its root mean square (eps inside the root), times `factor`. -> [tokens, heads * dv]"""
-    tokens = maps.shape[0]
-    out = torch.empty(tokens, heads * dv, dtype=maps.dtype, device=maps.device)
-    fn = _function("conv_heads", "omnia_map_difference",
-                   [c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_int, c_int, c_void_p])
-    _check(fn(_ptr(maps), heads, d, dv, lam, eps, factor, _ptr(out), tokens, _code(maps.dtype), _stream()), "map_difference")
-    return out

@@ -453,7 +453,8 @@ class DifferentialAttention(Mixer):
         self.taps = torch.cat([tensors[name + ".conv"] for name in names]).t().contiguous()
         self.o = tensors["o"].contiguous()
         a, b, c, d = (tensors[name].double() for name in ("lq1", "lk1", "lq2", "lk2"))
-        self.lam = float(torch.exp((a * b).sum()) - torch.exp((c * d).sum()) + self.diff)
+        lam = float(torch.exp((a * b).sum()) - torch.exp((c * d).sum()) + self.diff)
+        self.difference = ops.MapDifference(lam, self.norm_eps, 1.0 - self.diff, self.vdim)
 
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
         if ctx.kv is None:
@@ -464,6 +465,5 @@ class DifferentialAttention(Mixer):
                                    self.heads, self.kv_heads if self.own_kv else 0, self.MAPS, self.dim, self.vdim, self.row,
                                    self.position.table(), getattr(self.position, "pairing", "half") == "half",
                                    getattr(self.position, "amount", 1.0), ctx.kv)
-        maps = ops.paged_attention(q, ctx.kv, ctx.step, self.scale, window=self.window)
-        return ops.linear(ops.map_difference(maps, self.heads, self.row, self.vdim, self.lam, self.norm_eps, 1.0 - self.diff),
+        return ops.linear(ops.paged_attention(q, ctx.kv, ctx.step, self.scale, window=self.window, difference=self.difference),
                           self.o)
