@@ -89,7 +89,8 @@ extern "C" int omnia_latent_prepare(void* proj, int stride, int q_col, int heads
   if (tokens == 0) return 0;
   if (cq_out != nullptr && (q_rank < 1 || heads != 0)) return (int)cudaErrorInvalidValue;
   if (rot_dims % 2 != 0 || rot_dims > rot || (heads > 0 && rot > q_dim) || rank < 1) return (int)cudaErrorInvalidValue;
-  OMNIA_DISPATCH_DTYPE(dtype, (launch_pdl(latent_prepare_kernel<T>, tokens, 128, 0, stream, (T*)proj, stride, q_col,
+  const int threads = rank + q_rank > 512 ? 256 : 128;
+  OMNIA_DISPATCH_DTYPE(dtype, (launch_pdl(latent_prepare_kernel<T>, tokens, threads, 0, stream, (T*)proj, stride, q_col,
                                           heads, q_dim, down_col, rank, rot, w, eps, inv_freq, rot_dims, positions,
                                           slot_mapping, (T*)cache, total_slots, half_pairs, amount, cq_col,
                                           q_rank, cq_w, (T*)cq_out, err)));

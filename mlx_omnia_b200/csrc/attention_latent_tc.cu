@@ -11,7 +11,8 @@
 // cp.async double buffer. Warp (row group, column quarter): scores of its 16 rows against 8 of the
 // tile's keys; the row maxima of the four quarters meet in shared memory, the weights P go there as
 // bfloat16; then each warp adds P V for its quarter of the latent columns. The key range may be cut
-// into `splits` chunks (aligned to absolute positions) that separate blocks walk; each then leaves
+// into `splits` chunks (aligned to absolute positions; with a window counted from the chunk that holds the
+// first key the request's first row can see) that separate blocks walk; each then leaves
 // its unnormalised accumulator, maximum and sum in a workspace, and a second kernel merges a row's
 // chunks in ascending order. The sink and the gate are applied where the row is finished. Keys
 // outside a block's range are zero-filled in shared memory and never read from the cache.
@@ -128,8 +129,9 @@ __global__ void __launch_bounds__(THREADS) latent_attention_tc_kernel(const Args
   int key_lo = a.window > 0 ? max(0, first_pos - a.window + 1) : 0;
   int key_hi = last_pos;                            // inclusive; -1 for a padding request: no keys
   if (a.splits > 1) {
-    key_lo = max(key_lo, split * a.chunk);
-    key_hi = min(key_hi, (split + 1) * a.chunk - 1);
+    const int base = a.window > 0 ? max(0, pos0 - a.window + 1) / a.chunk * a.chunk : 0;
+    key_lo = max(key_lo, base + split * a.chunk);
+    key_hi = min(key_hi, base + (split + 1) * a.chunk - 1);
   }
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int rg = warp / CW, cw = warp % CW;

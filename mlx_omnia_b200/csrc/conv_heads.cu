@@ -173,6 +173,131 @@ __global__ void __launch_bounds__(256) conv_heads_prepare_kernel(const ConvArgs 
   }
 }
 
+// Many tokens: a thread owns eight neighbouring elements of the outputs and walks a run of tokens with the
+// last K - 1 inputs in registers, so an input is read once; what the elements are and where they go is worked
+// out once a run. grid (runs of RUN tokens, ceil(outputs / 8 / threads)); every width in eights.
+constexpr int RUN = 16;
+template <typename T>
+struct alignas(16) Octet {
+  T v[8];
+};
+
+template <typename T, int K>
+__global__ void __launch_bounds__(256) conv_heads_runs_kernel(const ConvArgs p) {
+  pdl_wait();
+  pdl_launch_dependents();
+  extern __shared__ float2 turn_s[];  // [RUN][half] (cos, sin)
+  __shared__ long long slot_s[RUN];
+  const int t0 = blockIdx.x * RUN, t1 = min(p.tokens, t0 + RUN);
+  const int half = p.inv_freq ? p.rot / 2 : 0;
+  for (int i = threadIdx.x; i < (t1 - t0) * half; i += blockDim.x) {
+    float s, c;
+    sincosf((float)p.positions[t0 + i / half] * p.inv_freq[i % half], &s, &c);
+    turn_s[i] = make_float2(c * p.amount, s * p.amount);
+  }
+  if (threadIdx.x < t1 - t0) {
+    long long slot = p.kv_heads > 0 ? p.slot_mapping[t0 + threadIdx.x] : -1;
+    if (slot >= p.num_slots) {
+      if (blockIdx.y == 0) atomicOr(p.err, OMNIA_ERR_SLOT);
+      slot = -1;
+    }
+    slot_s[threadIdx.x] = slot;
+  }
+  __syncthreads();
+  const int q_outs = p.heads * p.maps * p.d, k_outs = p.kv_heads * p.d, outs = q_outs + 2 * k_outs;
+  const int k_chan = p.heads * p.maps * p.dk, v_chan = k_chan + p.kv_heads * p.maps * p.dk;
+  const int o = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+  if (o >= outs) return;
+  int c = -1, dim = -1, head = 0, e = 0;
+  const bool query = o < q_outs, value = o >= q_outs + k_outs;
+  if (query) {
+    const int row = o / p.d, i = o - row * p.d - (row % p.maps) * p.dk;
+    if (i >= 0 && i < p.dk) c = row * p.dk + i, dim = i;
+  } else {
+    const int x = o - q_outs - (value ? k_outs : 0);
+    head = x / p.d, e = x - head * p.d;
+    if (value) {
+      if (e < p.dv) c = v_chan + head * p.dv + e;
+    } else if (e < p.maps * p.dk) {
+      c = k_chan + head * p.maps * p.dk + e, dim = e % p.dk;
+    }
+  }
+  T* pages = (T*)(value ? p.v_pages : p.k_pages);
+  auto store = [&](int t, const Octet<T>& y) {
+    T* dst;
+    if (query) {
+      dst = (T*)p.q_out + (size_t)t * q_outs + o;
+    } else {
+      const long long slot = slot_s[t - t0];
+      if (slot < 0) return;
+      dst = pages + (slot / p.page_size) * p.page_stride + ((long long)head * p.page_size + slot % p.page_size) * p.d + e;
+    }
+    *reinterpret_cast<Octet<T>*>(dst) = y;
+  };
+  if (c < 0) {
+    Octet<T> zero;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) zero.v[i] = from_f32<T>(0.f);
+    for (int t = t0; t < t1; ++t) store(t, zero);
+    return;
+  }
+  float w[K][8], bias[8], before[K > 1 ? K - 1 : 1][8];  // before[j]: the input j + 1 tokens back
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    bias[i] = p.bias ? p.bias[c + i] : 0.f;
+#pragma unroll
+    for (int j = 0; j < K; ++j) w[j][i] = p.taps[(size_t)(K - 1 - j) * p.channels + c + i];
+  }
+  const T* col = (const T*)p.proj + p.col0 + c;
+  int lo = 0, hi = p.num_seqs;
+  while (hi - lo > 1) {
+    const int mid = (lo + hi) >> 1;
+    if (p.cu_seqlens[mid] <= t0) lo = mid;
+    else hi = mid;
+  }
+  int end = t0;  // the first token of the run finds its request's inputs like the first of any request
+  for (int t = t0; t < t1; ++t) {
+    if (t >= end) {
+      while (p.cu_seqlens[lo + 1] <= t) ++lo;
+      end = p.cu_seqlens[lo + 1];
+      const int begin = p.cu_seqlens[lo];
+      const float* state = p.state + (size_t)p.state_slots[lo] * (K - 1) * p.channels + c;
+#pragma unroll
+      for (int j = 0; j < K - 1; ++j) {
+        const int src = t - 1 - j;
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          before[j][i] = src >= begin ? to_f32(col[(size_t)src * p.stride + i]) + bias[i]
+                                      : state[(size_t)(K - 1 - (begin - src)) * p.channels + i];
+      }
+    }
+    const Octet<T> raw = *reinterpret_cast<const Octet<T>*>(col + (size_t)t * p.stride);
+    float y[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float x = to_f32(raw.v[i]) + bias[i];
+      y[i] = w[0][i] * x;
+#pragma unroll
+      for (int j = 1; j < K; ++j) y[i] = fmaf(w[j][i], before[j - 1][i], y[i]);
+#pragma unroll
+      for (int j = K - 2; j > 0; --j) before[j][i] = before[j - 1][i];
+      if (K > 1) before[0][i] = x;
+    }
+    Octet<T> out;
+#pragma unroll
+    for (int i = 0; i < 8; i += 2) {
+      if (dim >= 0 && dim + i < 2 * half) {
+        const float2 turn = turn_s[(t - t0) * half + ((dim + i) >> 1)];
+        const float u = y[i] * turn.x - y[i + 1] * turn.y;
+        y[i + 1] = y[i + 1] * turn.x + y[i] * turn.y;
+        y[i] = u;
+      }
+      out.v[i] = from_f32<T>(y[i]), out.v[i + 1] = from_f32<T>(y[i + 1]);
+    }
+    store(t, out);
+  }
+}
+
 // A request's last K - 1 inputs, oldest first, after this step. grid (ceil(channels / 128), requests)
 template <typename T>
 __global__ void conv_heads_advance_kernel(const ConvArgs p) {
@@ -229,8 +354,17 @@ extern "C" int omnia_conv_heads_prepare(const void* proj, int stride, int col0, 
   const int enough = (4 * omnia_sm_count() + tokens - 1) / tokens;  // many tokens: fewer, longer blocks
   if (parts > enough) parts = enough;
   const dim3 grid(tokens, parts);
+  const bool runs = pairs && !single && tokens >= 2 * RUN && K <= 4 && dk % 8 == 0 && dv % 8 == 0 && d % 8 == 0 && stride % 8 == 0 &&
+                    col0 % 8 == 0 && page_stride % 8 == 0 &&
+                    (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages) & 15) == 0;
+  const size_t turns = inv_freq ? (size_t)RUN * (rot / 2) * sizeof(float2) : 0;
+  const dim3 run_grid((tokens + RUN - 1) / RUN, (outs / 8 + 255) / 256);
   OMNIA_DISPATCH_DTYPE(dtype, {
-    if (pairs) launch_pdl(conv_heads_prepare_kernel<T, true>, grid, dim3(256), 0, stream, p);
+    if (runs && K == 1) launch_pdl(conv_heads_runs_kernel<T, 1>, run_grid, dim3(256), turns, stream, p);
+    else if (runs && K == 2) launch_pdl(conv_heads_runs_kernel<T, 2>, run_grid, dim3(256), turns, stream, p);
+    else if (runs && K == 3) launch_pdl(conv_heads_runs_kernel<T, 3>, run_grid, dim3(256), turns, stream, p);
+    else if (runs && K == 4) launch_pdl(conv_heads_runs_kernel<T, 4>, run_grid, dim3(256), turns, stream, p);
+    else if (pairs) launch_pdl(conv_heads_prepare_kernel<T, true>, grid, dim3(256), 0, stream, p);
     else launch_pdl(conv_heads_prepare_kernel<T, false>, grid, dim3(256), 0, stream, p);
   });
   if (!p.advance && K > 1) {

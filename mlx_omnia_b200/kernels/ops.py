@@ -867,6 +867,31 @@ def _gemm_tcgen05(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epil
     return out
 
 
+_side_streams: dict[int, "torch.cuda.Stream"] = {}
+
+
+def side_by_side(first, second, device: torch.device):
+    """first() and second(), which must not depend on one another: while a graph is being captured the second
+    is recorded on a stream of its own beside the first, so a replay may run the two at the same time;
+    otherwise one after the other (launched from Python they would not overlap). -> both results
+
+    Memory: what second() allocates is handed out again only to the side stream, whose next work waits for
+    everything that was on the current stream by then, the readers of this call's result among it."""
+    if not torch.cuda.is_current_stream_capturing():
+        return first(), second()
+    index = device.index if device.index is not None else torch.cuda.current_device()
+    side = _side_streams.get(index)
+    if side is None:
+        side = _side_streams[index] = torch.cuda.Stream(device=device)
+    current = torch.cuda.current_stream(device)
+    side.wait_stream(current)
+    with torch.cuda.stream(side):
+        b = second()
+    a = first()
+    current.wait_stream(side)
+    return a, b
+
+
 def begin_pass(step: StepContext) -> None:
     """A pass over the model's layers begins: what kernels keep for the length of one pass (tables
     made from the step's positions, shared by the layers) is made afresh. A captured step is the
@@ -1559,11 +1584,20 @@ def latent_tc_supported(q_lat: torch.Tensor, q_rot: torch.Tensor, out: torch.Ten
                     for t in (q_lat, q_rot, out)))
 
 
-def latent_split_plan(q_lens, heads: int, longest: int, rows_per_block: int, sms: int) -> tuple[int, int]:
+def latent_split_plan(q_lens, heads: int, longest: int, rows_per_block: int, sms: int,
+                      window: int | None = None) -> tuple[int, int]:
     """(splits, keys per split) of the tensor-core latent attention kernel: one split while the step's
     row blocks fill the GPU; otherwise the keys are cut (in multiples of 32, at least 128 a split) so
-    that about two blocks run on every SM."""
+    that about two blocks run on every SM. With a window only the keys that a request's rows can see are
+    cut (at least 32 a split), into one more split than they fill: chunks are aligned to absolute positions."""
     blocks = sum(-(-q * heads // rows_per_block) for q in q_lens)
+    seen = window + max(q_lens) - 1 if window else longest
+    if window and seen < longest:
+        if blocks >= sms or seen <= 64:
+            return 1, 0
+        splits = max(1, min(-(-4 * sms // blocks), -(-seen // 32), 255))
+        chunk = -(-(-(-seen // splits)) // 32) * 32
+        return -(-seen // chunk) + 1, chunk
     if blocks >= sms or longest <= 128:
         return 1, 0
     splits = min(-(-2 * sms // blocks), -(-longest // 128), 256)
@@ -1590,7 +1624,7 @@ def latent_attention(q_lat: torch.Tensor, q_rot: torch.Tensor, kv: KVView, step:
         defines = {"LATENT_RANK": rank, "LATENT_ROT": rot, "LATENT_ROW_GROUPS": groups}
         # The bound on a request's length that is fixed for a captured step: its block table's width.
         longest = kv.block_table.shape[1] * kv.page_size
-        splits, chunk = latent_split_plan(step.q_lens, heads, longest, 16 * groups, sm_count(q_lat.device))
+        splits, chunk = latent_split_plan(step.q_lens, heads, longest, 16 * groups, sm_count(q_lat.device), kv.window)
         part_o = part_ml = None
         if splits > 1:
             part_o, part_ml = _step_buffers(step, q_lat.device, {
@@ -1872,12 +1906,14 @@ MINGRU_MAX_CLUSTER = 8
 
 
 def mingru_segments(longest: int, channels: int, requests: int, sms: int) -> tuple[int, int]:
-    """(warps a block, blocks a cluster) that the recurrence kernel cuts a request's portion over: segments of
-    about 16 tokens, more blocks to a cluster only while the SMs are not filled."""
+    """(warps a block, blocks a cluster) that the recurrence kernel cuts a request's portion over: a segment of 4
+    tokens at least, more blocks to a cluster only while the SMs are not filled. Measured, one request, us with
+    16 warps and 1 / 2 / 4 / 8 blocks: 2,048 tokens of 1,024 channels 95 / 50 / 27 / 26, of 2,048 96 / 50 / 37 /
+    32, of 4,096 96 / 51 / 58 / 57; 256 tokens of 2,048 14 / 9.3 / 8.3 / 7.9."""
     warps = max(1, min(MINGRU_MAX_WARPS, longest // 16))
     cluster = 1
-    while (cluster < MINGRU_MAX_CLUSTER and longest >= 32 * warps * cluster
-           and -(-channels // 32) * requests * cluster < 4 * sms):
+    while (cluster < MINGRU_MAX_CLUSTER and longest >= 8 * warps * cluster
+           and -(-channels // 64) * requests * cluster < 2 * sms):
         cluster *= 2
     return warps, cluster
 

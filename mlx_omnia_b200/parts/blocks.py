@@ -348,6 +348,10 @@ class BranchNormBlock(Block):
         return x, self._step(x, m, self.norms["norm2"], exit_norm, True)
 
 
+SIDE_BY_SIDE_ROWS = 256
+"""Up to this many rows a parallel block's two branches are captured side by side."""
+
+
 @register_block("parallel")
 class ParallelBlock(Block):
     """One norm whose output both branches read: r = x + mixer(norm(x)) + feed_forward(norm(x)). The
@@ -361,7 +365,8 @@ class ParallelBlock(Block):
     depth:        with `averaged`, how many layers the model runs (places for their results)
 
     The residual sum, the experts' weighted sum (where the feed-forward gives its rows), the average and
-    the next reader's norm are one pass over a row."""
+    the next reader's norm are one pass over a row. In captured steps of few rows the two branches run beside
+    one another."""
 
     def __init__(self, mixer: PartSpec, feed_forward: PartSpec | None, norm: PartSpec, averaged: int | None = None,
                  depth: int = 0, mixer_name: str = "mix", feed_forward_name: str = "mlp") -> None:
@@ -394,11 +399,17 @@ class ParallelBlock(Block):
 
     def forward(self, x, h, ctx, exit_norm):
         h = ops.settle(h)
-        branch = self.mixer.forward(h, ctx)
-        second = None
-        if self.feed_forward is not None:
-            rows = getattr(self.feed_forward, "gives_rows", False)
-            second = self.feed_forward.forward_rows(h, ctx) if rows else self.feed_forward.forward(h, ctx)
+        mix = lambda: self.mixer.forward(h, ctx)  # noqa: E731
+        if self.feed_forward is None:
+            branch, second = mix(), None
+        else:
+            ff = self.feed_forward
+            rows = getattr(ff, "gives_rows", False)
+            feed = lambda: ff.forward_rows(h, ctx) if rows else ff.forward(h, ctx)  # noqa: E731
+            if h.shape[0] <= SIDE_BY_SIDE_ROWS:
+                branch, second = ops.side_by_side(mix, feed, h.device)
+            else:
+                branch, second = mix(), feed()
         history = None
         if self.coef is not None:
             history = ops.depth_history(ctx.step, x, self.depth, self.averaged)

@@ -189,4 +189,4 @@ def test_the_segments_a_portion_is_cut_into():
     for longest, channels, requests in [(1, 64, 1), (17, 32, 3), (2048, 2048, 1), (100000, 40, 1), (300, 4096, 64)]:
         warps, cluster = ops.mingru_segments(longest, channels, requests, 148)
         assert 1 <= warps <= ops.MINGRU_MAX_WARPS and cluster in (1, 2, 4, 8)
-    assert ops.mingru_segments(2048, 2048, 1, 148)[1] > 1 and ops.mingru_segments(300, 4096, 64, 148)[1] == 1
+    assert ops.mingru_segments(2048, 2048, 1, 148) == (16, 8) and ops.mingru_segments(300, 4096, 64, 148)[1] == 1
