@@ -176,7 +176,7 @@ __global__ void __launch_bounds__(256) conv_heads_prepare_kernel(const ConvArgs 
 // Many tokens: a thread owns eight neighbouring elements of the outputs and walks a run of tokens with the
 // last K - 1 inputs in registers, so an input is read once; what the elements are and where they go is worked
 // out once a run. grid (runs of RUN tokens, ceil(outputs / 8 / threads)); every width in eights.
-constexpr int RUN = 16;
+constexpr int RUN = 16, AHEAD = 4;  // AHEAD tokens' inputs are asked for together
 template <typename T>
 struct alignas(16) Octet {
   T v[8];
@@ -256,7 +256,13 @@ __global__ void __launch_bounds__(256) conv_heads_runs_kernel(const ConvArgs p) 
     else hi = mid;
   }
   int end = t0;  // the first token of the run finds its request's inputs like the first of any request
+  Octet<T> raw[AHEAD];
   for (int t = t0; t < t1; ++t) {
+    if ((t - t0) % AHEAD == 0) {
+#pragma unroll
+      for (int i = 0; i < AHEAD; ++i)
+        raw[i] = *reinterpret_cast<const Octet<T>*>(col + (size_t)min(t + i, t1 - 1) * p.stride);
+    }
     if (t >= end) {
       while (p.cu_seqlens[lo + 1] <= t) ++lo;
       end = p.cu_seqlens[lo + 1];
@@ -271,11 +277,10 @@ __global__ void __launch_bounds__(256) conv_heads_runs_kernel(const ConvArgs p) 
                                       : state[(size_t)(K - 1 - (begin - src)) * p.channels + i];
       }
     }
-    const Octet<T> raw = *reinterpret_cast<const Octet<T>*>(col + (size_t)t * p.stride);
     float y[8];
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      const float x = to_f32(raw.v[i]) + bias[i];
+      const float x = to_f32(raw[0].v[i]) + bias[i];
       y[i] = w[0][i] * x;
 #pragma unroll
       for (int j = 1; j < K; ++j) y[i] = fmaf(w[j][i], before[j - 1][i], y[i]);
@@ -295,6 +300,8 @@ __global__ void __launch_bounds__(256) conv_heads_runs_kernel(const ConvArgs p) 
       out.v[i] = from_f32<T>(y[i]), out.v[i + 1] = from_f32<T>(y[i + 1]);
     }
     store(t, out);
+#pragma unroll
+    for (int i = 0; i + 1 < AHEAD; ++i) raw[i] = raw[i + 1];
   }
 }
 
