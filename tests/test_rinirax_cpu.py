@@ -84,7 +84,7 @@ def test_named_errors():
             architecture.parse(broken(change))
 
 
-@pytest.mark.parametrize("dims,base,scaling", [(32, 1e6, (2.0, 2048, 32.0, 1.0)), (6, 100.0, None), (16, 500.0, (8.0, 64, 16.0, 0.5)),
+@pytest.mark.parametrize("dims,base,scaling", [(48, 3e5, (6.0, 1024, 20.0, 2.0)), (6, 100.0, None), (16, 500.0, (8.0, 64, 16.0, 0.5)),
                                                (64, 10000.0, (40.0, 4096, 32.0, 1.0)), (8, 20.0, (3.0, 16, 1.0, 1.0))])
 def test_the_frequency_table(dims, base, scaling):
     part = Rotary(dims, base, "half", scaling)

@@ -115,8 +115,8 @@ CUTS = [[0, 30, 32, 33, 90, 131] + list(range(132, 139)), [0, 1, 2, 4, 20, 47] +
 def test_differential_attention_over_portions_slots_and_pages(dtype, H, G, dk, dv, K, rot, page):
     """Two requests in portions of 1 to 57 tokens (shorter than the convolution's reach among them), then
     single tokens, from state slots that others used before and shuffled pages filled with NaN; then a
-    second mixer with queries and a lambda of its own reads the first one's cache. A far input is made
-    loud, so that losing its key would show."""
+    second mixer with queries and a lambda of its own reads the first one's cache. Two far inputs, one at a
+    page's last place, are made loud, so that losing their keys would show."""
     D, eps, scale = 56, 1e-5, 0.9 * dk ** -0.5
     cfg = {"heads": H, "kv_heads": G, "dim": dk, "vdim": dv, "scale": scale, "conv": K, "rot": {"dims": rot, "base": 400.0}}
     position = PartSpec("rotary", {"dims": rot, "theta": 400.0, "pairing": "interleaved"}) if rot else None
@@ -129,9 +129,10 @@ def test_differential_attention_over_portions_slots_and_pages(dtype, H, G, dk, d
     lengths = [cuts[-1] for cuts in CUTS]
     g = torch.Generator().manual_seed(9)
     hs = [torch.randn(n, D, generator=g).to(DTYPES[dtype]) for n in lengths]
+    far = [3, 2 * page - 1]  # the latter a page's last place
     for h in hs:
-        h[3] *= 4.0
-        h[20:] += 0.3 * h[3]
+        h[far] *= 4.0
+        h[40:] += 0.25 * h[far].sum(0)
     pages = Pages(mixers[0], lengths, page, DTYPES[dtype], 4)
     states = [{"conv": torch.full((5, *m.state_spec()["conv"].shape), 3.0, device=CUDA)} for m in mixers]
     for s in states:
@@ -155,11 +156,11 @@ def test_differential_attention_over_portions_slots_and_pages(dtype, H, G, dk, d
             if dtype == "bfloat16":  # loud inputs make loud scores, whose rounded queries and keys cost single rows more
                 err = (mine.cpu().double() - want).abs().amax(-1) / want.abs().max()
                 assert float(err.median()) < 2.5e-2, (r, m)
-    if H > 1:
+    for place in far:
         quiet = hs[0].to(F64).clone()
-        quiet[3] = 0.0
-        assert rel(plain.differential_attention(quiet, weights[0], "", {**cfg, "diff": 0.3}, eps)[0][60:], want_of(got[0][0])[60:]) \
-            > 1.5 * tolerance
+        quiet[place] = 0.0
+        lost = plain.differential_attention(quiet, weights[0], "", {**cfg, "diff": 0.3}, eps)[0]
+        assert rel(lost[60:], want_of(got[0][0])[60:]) > 1.5 * tolerance
     if K > 1:
         for s in states:
             assert float((s["conv"][[0, 2, 4]] - 3.0).abs().max()) == 0.0  # nobody else's slot was touched
@@ -249,7 +250,7 @@ def test_convolution_of_half_split_pairs_and_of_widths_that_are_not_even():
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("H,dn,dr,dv,rank,qr,window,scaling,page", [
     (4, 32, 32, 16, 64, 48, 33, (8.0, 256, 16.0, 0.5), 16), (3, 24, 8, 20, 40, 28, 9, (4.0, 64, 8.0, 1.5), 4),
-    (5, 12, 6, 10, 20, 12, None, None, 8), (8, 16, 64, 24, 64, 40, 100, (2.0, 2048, 32.0, 1.0), 16),
+    (5, 12, 6, 10, 20, 12, None, None, 8), (8, 16, 64, 24, 64, 40, 100, (5.0, 1024, 20.0, 2.0), 16),
     (2, 32, 32, 32, 128, 64, 1, None, 16), (6, 64, 64, 64, 256, 96, 257, (40.0, 4096, 32.0, 1.0), 16)])
 def test_latent_attention_with_query_latents_and_a_window(dtype, H, dn, dr, dv, rank, qr, window, scaling, page):
     """A prompt of 330 tokens in portions and single tokens over shuffled NaN pages. Behind the window pages
@@ -341,7 +342,7 @@ def test_a_far_token_shows_through_a_closed_gate():
 
 
 @pytest.mark.parametrize("rows", [1, 9, 1300])
-@pytest.mark.parametrize("experts,top,count,keep,shift", [(16, 4, 2, 1, 0.0), (12, 3, 4, 2, -3.0), (8, 8, 4, 4, 0.0), (9, 4, 3, 2, -0.8),
+@pytest.mark.parametrize("experts,top,count,keep,shift", [(24, 5, 2, 1, 0.0), (12, 3, 4, 2, -3.0), (8, 8, 4, 4, 0.0), (9, 4, 3, 2, -0.8),
                                                           (6, 2, 6, 3, -2.0), (5, 2, 1, 1, 0.5), (256, 8, 8, 4, 0.0), (1, 1, 1, 1, -1.0)])
 def test_choice_within_the_best_groups(rows, experts, top, count, keep, shift):
     """The router kernel against the plain choice: the same experts, and weights that are shares of the chosen
