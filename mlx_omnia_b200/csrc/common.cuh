@@ -52,6 +52,30 @@ __device__ __forceinline__ float xielu(float z, float rise, float fall) {
   return z > 0.f ? fmaf(rise * z, z, 0.5f * z) : fmaf(fall, expm1f(z) - z, 0.5f * z);
 }
 
+// The tanh form of GELU, 0.5 z (1 + tanh(a)) with a = sqrt(2 / pi) (z + 0.044715 z^3), as z times the sigmoid
+// of 2 a (the same number: 1 + tanh(a) = 2 sigmoid(2 a)).
+__device__ __forceinline__ float gelu_tanh(float z) {
+  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+
+// The exact GELU, z times the normal distribution's mass below z.
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + erff(z * 0.7071067811865476f)); }
+
+// What a product's epilogue does with a (gate, up) pair, chosen by `cap`: 0 silu(gate) * up; above 0 the clamped
+// unit min(gate, cap) * sigmoid(slope * min(gate, cap)) * (clamp(up, +-cap) + 1); -1 relu(gate) * up; -2 the
+// tanh form of GELU, gelu(gate) * up. (Kernels with an epilogue of their own to hurry take the same codes.)
+#define OMNIA_UNIT_RELU (-1.f)
+#define OMNIA_UNIT_GELU_TANH (-2.f)
+__device__ __forceinline__ float gated_unit(float gate, float up, float slope, float cap) {
+  if (cap > 0.f) {
+    const float g = fminf(gate, cap), u = fminf(fmaxf(up, -cap), cap);
+    return g / (1.f + expf(-slope * g)) * (u + 1.f);
+  }
+  if (cap <= OMNIA_UNIT_GELU_TANH) return gelu_tanh(gate) * up;
+  if (cap < 0.f) return fmaxf(gate, 0.f) * up;
+  return gate / (1.f + expf(-gate)) * up;
+}
+
 // Attention whose heads are the difference of two softmax maps (query heads 2 h and 2 h + 1): a head's output
 // is a_1 - lambda a_2 over its `dv` values, divided by its own root mean square (eps inside the root), times
 // `factor`. The kernels that finish rows take this in their epilogue, in float32.

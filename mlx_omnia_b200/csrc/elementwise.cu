@@ -482,7 +482,8 @@ qkv_prepare_kernel(const T* __restrict__ proj, int row_stride, int q_col, int k_
                    const float* __restrict__ inv_freq, int rot, const int* __restrict__ positions,
                    const long long* __restrict__ slot_mapping, T* __restrict__ q_out,
                    T* __restrict__ k_pages, T* __restrict__ v_pages, long long page_stride,
-                   int page_size, long long num_slots, int whole, int interleaved, int* err) {
+                   int page_size, long long num_slots, int whole, int interleaved, const T* __restrict__ other,
+                   int other_stride, float lam, int* err) {
   pdl_wait();
   pdl_launch_dependents();
   // One block per token: the token's angles are worked out once for all its heads.
@@ -538,6 +539,11 @@ qkv_prepare_kernel(const T* __restrict__ proj, int row_stride, int q_col, int k_
       dst = (kind == 1 ? k_pages : v_pages) + page * page_stride + ((long long)head * page_size + off) * d;
     }
     if (kind == 2) {
+      if (other != nullptr) {  // the token's values of another layer mixed in
+        const T* o = other + (size_t)t * other_stride + head * d;
+        for (int i = lane; i < d; i += 32) dst[i] = from_f32<T>((1.f - lam) * to_f32(src[i]) + lam * to_f32(o[i]));
+        continue;
+      }
       for (int i = lane; i < d; i += 32) dst[i] = from_f32<T>(to_f32(src[i]) + (b ? to_f32(b[i]) : 0.f));
       continue;
     }
@@ -572,7 +578,8 @@ extern "C" int omnia_qkv_prepare(const void* proj, int row_stride, int q_col, in
                                  float eps, const float* inv_freq, int rot, const int* positions,
                                  const long long* slot_mapping, void* q_out, void* k_pages, void* v_pages,
                                  long long page_stride, int page_size, long long num_slots, int tokens, int whole,
-                                 int interleaved, int dtype, int* err, cudaStream_t stream) {
+                                 int interleaved, const void* other, int other_stride, float lam, int dtype, int* err,
+                                 cudaStream_t stream) {
   if (tokens == 0) return 0;
   if (dk > 256 || dv > 256 || rot > dk || (rot & 1) || (whole && nq + nkv > QKV_PREPARE_MAX_NORMED))
     return (int)cudaErrorInvalidValue;
@@ -581,7 +588,7 @@ extern "C" int omnia_qkv_prepare(const void* proj, int row_stride, int q_col, in
   OMNIA_DISPATCH_DTYPE(dtype, (launch_pdl(qkv_prepare_kernel<T>, tokens, threads, 0, stream, (const T*)proj, row_stride, q_col,
                                           k_col, v_col, nq, nkv, dk, dv, (const T*)bias, q_weight, k_weight, eps,
                                           inv_freq, rot, positions, slot_mapping, (T*)q_out, (T*)k_pages, (T*)v_pages,
-                                          page_stride, page_size, num_slots, whole, interleaved, err)));
+                                          page_stride, page_size, num_slots, whole, interleaved, (const T*)other, other_stride, lam, err)));
   return OMNIA_LAUNCH_RESULT();
 }
 
@@ -660,8 +667,8 @@ extern "C" int omnia_round_rows(const float* x, void* h, long long total, int dt
 
 // ---------------------------------------------------------------------------------
 // The clamped gated unit: g = min(gu[t, i], limit), u = clamp(gu[t, inner + i], -limit, limit);
-// act[t, i] = g * sigmoid(alpha * g) * (u + 1), in float32, rounded once. limit < 0 selects the unit
-// whose gate goes through a relu instead: act[t, i] = relu(gu[t, i]) * gu[t, inner + i].
+// act[t, i] = g * sigmoid(alpha * g) * (u + 1), in float32, rounded once. limit < 0 selects a unit that clamps
+// nothing (see gated_unit in common.cuh): -1 relu(gate) * up, -2 the tanh form of GELU, gelu(gate) * up.
 template <typename T>
 __global__ void clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ act, long long total, int inner,
                                    float alpha, float limit) {
@@ -671,13 +678,7 @@ __global__ void clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ act
   for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += stride) {
     const long long t = idx / inner;
     const int i = (int)(idx - t * inner);
-    if (limit < 0.f) {  // the gate through a relu, nothing clamped: relu(gate) * up
-      act[idx] = from_f32<T>(fmaxf(to_f32(gu[t * 2 * inner + i]), 0.f) * to_f32(gu[t * 2 * inner + inner + i]));
-      continue;
-    }
-    const float g = fminf(to_f32(gu[t * 2 * inner + i]), limit);
-    const float u = fminf(fmaxf(to_f32(gu[t * 2 * inner + inner + i]), -limit), limit);
-    act[idx] = from_f32<T>(g / (1.f + expf(-alpha * g)) * (u + 1.f));
+    act[idx] = from_f32<T>(gated_unit(to_f32(gu[t * 2 * inner + i]), to_f32(gu[t * 2 * inner + inner + i]), alpha, limit));
   }
 }
 
@@ -711,22 +712,58 @@ __global__ void activation_kernel(const T* __restrict__ z, T* __restrict__ act, 
       y = 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
     } else if (kind == 2) {
       y = v / (1.f + expf(-v));
-    } else {
+    } else if (kind == 3) {
       y = xielu(v, first, second);
+    } else {
+      y = gelu_erf(v);
     }
     act[idx] = from_f32<T>(y);
   }
 }
 
-// kind: 0 relu^2, 1 tanh-GELU, 2 SiLU, 3 xIELU with the constants `first` (above zero) and `second` (below).
+// kind: 0 relu^2, 1 tanh-GELU, 2 SiLU, 3 xIELU with the constants `first` (above zero) and `second` (below), 4 exact GELU.
 extern "C" int omnia_activation(const void* z, void* act, long long total, int kind, float first, float second, int dtype,
                                 cudaStream_t stream) {
   if (total == 0) return 0;
-  if (kind < 0 || kind > 3) return (int)cudaErrorInvalidValue;
+  if (kind < 0 || kind > 4) return (int)cudaErrorInvalidValue;
   const long long most = 16LL * omnia_sm_count();
   const int blocks = (int)((total + 255) / 256 < most ? (total + 255) / 256 : most);
   OMNIA_DISPATCH_DTYPE(dtype, (launch_pdl(activation_kernel<T>, blocks, 256, 0, stream, (const T*)z, (T*)act,
                                           total, kind, first, second)));
+  return OMNIA_LAUNCH_RESULT();
+}
+
+// ---------------------------------------------------------------------------------
+// In place: out[t, c] *= sigmoid(gate[t, c]), the gate's rows `gate_stride` apart; float32, rounded once. A block
+// per token; sixteen bytes a thread where both rows start on sixteen.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gate_rows_kernel(T* __restrict__ out, const T* __restrict__ gate, int gate_stride, int width) {
+  pdl_wait();
+  pdl_launch_dependents();
+  T* o = out + (size_t)blockIdx.x * width;
+  const T* g = gate + (size_t)blockIdx.x * gate_stride;
+  constexpr int VEC = 16 / (int)sizeof(T);
+  if (width % VEC == 0 && gate_stride % VEC == 0 && (((uintptr_t)out | (uintptr_t)gate) & 15) == 0) {
+    for (int c = threadIdx.x * VEC; c < width; c += blockDim.x * VEC) {
+      uint4 po = *reinterpret_cast<const uint4*>(o + c);
+      const uint4 pg = *reinterpret_cast<const uint4*>(g + c);
+      T* vo = reinterpret_cast<T*>(&po);
+      const T* vg = reinterpret_cast<const T*>(&pg);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) vo[e] = from_f32<T>(to_f32(vo[e]) / (1.f + expf(-to_f32(vg[e]))));
+      *reinterpret_cast<uint4*>(o + c) = po;
+    }
+    return;
+  }
+  for (int c = threadIdx.x; c < width; c += blockDim.x) o[c] = from_f32<T>(to_f32(o[c]) / (1.f + expf(-to_f32(g[c]))));
+}
+
+extern "C" int omnia_gate_rows(void* out, const void* gate, int gate_stride, int tokens, int width, int dtype,
+                               cudaStream_t stream) {
+  if (tokens == 0 || width == 0) return 0;
+  OMNIA_DISPATCH_DTYPE(dtype, (launch_pdl(gate_rows_kernel<T>, tokens, 256, 0, stream, (T*)out, (const T*)gate, gate_stride,
+                                          width)));
   return OMNIA_LAUNCH_RESULT();
 }
 

@@ -284,8 +284,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 // cap > 0: the clamped unit (gate below cap, up within +-cap and moved by one, slope `multiplier`).
                 const float gc = cap > 0.f ? fminf(g, cap) : g;
                 const float uc = cap > 0.f ? fminf(fmaxf(u, -cap), cap) + 1.f : u;
-                // cap < 0: the gate through a relu, relu(gate) * up.
-                v[e] = cap < 0.f ? fmaxf(g, 0.f) * u : __fdividef(gc, 1.f + __expf(-multiplier * gc)) * uc;
+                // cap -1: the gate through a relu; cap -2: through the tanh form of GELU, g sigmoid(2 a).
+                const float z = cap < OMNIA_UNIT_RELU ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : multiplier * gc;
+                v[e] = cap == OMNIA_UNIT_RELU ? fmaxf(g, 0.f) * u : __fdividef(gc, 1.f + __expf(-z)) * uc;
               }
               const int col = n0 + c + j;
               if (col + 1 < pair_offset && (pair_offset & 1) == 0) {
@@ -314,6 +315,12 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             }
           } else {
             bf16* dst = reinterpret_cast<bf16*>(out) + (size_t)row * n + n0 + c;
+            // cap 5: the exact GELU of the product, as bfloat16 would hold it (a separate kernel would read it so).
+            if (cap == 5.f) {
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                acc[j] = __float_as_uint(gelu_erf(__bfloat162float(__float2bfloat16_rn(__uint_as_float(acc[j])))));
+            }
             if (n0 + c + 32 <= n && (n & 7) == 0) {
 #pragma unroll
               for (int j = 0; j < 32; j += 8) {
@@ -438,7 +445,7 @@ int launch_grouped(const void* a, const void* w, void* out, int m, int n, int k,
 
 }  // namespace
 
-// epilogue: 0 store bfloat16 [m, n]; 1 SwiGLU, w = [gate rows | up rows] with n = 2 * inner,
+// epilogue: 0 store bfloat16 [m, n] (cap 5: the exact GELU of the product); 1 SwiGLU, w = [gate rows | up rows] with n = 2 * inner,
 // out bfloat16 [m, inner] (cap > 0: the clamped unit, the sigmoid's slope in `multiplier`); 2 soft cap, out float32 [m, n]. a and w must be 16-byte aligned and
 // k a multiple of 8 (rows of both matrices start on 16 bytes).
 extern "C" int omnia_gemm_tcgen05(const void* a, const void* w, void* out, int m, int n, int k, int epilogue,
@@ -450,20 +457,20 @@ extern "C" int omnia_gemm_tcgen05(const void* a, const void* w, void* out, int m
     return launch<256, 4, EPI_SWIGLU>(a, w, out, m, n, k, n / 2, cap > 0.f ? multiplier : 1.f, cap, err, stream);
   }
   if (epilogue == EPI_SOFTCAP) return launch<256, 4, EPI_SOFTCAP>(a, w, out, m, n, k, 0, multiplier, cap, err, stream);
-  if (epilogue != EPI_STORE) return (int)cudaErrorInvalidValue;
+  if (epilogue != EPI_STORE || (cap != 0.f && cap != 5.f)) return (int)cudaErrorInvalidValue;
   // 256-wide tiles do twice the work per byte staged; 128-wide tiles win only when they fill
   // SMs that the wide tiling would leave idle. Cost in units of one wide tile per round of all SMs.
   const long long m_tiles = (m + 127) / 128, sms = omnia_sm_count();
   const long long wide_rounds = (((n + 255) / 256) * m_tiles + sms - 1) / sms;
   const long long narrow_rounds = (((n + 127) / 128) * m_tiles + sms - 1) / sms;
-  if (wide_rounds * 100 <= narrow_rounds * 65) return launch<256, 4, EPI_STORE>(a, w, out, m, n, k, 0, 1.f, 0.f, err, stream);
-  return launch<128, 6, EPI_STORE>(a, w, out, m, n, k, 0, 1.f, 0.f, err, stream);
+  if (wide_rounds * 100 <= narrow_rounds * 65) return launch<256, 4, EPI_STORE>(a, w, out, m, n, k, 0, 1.f, cap, err, stream);
+  return launch<128, 6, EPI_STORE>(a, w, out, m, n, k, 0, 1.f, cap, err, stream);
 }
 
 // The grouped product of routed experts: a [m, k] rows sorted by expert; w [experts, n, k]; tiles
 // [max_tiles, 3] = (expert, first row, rows <= 128) and tile_count [1] in device memory. epilogue 0:
-// out [m, n] = a w_e^T; 1: n = 2 * inner (gate rows, then up rows), out [m, inner] = silu(gate) * up, or with
-// cap > 0 the clamped unit (the sigmoid's slope in `multiplier`), with cap < 0 relu(gate) * up.
+// out [m, n] = a w_e^T (cap 5: its exact GELU); 1: n = 2 * inner (gate rows, then up rows), out [m, inner] = silu(gate) * up, or with
+// cap > 0 the clamped unit (the sigmoid's slope in `multiplier`), with cap -1 relu(gate) * up, -2 tanh-GELU(gate) * up.
 extern "C" int omnia_gemm_tcgen05_grouped(const void* a, const void* w, void* out, int m, int n, int k, int experts,
                                           int epilogue, const int* tiles, const int* tile_count, int max_tiles,
                                           float multiplier, float cap, int* err, cudaStream_t stream) {
@@ -474,7 +481,7 @@ extern "C" int omnia_gemm_tcgen05_grouped(const void* a, const void* w, void* ou
     return launch_grouped<256, 4, EPI_SWIGLU>(a, w, out, m, n, k, experts, n / 2, tiles, tile_count, max_tiles,
                                               cap > 0.f ? multiplier : 1.f, cap, err, stream);
   }
-  if (epilogue != EPI_STORE) return (int)cudaErrorInvalidValue;
-  return launch_grouped<256, 4, EPI_STORE>(a, w, out, m, n, k, experts, 0, tiles, tile_count, max_tiles, 1.f, 0.f, err, stream);
+  if (epilogue != EPI_STORE || (cap != 0.f && cap != 5.f)) return (int)cudaErrorInvalidValue;
+  return launch_grouped<256, 4, EPI_STORE>(a, w, out, m, n, k, experts, 0, tiles, tile_count, max_tiles, 1.f, cap, err, stream);
 }
 

@@ -320,8 +320,9 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
                 // cap > 0: the clamped unit (gate below cap, up within +-cap and moved by one, slope `multiplier`).
                 const float gc = cap > 0.f ? fminf(g, cap) : g;
                 const float uc = cap > 0.f ? fminf(fmaxf(u, -cap), cap) + 1.f : u;
-                // cap < 0: the gate through a relu, relu(gate) * up.
-                v[e] = cap < 0.f ? fmaxf(g, 0.f) * u : __fdividef(gc, 1.f + __expf(-multiplier * gc)) * uc;
+                // cap -1: the gate through a relu; cap -2: through the tanh form of GELU, g sigmoid(2 a).
+                const float z = cap < OMNIA_UNIT_RELU ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : multiplier * gc;
+                v[e] = cap == OMNIA_UNIT_RELU ? fmaxf(g, 0.f) * u : __fdividef(gc, 1.f + __expf(-z)) * uc;
               }
               const int col = n0 + c + j;
               if (col + 1 < pair_offset && (pair_offset & 1) == 0) {

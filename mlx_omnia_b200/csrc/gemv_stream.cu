@@ -432,13 +432,8 @@ gemv_stream_kernel(const bf16* __restrict__ a, const __grid_constant__ CUtensorM
           // The two halves are rounded to bfloat16 first, as a separate product would round them.
           const float gate = __bfloat162float(__float2bfloat16_rn(v));
           up = __bfloat162float(__float2bfloat16_rn(up));
-          // cap > 0 is the clamped unit: gate held below cap, up within +-cap and moved by one, the
-          // sigmoid's slope in `multiplier`; otherwise silu(gate) * up (multiplier 1).
-          // cap < 0: the gate through a relu, relu(gate) * up.
-          float g = gate;
-          if (cap > 0.f) g = fminf(g, cap), up = fminf(fmaxf(up, -cap), cap) + 1.f;
-          reinterpret_cast<bf16*>(out)[(size_t)token * inner + col] =
-              __float2bfloat16_rn(cap < 0.f ? fmaxf(g, 0.f) * up : g / (1.f + expf(-multiplier * g)) * up);
+          // `cap` says which unit (gated_unit in common.cuh), `multiplier` is the clamped one's slope.
+          reinterpret_cast<bf16*>(out)[(size_t)token * inner + col] = __float2bfloat16_rn(gated_unit(gate, up, multiplier, cap));
         } else {
           const int col = tile * TILE_ROWS + r;
           if (col >= n) continue;
@@ -447,7 +442,7 @@ gemv_stream_kernel(const bf16* __restrict__ a, const __grid_constant__ CUtensorM
             reinterpret_cast<float*>(out)[(size_t)token * n + col] = cap > 0.f ? cap * tanhf(z / cap) : z;
           } else {
             // cap selects an activation of the stored product (0 none, 1 relu^2, 2 tanh-GELU, 3 SiLU, 4 xIELU
-            // with the constants `multiplier` and `second`), applied to the product as bfloat16 would hold it, as a separate kernel would read it.
+            // with the constants `multiplier` and `second`, 5 exact GELU), applied to the product as bfloat16 would hold it, as a separate kernel would read it.
             if (cap != 0.f) {
               const float z = __bfloat162float(__float2bfloat16_rn(v));
               if (cap == 1.f) {
@@ -457,8 +452,10 @@ gemv_stream_kernel(const bf16* __restrict__ a, const __grid_constant__ CUtensorM
                 v = 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
               } else if (cap == 3.f) {
                 v = z / (1.f + expf(-z));
-              } else {
+              } else if (cap == 4.f) {
                 v = xielu(z, multiplier, second);
+              } else {
+                v = gelu_erf(z);
               }
             }
             reinterpret_cast<bf16*>(out)[(size_t)token * n + col] = __float2bfloat16_rn(v);
@@ -545,8 +542,8 @@ int launch_rows(const bf16* a, const bf16* w, void* out, int m, int n, int k, in
 
 }  // namespace
 
-// epilogue: 0 store bfloat16 [m, n] (cap 1, 2, 3: relu^2, tanh-GELU or SiLU of the product, 4: xIELU with the constants `multiplier` and `second`; 0: as it is); 1 SwiGLU, w = [gate rows | up rows] with n = 2 * inner,
-// out bfloat16 [m, inner] (cap > 0: the clamped unit min(gate, cap) * sigmoid(multiplier * min(gate, cap)) * (clamp(up, +-cap) + 1); cap < 0: relu(gate) * up); 2 soft cap, out float32 [m, n]. err: the device error word.
+// epilogue: 0 store bfloat16 [m, n] (cap 1, 2, 3: relu^2, tanh-GELU or SiLU of the product, 4: xIELU with the constants `multiplier` and `second`, 5: exact GELU; 0: as it is); 1 SwiGLU, w = [gate rows | up rows] with n = 2 * inner,
+// out bfloat16 [m, inner] (cap > 0: the clamped unit min(gate, cap) * sigmoid(multiplier * min(gate, cap)) * (clamp(up, +-cap) + 1); cap -1: relu(gate) * up, -2: tanh-GELU(gate) * up); 2 soft cap, out float32 [m, n]. err: the device error word.
 extern "C" int omnia_gemv_stream(const void* a, const void* w, void* out, int m, int n, int k, int epilogue,
                                  float multiplier, float cap, float second, int* err, cudaStream_t stream) {
   if (m == 0 || n == 0) return 0;
@@ -561,7 +558,7 @@ extern "C" int omnia_gemv_stream(const void* a, const void* w, void* out, int m,
   }
   if (epilogue == EPI_SOFTCAP)
     return launch_rows<EPI_SOFTCAP, false>(ap, wp, out, m, n, k, 0, multiplier, cap, 0.f, none, err, stream);
-  if (epilogue != EPI_STORE || cap < 0.f || cap > 4.f) return (int)cudaErrorInvalidValue;
+  if (epilogue != EPI_STORE || cap < 0.f || cap > 5.f) return (int)cudaErrorInvalidValue;
   return launch_rows<EPI_STORE, false>(ap, wp, out, m, n, k, 0, cap == 4.f ? multiplier : 1.f, cap, second, none, err, stream);
 }
 
@@ -572,7 +569,7 @@ extern "C" int omnia_gemv_stream_pending_max_k(void) { return PENDING_MAX_K; }
 // x, x_out float32 [m, k] (different buffers, m <= 8), branch bfloat16 [m, k], wb, wo float32 [k] or null.
 extern "C" int omnia_gemv_stream_pending(const float* x, float* x_out, const void* branch, const float* wb,
                                          float eps_b, int norm_branch, const float* wo, float eps_o, const void* w,
-                                         void* out, int m, int n, int k, int epilogue, int* err,
+                                         void* out, int m, int n, int k, int epilogue, float cap, int* err,
                                          cudaStream_t stream) {
   if (m == 0 || n == 0) return 0;
   if (m > 8 || k % 8 != 0 || k <= 0 || k > PENDING_MAX_K || x == x_out) return (int)cudaErrorInvalidValue;
@@ -581,9 +578,9 @@ extern "C" int omnia_gemv_stream_pending(const float* x, float* x_out, const voi
     return (int)cudaErrorInvalidValue;
   const PendingStep pending{x, x_out, (const bf16*)branch, wb, wo, eps_b, eps_o, norm_branch};
   const bf16* wp = (const bf16*)w;
-  if (epilogue == EPI_SWIGLU) {
-    if (n % 2) return (int)cudaErrorInvalidValue;
-    return launch_rows<EPI_SWIGLU, true>(nullptr, wp, out, m, n, k, n / 2, 1.f, 0.f, 0.f, pending, err, stream);
+  if (epilogue == EPI_SWIGLU) {  // cap <= 0: which unit (gated_unit in common.cuh)
+    if (n % 2 || cap > 0.f) return (int)cudaErrorInvalidValue;
+    return launch_rows<EPI_SWIGLU, true>(nullptr, wp, out, m, n, k, n / 2, 1.f, cap, 0.f, pending, err, stream);
   }
   if (epilogue != EPI_STORE) return (int)cudaErrorInvalidValue;
   return launch_rows<EPI_STORE, true>(nullptr, wp, out, m, n, k, 0, 1.f, 0.f, 0.f, pending, err, stream);

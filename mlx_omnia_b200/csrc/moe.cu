@@ -4,14 +4,16 @@
 //   route     per token: router logits in float32, softmax over all router outputs, choice by
 //             score + correction, the `top` largest (optionally only among the experts of the groups
 //             whose two largest choice scores sum highest); the weights are the scores themselves, or
-//             the chosen ones' shares of their sum times a constant. Router
+//             the chosen ones' shares of their sum times a constant, or a softmax over the chosen
+//             logits. The same pass can give a gate for an expert that every token uses. Router
 //             outputs at or beyond `experts` name identity experts (they have no tensors).
 //   plan      one block: where each expert's rows begin in the sorted order, and the list of row
 //             tiles (expert, first row, rows) that the grouped products walk.
 //   scatter   per (token, choice): its place among its expert's rows.
 //   grouped products over the sorted rows, a tile of rows belonging to one expert:
-//             act = silu(h W_gate^T) * (h W_up^T) (the rows of h gathered through the sorted order),
-//             then out = act W_down^T.
+//             act = silu(h W_gate^T) * (h W_up^T), or another unit of a gate and an up part, or the exact
+//             GELU of h W_up^T alone (the rows of h gathered through the sorted order), then
+//             out = act W_down^T.
 //   combine   per token: the weighted sum of its choices' rows in a fixed order (identity experts
 //             add the token's own input), rounded once.
 //
@@ -25,16 +27,6 @@ namespace {
 
 constexpr int TILE_ROWS = 64;  // rows of a tile of the grouped products
 
-// What an expert does with its gate and up values: silu(gate) * up, or with limit > 0 the clamped
-// unit g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(alpha * g) * (u + 1).
-__device__ __forceinline__ float gated_unit(float gate, float up, float alpha, float limit) {
-  if (limit > 0.f) {
-    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
-    return g / (1.f + expf(-alpha * g)) * (u + 1.f);
-  }
-  return gate / (1.f + expf(-gate)) * up;
-}
-
 // ---------------------------------------------------------------------------------
 // A block routes TOK consecutive tokens (8 where there are many: every router row is then fetched
 // once for eight tokens instead of once a token; 1 in a small step, which wants warps, not reuse).
@@ -44,14 +36,16 @@ __device__ __forceinline__ float gated_unit(float gate, float up, float alpha, f
 template <typename T, int TOK, int THREADS, int CHUNK>
 __global__ void __launch_bounds__(THREADS)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
-                 int tokens, int outputs, int experts, int hidden, int top, int sigmoid_scores, int groups,
-                 int keep_groups, int normalise, float weight_scale, int* __restrict__ choice, float* __restrict__ weight, int* __restrict__ counts) {
+                 const float* __restrict__ bias, float* __restrict__ shared_gate, int tokens, int outputs, int experts,
+                 int hidden, int top, int scoring, int groups, int keep_groups, int normalise, float weight_scale,
+                 int* __restrict__ choice, float* __restrict__ weight, int* __restrict__ counts) {
   pdl_wait();
   pdl_launch_dependents();
   constexpr int WARPS = THREADS / 32;
   static_assert(TOK <= WARPS, "a warp finishes a token");
   extern __shared__ __align__(16) float route_s[];
-  const int padded = (outputs + 3) / 4 * 4;
+  const int rows = outputs + (shared_gate != nullptr);  // the router's rows: a last one for the shared gate
+  const int padded = (rows + 3) / 4 * 4;
   float* hrow = route_s;                           // [TOK][hidden]
   float* scores = hrow + (size_t)TOK * hidden;     // [TOK][padded] logits, then scores; [TOK][padded] choice scores; [TOK][padded] groups
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -65,7 +59,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
   // times the unrolling, are in flight together. (A single token: 32 warps, an output each, eight
   // steps of the columns in flight: the router's rows come from memory, and the block is their latency.)
   const bool wide = (hidden & 3) == 0 && ((uintptr_t)router & 15) == 0;
-  for (int e0 = warp; e0 < outputs; e0 += WARPS * CHUNK) {
+  for (int e0 = warp; e0 < rows; e0 += WARPS * CHUNK) {
     float acc[CHUNK][TOK];
 #pragma unroll
     for (int c = 0; c < CHUNK; ++c)
@@ -81,7 +75,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
 #pragma unroll
         for (int c = 0; c < CHUNK; ++c) {
           const int e = e0 + c * WARPS;
-          b[c] = e < outputs ? __ldg(w4 + (size_t)e * quads + q) : make_float4(0.f, 0.f, 0.f, 0.f);
+          b[c] = e < rows ? __ldg(w4 + (size_t)e * quads + q) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
 #pragma unroll
         for (int tok = 0; tok < TOK; ++tok) {
@@ -95,7 +89,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
 #pragma unroll
         for (int c = 0; c < CHUNK; ++c) {
           const int e = e0 + c * WARPS;
-          const float b = e < outputs ? router[(size_t)e * hidden + i] : 0.f;
+          const float b = e < rows ? router[(size_t)e * hidden + i] : 0.f;
 #pragma unroll
           for (int tok = 0; tok < TOK; ++tok) acc[c][tok] += hrow[(size_t)tok * hidden + i] * b;
         }
@@ -106,7 +100,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
       for (int tok = 0; tok < TOK; ++tok) {
         const float v = warp_sum(acc[c][tok]);
         const int e = e0 + c * WARPS;
-        if (lane == 0 && e < outputs) scores[(size_t)tok * padded + e] = v;
+        if (lane == 0 && e < rows) scores[(size_t)tok * padded + e] = v + (bias && e < outputs ? bias[e] : 0.f);
       }
   }
   __syncthreads();
@@ -114,6 +108,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
   const int t = t0 + warp;
   float* score = scores + (size_t)warp * padded;
   float* pick = scores + (size_t)(TOK + warp) * padded;
+  if (shared_gate != nullptr && lane == 0) shared_gate[t] = 1.f / (1.f + expf(-score[outputs]));
   float top_z = -INFINITY;
   for (int e = lane; e < outputs; e += 32) top_z = fmaxf(top_z, score[e]);
   top_z = warp_max(top_z);
@@ -121,8 +116,8 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
   for (int e = lane; e < outputs; e += 32) sum += expf(score[e] - top_z);
   sum = warp_sum(sum);
   for (int e = lane; e < outputs; e += 32) {
-    // Every output's score by itself (a sigmoid), or its share among all outputs (a softmax).
-    const float s = sigmoid_scores ? 1.f / (1.f + expf(-score[e])) : expf(score[e] - top_z) / sum;
+    // Every output's score by itself (a sigmoid), its share among all outputs (a softmax), or its logit.
+    const float s = scoring == 2 ? score[e] : scoring == 1 ? 1.f / (1.f + expf(-score[e])) : expf(score[e] - top_z) / sum;
     score[e] = s;
     pick[e] = s + (correction ? correction[e] : 0.f);
   }
@@ -179,6 +174,17 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
       chosen_sum += score[best_e];
     }
     __syncwarp();
+  }
+  if (scoring == 2) {
+    // A softmax over the chosen logits only.
+    float* w = weight + (size_t)t * top;
+    float most = -INFINITY, total = 0.f;
+    for (int k = lane; k < top; k += 32) most = fmaxf(most, w[k]);
+    most = warp_max(most);
+    for (int k = lane; k < top; k += 32) total += expf(w[k] - most);
+    total = warp_sum(total);
+    for (int k = lane; k < top; k += 32) w[k] = expf(w[k] - most) / total * weight_scale;
+    return;
   }
   if (normalise || weight_scale != 1.f) {
     chosen_sum = __shfl_sync(0xffffffffu, chosen_sum, 0);
@@ -329,6 +335,7 @@ moe_product_kernel(const T* __restrict__ a, const int* __restrict__ source, cons
       if (c >= n) continue;
       float v = acc[0][i][j];
       if (DUAL) v = gated_unit(v, acc[1][i][j], alpha, limit);
+      else if (limit == 5.f) v = gelu_erf(v);
       out[(size_t)(row0 + r) * n + c] = from_f32<T>(v);
     }
   }
@@ -473,6 +480,7 @@ moe_product_tc_kernel(const bf16* __restrict__ a, const int* __restrict__ source
         if (c >= n) continue;
         float v = acc[0][j][2 * half + e];
         if (DUAL) v = gated_unit(v, acc[PARTS - 1][j][2 * half + e], alpha, limit);
+        else if (limit == 5.f) v = gelu_erf(__bfloat162float(__float2bfloat16_rn(v)));
         out[(size_t)(row0 + r) * n + c] = __float2bfloat16_rn(v);
       }
     }
@@ -482,15 +490,16 @@ moe_product_tc_kernel(const bf16* __restrict__ a, const int* __restrict__ source
 // ---------------------------------------------------------------------------------
 // y[t] = sum over the token's choices, in their order, of weight * (the choice's row of `rows`, or the
 // token's own input h[t] for an identity expert), plus row t of `extra` when given (an expert that every
-// token uses). No `weight`: every choice counts once (the weights went into the experts' inputs). One
+// token uses; times `extra_scale[t]` when given). No `weight`: every choice counts once (the weights went into the experts' inputs). One
 // block per token.
 template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ rows, const T* __restrict__ h, const int* __restrict__ place,
-                                   const float* __restrict__ weight, const T* __restrict__ extra, T* __restrict__ y,
-                                   int hidden, int top) {
+                                   const float* __restrict__ weight, const T* __restrict__ extra,
+                                   const float* __restrict__ extra_scale, T* __restrict__ y, int hidden, int top) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x;
+  const float shared = extra_scale ? extra_scale[t] : 1.f;
   constexpr int VEC = 16 / (int)sizeof(T);
   const bool wide = hidden % VEC == 0 && ((uintptr_t)rows & 15) == 0 && ((uintptr_t)h & 15) == 0 &&
                     ((uintptr_t)y & 15) == 0 && ((uintptr_t)extra & 15) == 0;
@@ -512,7 +521,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, const T* __restri
         const uint4 piece = *reinterpret_cast<const uint4*>(extra + (size_t)t * hidden + i);
         const T* v = reinterpret_cast<const T*>(&piece);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) acc[e] += to_f32(v[e]);
+        for (int e = 0; e < VEC; ++e) acc[e] += shared * to_f32(v[e]);
       }
       uint4 out;
       T* o = reinterpret_cast<T*>(&out);
@@ -529,47 +538,53 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, const T* __restri
       const float v = p >= 0 ? to_f32(rows[(size_t)p * hidden + i]) : to_f32(h[(size_t)t * hidden + i]);
       acc += weight ? weight[(size_t)t * top + k] * v : v;
     }
-    if (extra) acc += to_f32(extra[(size_t)t * hidden + i]);
+    if (extra) acc += shared * to_f32(extra[(size_t)t * hidden + i]);
     y[(size_t)t * hidden + i] = from_f32<T>(acc);
   }
 }
 
 template <typename T, int TOK, int THREADS, int CHUNK>
-int launch_route(const T* h, const float* router, const float* correction, int tokens, int outputs, int experts,
-                 int hidden, int top, int sigmoid_scores, int groups, int keep_groups, int normalise, float weight_scale,
+int launch_route(const T* h, const float* router, const float* correction, const float* bias, float* shared_gate, int tokens,
+                 int outputs, int experts, int hidden, int top, int scoring, int groups, int keep_groups, int normalise, float weight_scale,
                  int* choice, float* weight, int* counts, size_t smem, cudaStream_t stream) {
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(moe_route_kernel<T, TOK, THREADS, CHUNK>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  launch_pdl(moe_route_kernel<T, TOK, THREADS, CHUNK>, (tokens + TOK - 1) / TOK, THREADS, smem, stream, h, router, correction, tokens,
-             outputs, experts, hidden, top, sigmoid_scores, groups, keep_groups, normalise, weight_scale, choice, weight, counts);
+  launch_pdl(moe_route_kernel<T, TOK, THREADS, CHUNK>, (tokens + TOK - 1) / TOK, THREADS, smem, stream, h, router, correction, bias,
+             shared_gate, tokens, outputs, experts, hidden, top, scoring, groups, keep_groups, normalise, weight_scale, choice, weight, counts);
   return OMNIA_LAUNCH_RESULT();
 }
 
 }  // namespace
 
-extern "C" int omnia_moe_route(const void* h, const float* router, const float* correction, int tokens, int outputs,
-                               int experts, int hidden, int top, int sigmoid_scores, int groups, int keep_groups,
+// router [outputs (+ 1), hidden]; bias [outputs] (or null) is added to the logits; correction [outputs] (or null) to
+// the scores a choice is made by. scoring: 0 softmax over all outputs, 1 sigmoids, 2 the logits themselves, the
+// weights then a softmax over the chosen ones. shared_gate (or null): float32 [tokens], the sigmoid of the router's
+// row after the last output.
+extern "C" int omnia_moe_route(const void* h, const float* router, const float* correction, const float* bias,
+                               float* shared_gate, int tokens, int outputs,
+                               int experts, int hidden, int top, int scoring, int groups, int keep_groups,
                                int normalise, float weight_scale, int* choice, float* weight, int* counts, int dtype,
                                cudaStream_t stream) {
   if (tokens == 0) return 0;
   if (groups < 1 || outputs % groups || keep_groups < 1 || keep_groups > groups || top > keep_groups * (outputs / groups))
     return (int)cudaErrorInvalidValue;
+  if (scoring < 0 || scoring > 2 || (scoring == 2 && normalise)) return (int)cudaErrorInvalidValue;
   if (top < 1 || top > outputs || experts < 0 || experts > outputs || outputs > 4096) return (int)cudaErrorInvalidValue;
-  const int padded = (outputs + 3) / 4 * 4;
+  const int padded = (outputs + (shared_gate != nullptr) + 3) / 4 * 4;
   auto bytes = [&](int tok) { return ((size_t)tok * hidden + (size_t)(groups > 1 ? 3 : 2) * tok * padded) * sizeof(float); };
   // Eight tokens a block where there are enough tokens to fill the GPU so and their rows fit.
   const bool many = tokens >= 8 * omnia_sm_count() && bytes(8) <= 160 * 1024;
   if (bytes(1) > 200 * 1024) return (int)cudaErrorInvalidValue;
   OMNIA_DISPATCH_DTYPE(dtype, {
     if (many)
-      return launch_route<T, 8, 256, 4>((const T*)h, router, correction, tokens, outputs, experts, hidden, top,
-                                        sigmoid_scores, groups, keep_groups, normalise, weight_scale, choice, weight, counts,
+      return launch_route<T, 8, 256, 4>((const T*)h, router, correction, bias, shared_gate, tokens, outputs, experts, hidden, top,
+                                        scoring, groups, keep_groups, normalise, weight_scale, choice, weight, counts,
                                         bytes(8), stream);
-    return launch_route<T, 1, 1024, 1>((const T*)h, router, correction, tokens, outputs, experts, hidden, top,
-                                       sigmoid_scores, groups, keep_groups, normalise, weight_scale, choice, weight, counts,
+    return launch_route<T, 1, 1024, 1>((const T*)h, router, correction, bias, shared_gate, tokens, outputs, experts, hidden, top,
+                                       scoring, groups, keep_groups, normalise, weight_scale, choice, weight, counts,
                                        bytes(1), stream);
   });
   return (int)cudaErrorInvalidValue;
@@ -630,7 +645,8 @@ extern "C" int omnia_moe_plan(const int* choice, int* counts, int* cursors, int*
 
 // dual != 0: w holds [experts, 2 n, k] (gate rows, then up rows) and out = silu(gate) * up.
 // limit > 0: the clamped unit instead, g = min(gate, limit), u = clamp(up, -limit, limit),
-// out = g * sigmoid(alpha * g) * (u + 1).
+// out = g * sigmoid(alpha * g) * (u + 1). dual == 0: w [experts, n, k], out the product itself or, with limit 5,
+// its exact GELU.
 extern "C" int omnia_moe_product(const void* a, const int* source, const void* w, void* out, const int* tiles,
                                  const int* tile_count, int max_tiles, int n, int k, int dual, float alpha,
                                  float limit, int dtype, int tensor_cores, cudaStream_t stream) {
@@ -735,9 +751,9 @@ extern "C" int omnia_moe_gather(const void* h, const int* source, const int* tot
 }
 
 extern "C" int omnia_moe_combine(const void* rows, const void* h, const int* place, const float* weight, const void* extra,
-                                 void* y, int tokens, int hidden, int top, int dtype, cudaStream_t stream) {
+                                 const float* extra_scale, void* y, int tokens, int hidden, int top, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
   OMNIA_DISPATCH_DTYPE(dtype, (launch_pdl(moe_combine_kernel<T>, tokens, 256, 0, stream, (const T*)rows, (const T*)h,
-                                          place, weight, (const T*)extra, (T*)y, hidden, top)));
+                                          place, weight, (const T*)extra, extra_scale, (T*)y, hidden, top)));
   return OMNIA_LAUNCH_RESULT();
 }

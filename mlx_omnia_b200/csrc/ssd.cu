@@ -1,0 +1,336 @@
+// A state-space mixer of the Mamba-2 form around its recurrence. The projected row of a token holds, from
+// `col0`, [z: inner | x: inner | B: G * N | C: G * N | dt: H] with inner = H * dv; per head h, its B and C those of
+// group h / (H / G):
+//
+//   x, B, C = silu(causal convolution per channel + bias)   (the C channels x | B | C together, K taps, the
+//             last one the current token's; a request's last K - 1 inputs carried in a state slot)
+//   dt = softplus(dt + dt_bias[h]),  a = exp(-exp(A_log[h]) dt)
+//   S_t = a S_(t-1) + dt B_t x_t^T   [N, dv],   y_t = S_t^T C_t + D_h x_t
+//   out = RMSnorm(y * silu(z)) * w, the norm taken over `norm_groups` equal runs of the heads side by side
+//
+// Three kernels, everything in float32 up to what they hand on:
+//
+//   inputs   a thread walks a channel (or a head's dt) over a run of tokens with the taps' window in registers,
+//            so every projected value is read once. Out: float32 rows [C | B | x | (a, dt) a head] for the token-by-
+//            token recurrence (state_recurrence.cu), or for the chunked one (ssd_chunk.cu) rows [x | B | C] in the
+//            element type beside float32 pairs (log a, dt).
+//   step     a step in which every request brings one token: convolution, step sizes and recurrence in one
+//            kernel, a block per (request, head, run of columns).
+//   out      per token: the skip's y times silu(z), norm and weight, rounded once; and, after the last token,
+//            per request: the convolution's carried inputs moved on.
+#include "common.cuh"
+
+namespace {
+
+constexpr int MAX_TAPS = 16;
+constexpr int RUN = 16;  // tokens a thread of the input step walks
+
+__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
+
+// The request that token t belongs to.
+__device__ __forceinline__ int request_of(const int* __restrict__ cu, int num_seqs, int t) {
+  int lo = 0, hi = num_seqs - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi) >> 1;
+    if (cu[mid + 1] > t) hi = mid;
+    else lo = mid + 1;
+  }
+  return lo;
+}
+
+struct Sizes {
+  int H, dv, G, N;
+  __host__ __device__ int inner() const { return H * dv; }
+  __host__ __device__ int channels() const { return H * dv + 2 * G * N; }
+};
+
+// grid (ceil((channels + H) / 128), ceil(tokens / RUN)), 128 threads. KT: taps held in registers (>= taps).
+// Places of x, B and C in an output row are at_x, at_b, at_c; the pairs' rows are pair_stride floats apart.
+template <typename T, typename O, int KT>
+__global__ void __launch_bounds__(128)
+ssd_inputs_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, const float* __restrict__ taps,
+                  const float* __restrict__ conv_bias, int K, const float* __restrict__ conv_state,
+                  const float* __restrict__ dt_bias, const float* __restrict__ A_log, const int* __restrict__ cu_seqlens,
+                  const int* __restrict__ state_slots, int num_seqs, int tokens, O* __restrict__ rows, int row_stride,
+                  int at_x, int at_b, int at_c, float* __restrict__ pairs, int pair_stride, int log_decay) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int C = s.channels(), inner = s.inner(), gn = s.G * s.N;
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= C + s.H) return;
+  const int t0 = blockIdx.y * RUN, t1 = min(tokens, t0 + RUN);
+  if (c >= C) {
+    const int h = c - C;
+    const float bias = dt_bias[h], rate = expf(A_log[h]);
+    for (int t = t0; t < t1; ++t) {
+      const float dt = softplus(to_f32(proj[(size_t)t * stride + col0 + inner + C + h]) + bias);
+      float2* pair = reinterpret_cast<float2*>(pairs + (size_t)t * pair_stride) + h;
+      *pair = make_float2(log_decay ? -rate * dt : expf(-rate * dt), dt);
+    }
+    return;
+  }
+  // taps [C, K]: w[KT - 1] the current token's, zeros ahead of the first.
+  float w[KT], u[KT];
+#pragma unroll
+  for (int j = 0; j < KT; ++j) {
+    const int tap = j - (KT - K);
+    w[j] = tap >= 0 ? taps[(size_t)c * K + tap] : 0.f;
+    u[j] = 0.f;
+  }
+  const float bias = conv_bias[c];
+  const T* column = proj + col0 + inner + c;
+  O* out = rows + (c < inner ? at_x + c : c < inner + gn ? at_b + (c - inner) : at_c + (c - inner - gn));
+  int seq = request_of(cu_seqlens, num_seqs, t0);
+  int begin = cu_seqlens[seq], end = cu_seqlens[seq + 1];
+  // The K - 1 inputs ahead of token t of the request: in the batch, or carried in its slot.
+  auto window = [&](int t) {
+    const float* held = conv_state + (size_t)state_slots[seq] * max(K - 1, 1) * C + c;
+#pragma unroll
+    for (int j = 0; j < KT - 1; ++j) {
+      const int back = KT - 1 - j;  // how many tokens before t
+      if (back > K - 1) {
+        u[j + 1] = 0.f;
+        continue;
+      }
+      const int at = t - back;
+      u[j + 1] = at >= begin ? to_f32(column[(size_t)at * stride]) : held[(size_t)(K - 1 + at - begin) * C];
+    }
+  };
+  window(t0);
+  T next = column[(size_t)t0 * stride];
+  for (int t = t0; t < t1; ++t) {
+    const float now = to_f32(next);
+    if (t + 1 < t1) next = column[(size_t)(t + 1) * stride];
+    if (t >= end) {
+      do {
+        ++seq;
+        begin = end, end = cu_seqlens[seq + 1];
+      } while (t >= end && seq + 1 < num_seqs);
+      window(t);
+    }
+    // u[1 .. KT - 1] are the inputs before this token, oldest first.
+    float y = bias;
+#pragma unroll
+    for (int j = 0; j < KT - 1; ++j) u[j] = u[j + 1], y = fmaf(w[j], u[j], y);
+    u[KT - 1] = now;
+    y = fmaf(w[KT - 1], now, y);
+    out[(size_t)t * row_stride] = from_f32<O>(silu(y));
+  }
+}
+
+// A block per (head x run of columns, request), 256 threads: the token's B and C (its group's) and x columns from the
+// convolution, then S moved on in place, four columns and every `teams`-th row a thread, the teams' sums added in
+// their order. y float32 [tokens, inner].
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+ssd_step_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, int cols, const float* __restrict__ taps,
+                const float* __restrict__ conv_bias, int K, const float* __restrict__ conv_state,
+                const float* __restrict__ dt_bias, const float* __restrict__ A_log, const float* __restrict__ D,
+                float* __restrict__ S_state, const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots,
+                float* __restrict__ y) {
+  pdl_wait();
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float step_s[];
+  const int parts = (s.dv + cols - 1) / cols;
+  const int head = blockIdx.x / parts, j0 = (blockIdx.x % parts) * cols, mine = min(cols, s.dv - j0), seq = blockIdx.y;
+  const int t = cu_seqlens[seq];
+  if (cu_seqlens[seq + 1] <= t) return;
+  const int C = s.channels(), inner = s.inner(), gn = s.G * s.N, N = s.N, group = head / (s.H / s.G);
+  float* b_s = step_s;                          // [N]
+  float* c_s = b_s + N;                         // [N]
+  float* x_s = c_s + N;                         // [cols]
+  float* part = x_s + ((cols + 3) & ~3);        // [teams][mine]
+  const T* row = proj + (size_t)t * stride + col0;
+  const int slot = state_slots[seq];
+  const float* held = conv_state + (size_t)slot * max(K - 1, 1) * C;
+  for (int i = threadIdx.x; i < 2 * N + mine; i += blockDim.x) {
+    const int c = i < N ? inner + group * N + i : i < 2 * N ? inner + gn + group * N + (i - N) : head * s.dv + j0 + (i - 2 * N);
+    float v = conv_bias[c];
+    for (int j = 0; j < K - 1; ++j) v = fmaf(taps[(size_t)c * K + j], held[(size_t)j * C + c], v);
+    v = fmaf(taps[(size_t)c * K + K - 1], to_f32(row[inner + c]), v);
+    (i < 2 * N ? b_s[i] : x_s[i - 2 * N]) = silu(v);
+  }
+  const float dt = softplus(to_f32(row[inner + C + head]) + dt_bias[head]);
+  const float a = expf(-expf(A_log[head]) * dt);
+  __syncthreads();
+  float* S = S_state + ((size_t)slot * s.H + head) * N * s.dv + j0;
+  const int runs = mine / VEC, teams = max(1, (int)blockDim.x / max(runs, 1));
+  for (int item = threadIdx.x; item < teams * runs; item += blockDim.x) {
+    const int m = item / runs, j = (item % runs) * VEC;
+    float sum[VEC], v[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) sum[e] = 0.f, v[e] = dt * x_s[j + e];
+#pragma unroll 8
+    for (int r = m; r < N; r += teams) {
+      float* at = S + (size_t)r * s.dv + j;
+      const float b = b_s[r], c = c_s[r];
+      if constexpr (VEC == 4) {
+        float4 st = *reinterpret_cast<const float4*>(at);
+        st.x = fmaf(b, v[0], a * st.x), st.y = fmaf(b, v[1], a * st.y);
+        st.z = fmaf(b, v[2], a * st.z), st.w = fmaf(b, v[3], a * st.w);
+        *reinterpret_cast<float4*>(at) = st;
+        sum[0] = fmaf(st.x, c, sum[0]), sum[1] = fmaf(st.y, c, sum[1]);
+        sum[2] = fmaf(st.z, c, sum[2]), sum[3] = fmaf(st.w, c, sum[3]);
+      } else {
+        const float st = fmaf(b, v[0], a * at[0]);
+        at[0] = st;
+        sum[0] = fmaf(st, c, sum[0]);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) part[m * mine + j + e] = sum[e];
+  }
+  __syncthreads();
+  for (int j = threadIdx.x; j < mine; j += blockDim.x) {
+    float o = 0.f;
+    for (int m = 0; m < teams; ++m) o += part[m * mine + j];
+    y[(size_t)t * inner + head * s.dv + j0 + j] = fmaf(D[head], x_s[j], o);
+  }
+}
+
+// Blocks 0 .. tokens - 1: a token each; the others: a request's carried inputs each.
+template <typename T>
+__global__ void __launch_bounds__(256)
+ssd_out_kernel(const float* __restrict__ y, const T* __restrict__ proj, int stride, int col0, Sizes s, int norm_groups,
+               float eps, const float* __restrict__ norm_w, int K, float* __restrict__ conv_state,
+               const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, int tokens, T* __restrict__ out) {
+  pdl_wait();
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float out_s[];
+  __shared__ float red[33];
+  const int inner = s.inner(), C = s.channels();
+  if ((int)blockIdx.x >= tokens) {
+    const int seq = blockIdx.x - tokens, begin = cu_seqlens[seq], n = cu_seqlens[seq + 1] - begin;
+    if (n <= 0 || K < 2) return;
+    float* held = conv_state + (size_t)state_slots[seq] * (K - 1) * C;
+    for (int c = threadIdx.x; c < C; c += blockDim.x)
+      // Place j of the new window is n tokens further on than place j of the old one; ascending, so that a
+      // place is read before it is written.
+      for (int j = 0; j < K - 1; ++j)
+        held[(size_t)j * C + c] = j + n < K - 1 ? held[(size_t)(j + n) * C + c]
+                                                : to_f32(proj[(size_t)(begin + j + n - (K - 1)) * stride + col0 + inner + c]);
+    return;
+  }
+  const size_t t = blockIdx.x;
+  const float* yt = y + t * inner;
+  const T* z = proj + t * stride + col0;
+  const int run = inner / norm_groups;
+  if (norm_groups == 1) {
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < inner; c += blockDim.x) {
+      const float v = yt[c] * silu(to_f32(z[c]));
+      out_s[c] = v;
+      ss += v * v;
+    }
+    const float r = 1.f / sqrtf(block_sum(ss, red) / (float)run + eps);
+    for (int c = threadIdx.x; c < inner; c += blockDim.x) out[t * inner + c] = from_f32<T>(out_s[c] * r * norm_w[c]);
+    return;
+  }
+  // A warp takes a group at a time.
+  const int lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  for (int g = threadIdx.x >> 5; g < norm_groups; g += warps) {
+    const int c0 = g * run;
+    float ss = 0.f;
+    for (int i = lane; i < run; i += 32) {
+      const float v = yt[c0 + i] * silu(to_f32(z[c0 + i]));
+      out_s[c0 + i] = v;
+      ss += v * v;
+    }
+    const float r = 1.f / sqrtf(warp_sum(ss) / (float)run + eps);
+    __syncwarp();
+    for (int i = lane; i < run; i += 32) out[t * inner + c0 + i] = from_f32<T>(out_s[c0 + i] * r * norm_w[c0 + i]);
+  }
+}
+
+template <typename T, typename O>
+int launch_inputs(const void* proj, int stride, int col0, const Sizes& s, const float* taps, const float* conv_bias, int K,
+                  const float* conv_state, const float* dt_bias, const float* A_log, const int* cu_seqlens,
+                  const int* state_slots, int num_seqs, int tokens, void* rows, int row_stride, int at_x, int at_b, int at_c,
+                  float* pairs, int pair_stride, int log_decay, cudaStream_t stream) {
+  const dim3 grid((s.channels() + s.H + 127) / 128, (tokens + RUN - 1) / RUN);
+#define OMNIA_SSD_INPUTS(KT)                                                                                              \
+  launch_pdl(ssd_inputs_kernel<T, O, KT>, grid, dim3(128), 0, stream, (const T*)proj, stride, col0, s, taps, conv_bias, K, \
+             conv_state, dt_bias, A_log, cu_seqlens, state_slots, num_seqs, tokens, (O*)rows, row_stride, at_x, at_b, at_c,  \
+             pairs, pair_stride, log_decay)
+  if (K <= 4) OMNIA_SSD_INPUTS(4);
+  else if (K <= 8) OMNIA_SSD_INPUTS(8);
+  else OMNIA_SSD_INPUTS(MAX_TAPS);
+#undef OMNIA_SSD_INPUTS
+  return OMNIA_LAUNCH_RESULT();
+}
+
+bool sizes_ok(const Sizes& s, int K) {
+  return s.H >= 1 && s.dv >= 1 && s.G >= 1 && s.N >= 1 && s.H % s.G == 0 && K >= 1 && K <= MAX_TAPS;
+}
+
+}  // namespace
+
+// wide_rows != 0: float32 rows (whatever the element type) and (a, dt) pairs; else rows in the element type and
+// (log a, dt) pairs. Places and strides in elements of what they index; pairs must start on 8 bytes in every row.
+extern "C" int omnia_ssd_inputs(const void* proj, int stride, int col0, int H, int dv, int G, int N, const float* taps,
+                                const float* conv_bias, int K, const float* conv_state, const float* dt_bias,
+                                const float* A_log, const int* cu_seqlens, const int* state_slots, int num_seqs, int tokens,
+                                void* rows, int row_stride, int at_x, int at_b, int at_c, float* pairs, int pair_stride,
+                                int wide_rows, int dtype, cudaStream_t stream) {
+  if (tokens == 0) return 0;
+  const Sizes s{H, dv, G, N};
+  if (!sizes_ok(s, K) || num_seqs < 1 || pair_stride % 2 || ((uintptr_t)pairs & 7)) return (int)cudaErrorInvalidValue;
+  OMNIA_DISPATCH_DTYPE(dtype, {
+    if (wide_rows)
+      return launch_inputs<T, float>(proj, stride, col0, s, taps, conv_bias, K, conv_state, dt_bias, A_log, cu_seqlens,
+                                     state_slots, num_seqs, tokens, rows, row_stride, at_x, at_b, at_c, pairs, pair_stride, 0, stream);
+    return launch_inputs<T, T>(proj, stride, col0, s, taps, conv_bias, K, conv_state, dt_bias, A_log, cu_seqlens, state_slots,
+                               num_seqs, tokens, rows, row_stride, at_x, at_b, at_c, pairs, pair_stride, 1, stream);
+  });
+  return (int)cudaErrorInvalidValue;
+}
+
+// cols: value columns a block takes (a multiple of 4 where dv is one).
+extern "C" int omnia_ssd_step(const void* proj, int stride, int col0, int H, int dv, int G, int N, int cols, const float* taps,
+                              const float* conv_bias, int K, const float* conv_state, const float* dt_bias,
+                              const float* A_log, const float* D, float* S_state, const int* cu_seqlens,
+                              const int* state_slots, int num_seqs, float* y, int dtype, cudaStream_t stream) {
+  if (num_seqs == 0) return 0;
+  const Sizes s{H, dv, G, N};
+  if (!sizes_ok(s, K) || cols < 1 || cols > dv) return (int)cudaErrorInvalidValue;
+  const bool fours = dv % 4 == 0 && cols % 4 == 0 && ((uintptr_t)S_state & 15) == 0;
+  // The teams' partial sums: a float for each thread's column, or more columns than threads.
+  const size_t floats = 2 * (size_t)N + ((cols + 3) & ~3) + (cols > 1024 ? cols : 1024);
+  const size_t smem = floats * sizeof(float);
+  if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+  const dim3 grid(H * ((dv + cols - 1) / cols), num_seqs);
+#define OMNIA_SSD_STEP(VEC)                                                                                               \
+  do {                                                                                                                    \
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(ssd_step_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize,       \
+                                                 (int)smem) != cudaSuccess)                                               \
+      return (int)cudaGetLastError();                                                                                     \
+    launch_pdl(ssd_step_kernel<T, VEC>, grid, dim3(256), smem, stream, (const T*)proj, stride, col0, s, cols, taps, conv_bias, \
+               K, conv_state, dt_bias, A_log, D, S_state, cu_seqlens, state_slots, y);                                     \
+  } while (0)
+  OMNIA_DISPATCH_DTYPE(dtype, {
+    if (fours) OMNIA_SSD_STEP(4);
+    else OMNIA_SSD_STEP(1);
+  });
+#undef OMNIA_SSD_STEP
+  return OMNIA_LAUNCH_RESULT();
+}
+
+extern "C" int omnia_ssd_out(const float* y, const void* proj, int stride, int col0, int H, int dv, int G, int N,
+                             int norm_groups, float eps, const float* norm_w, int K, float* conv_state,
+                             const int* cu_seqlens, const int* state_slots, int num_seqs, int tokens, void* out, int dtype,
+                             cudaStream_t stream) {
+  if (tokens == 0) return 0;
+  const Sizes s{H, dv, G, N};
+  if (!sizes_ok(s, K) || norm_groups < 1 || s.inner() % norm_groups) return (int)cudaErrorInvalidValue;
+  const size_t smem = (size_t)s.inner() * sizeof(float);
+  if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+  OMNIA_DISPATCH_DTYPE(dtype, {
+    if (smem > 47 * 1024 &&
+        cudaFuncSetAttribute(ssd_out_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      return (int)cudaGetLastError();
+    launch_pdl(ssd_out_kernel<T>, dim3(tokens + num_seqs), dim3(256), smem, stream, y, (const T*)proj, stride, col0, s,
+               norm_groups, eps, norm_w, K, conv_state, cu_seqlens, state_slots, tokens, (T*)out);
+  });
+  return OMNIA_LAUNCH_RESULT();
+}

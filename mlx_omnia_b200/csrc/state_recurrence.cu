@@ -1,8 +1,12 @@
 // Linear attention as a recurrence over a request's tokens from a float32 state carried in a slot,
-// with a decay that is a constant per head or a factor per token, head and key channel:
+// with a decay that is a constant per head, a factor per token, head and key channel, or a factor per token
+// and head (the recurrence then also takes a step size per token and head):
 //
 //   S_t = diag(a_t) S_(t-1) + k_t v_t^T      [DK, dv] per head, float32
 //   o_t = S_t^T q_t
+//
+// With a decay per token and head: S_t = a_t S_(t-1) + k_t (dt_t v_t)^T, o_t = S_t^T q_t + skip_h v_t, the q and k of
+// a head shared by a group of neighbouring heads (ssd.cu makes such rows).
 //
 // Three kernels, each taking every constant as an argument:
 //
@@ -86,16 +90,20 @@ __global__ void state_inputs_kernel(const T* __restrict__ proj, int stride, int 
   for (int c = threadIdx.x; c < H * dv; c += blockDim.x) out[v_at + c] = to_f32(row[v_col + c]);
 }
 
-// CHANNEL: a decay per token and key channel (section a of the rows); else the head's constant.
-template <int P, bool CHANNEL>
+enum { DECAY_CONSTANT = 0, DECAY_CHANNEL = 1, DECAY_TOKEN = 2 };
+
+// MODE: the head's constant; a decay per token and key channel (section a of the rows); or a decay and a step
+// size per token and head (section a: pairs). qk_heads: heads of q and k, each read by H / qk_heads heads.
+template <int P, int MODE>
 __global__ void __launch_bounds__(STATE_THREADS + STATE_LOADERS) state_recurrence_kernel(
     const float* __restrict__ rows, int row_floats, int H, int dv, int cols, int parts, int column_threads,
-    const float* __restrict__ decay,
+    const float* __restrict__ decay, int qk_heads, const float* __restrict__ skip,
     float* __restrict__ S_state, const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots,
     float* __restrict__ o_raw) {
   pdl_wait();
   pdl_launch_dependents();
   constexpr int DK = STATE_DK;
+  constexpr bool CHANNEL = MODE == DECAY_CHANNEL, TOKEN = MODE == DECAY_TOKEN;
   constexpr int R = (DK + P - 1) / P;
   // A thread's rows sit in a segment of their own, padded so that the P segments fall on different
   // banks: by four floats when the rows come in fours (segments then start on 16 bytes), else by one.
@@ -107,7 +115,8 @@ __global__ void __launch_bounds__(STATE_THREADS + STATE_LOADERS) state_recurrenc
   constexpr bool EXACT = P * R == DK;
   extern __shared__ __align__(16) float shared[];
   const int vcols = pad4(cols);
-  const int half = TC * (VECS * VROW + vcols);  // floats of one buffer: q | k | (a) [TC][VROW], v [TC][vcols]
+  // floats of one buffer: q | k | (a) [TC][VROW], v [TC][vcols], (decay, step size) [TC][2]
+  const int half = TC * (VECS * VROW + vcols + (TOKEN ? 2 : 0));
   const int head = blockIdx.x / parts, part = blockIdx.x % parts, seq = blockIdx.y;
   const int col0 = part * cols;
   const int begin = cu_seqlens[seq], end = cu_seqlens[seq + 1];
@@ -116,12 +125,14 @@ __global__ void __launch_bounds__(STATE_THREADS + STATE_LOADERS) state_recurrenc
   const int loaders = (int)blockDim.x - column_threads, lt = (int)threadIdx.x - column_threads;
   const int j = threadIdx.x / P, p = threadIdx.x % P;
   const bool live = !loader && j < cols && col0 + j < dv;
-  const float lambda = CHANNEL ? 1.f : decay[head];
-  const int qk = H * DK, k_at = pad4(qk), v_at = 2 * pad4(qk), a_at = v_at + pad4(H * dv);
+  const float constant = MODE == DECAY_CONSTANT ? decay[head] : 1.f;
+  const float direct = TOKEN && skip != nullptr ? skip[head] : 0.f;
+  const int qk_head = head / (H / qk_heads);
+  const int qk = qk_heads * DK, k_at = pad4(qk), v_at = 2 * pad4(qk), a_at = v_at + pad4(H * dv);
   // Whole 16-byte pieces from starts on 16 bytes: the asynchronous way.
   const bool wide = FOURS && cols % 4 == 0 && dv % 4 == 0 && row_floats % 4 == 0;
   constexpr int PIECES = DK / 4 > 0 ? DK / 4 : 1;
-  const int per_token = VECS * PIECES + cols / 4;
+  const int per_token = VECS * PIECES + cols / 4 + (TOKEN ? 1 : 0);
 
   auto section = [&](int which) { return which == 0 ? 0 : which == 1 ? k_at : a_at; };
   auto fetch = [&](int t0, int n, float* buf) {
@@ -136,8 +147,14 @@ __global__ void __launch_bounds__(STATE_THREADS + STATE_LOADERS) state_recurrenc
         bool past = false;
         if (piece < VECS * PIECES) {
           const int which = piece / PIECES, i0 = (piece % PIECES) * 4;
-          src = row + section(which) + head * DK + i0;
+          src = row + section(which) + qk_head * DK + i0;
           dst = buf + (which * TC + tok) * VROW + (i0 / R) * SEG + i0 % R;
+        } else if (TOKEN && piece == per_token - 1) {
+          asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"((uint32_t)__cvta_generic_to_shared(
+                           buf + TC * (VECS * VROW + vcols) + 2 * tok)), "l"(row + a_at + 2 * head) : "memory");
+          piece += loaders;
+          while (piece >= per_token) piece -= per_token, ++tok;
+          continue;
         } else {
           const int c = (piece - VECS * PIECES) * 4;
           src = row + v_at + head * dv + col0 + c;
@@ -155,7 +172,7 @@ __global__ void __launch_bounds__(STATE_THREADS + STATE_LOADERS) state_recurrenc
     } else {
       for (int idx = lt; idx < n * DK; idx += loaders) {
         const int tok = idx / DK, i = idx % DK;
-        const float* row = rows + (size_t)(t0 + tok) * row_floats + head * DK + i;
+        const float* row = rows + (size_t)(t0 + tok) * row_floats + qk_head * DK + i;
         const int at = tok * VROW + (i / R) * SEG + i % R;
         buf[at] = row[0];
         buf[TC * VROW + at] = row[k_at];
@@ -166,6 +183,9 @@ __global__ void __launch_bounds__(STATE_THREADS + STATE_LOADERS) state_recurrenc
         buf[VECS * TC * VROW + tok * vcols + c] =
             col0 + c < dv ? rows[(size_t)(t0 + tok) * row_floats + v_at + head * dv + col0 + c] : 0.f;
       }
+      if (TOKEN)
+        for (int idx = lt; idx < 2 * n; idx += loaders)
+          buf[TC * (VECS * VROW + vcols) + idx] = rows[(size_t)(t0 + idx / 2) * row_floats + a_at + 2 * head + idx % 2];
     }
   };
 
@@ -192,6 +212,7 @@ __global__ void __launch_bounds__(STATE_THREADS + STATE_LOADERS) state_recurrenc
     const float* ks = qs + TC * VROW;
     const float* as = ks + TC * VROW;
     const float* vs = qs + VECS * TC * VROW;
+    const float* steps = vs + TC * vcols;
     float sums[TC];
 #pragma unroll
     for (int tok = 0; tok < TC; ++tok) {
@@ -200,7 +221,8 @@ __global__ void __launch_bounds__(STATE_THREADS + STATE_LOADERS) state_recurrenc
         const float* kt = ks + tok * VROW + p * SEG;
         const float* qt = qs + tok * VROW + p * SEG;
         const float* at = as + tok * VROW + p * SEG;
-        const float v = live ? vs[tok * vcols + j] : 0.f;
+        float v = live ? vs[tok * vcols + j] : 0.f, lambda = constant;
+        if constexpr (TOKEN) lambda = steps[2 * tok], v *= steps[2 * tok + 1];
         float o[4] = {0.f, 0.f, 0.f, 0.f};
         if constexpr (FOURS) {
 #pragma unroll
@@ -234,6 +256,7 @@ __global__ void __launch_bounds__(STATE_THREADS + STATE_LOADERS) state_recurrenc
         float o = sums[tok];
 #pragma unroll
         for (int w = 1; w < P; w <<= 1) o += __shfl_xor_sync(0xffffffffu, o, w);
+        if (TOKEN && live) o = fmaf(direct, vs[tok * vcols + j], o);
         if (live && p == 0) o_raw[(size_t)(t0 + tok) * H * dv + head * dv + col0 + j] = o;
       }
   }
@@ -355,6 +378,12 @@ extern "C" int omnia_state_row_floats(int H, int dv, int channel) {
   return 2 * qk + v + (channel ? qk : 0);
 }
 
+// Floats of a row with a decay and a step size per token and head: [q | k | v | (decay, step size) a head].
+extern "C" int omnia_state_token_row_floats(int H, int qk_heads, int dv) {
+  const int qk = (qk_heads * STATE_DK + 3) & ~3, v = (H * dv + 3) & ~3;
+  return 2 * qk + v + ((2 * H + 3) & ~3);
+}
+
 // proj: projected rows [tokens, stride] with q at q_col, k at k_col (H * DK each), v at v_col (H * dv).
 // inv_freq: float32 [rot / 2] or null; z: decay logits, float32 [tokens, z_stride] (H * DK used) or null, with
 // z_bias float32 [H * DK] or null and inv_tau = 1 / tau. rows: float32 [tokens, row_floats].
@@ -380,36 +409,42 @@ extern "C" int omnia_state_max_cols(void) {
 }
 
 // rows: the prepared rows; channel != 0: they carry a decay per key channel, else decay float32 [H].
+// channel 2: they carry (decay, step size) per token and head, [2 H] after v; q and k then hold qk_heads heads
+// (H a multiple of them) and skip (float32 [H] or null) adds skip_h v_t to the output.
 // S_state float32 [slots, H, DK, dv], updated in place; o_raw float32 [tokens, H * dv]. cols: value
 // columns a block takes (a head is cut into ceil(dv / cols) runs; at most omnia_state_max_cols());
 // column_team: threads a column (1, 2, 4, 8 or 16; 0: chosen here).
 extern "C" int omnia_state_recurrence(const float* rows, int H, int dv, int cols, int channel, const float* decay,
-                                      float* S_state, const int* cu_seqlens, const int* state_slots, int num_seqs,
+                                      int qk_heads, const float* skip, float* S_state, const int* cu_seqlens, const int* state_slots, int num_seqs,
                                       float* o_raw, int column_team, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
-  if (H < 1 || dv < 1 || cols < 1 || cols > omnia_state_max_cols() || (!channel && decay == nullptr))
+  if (H < 1 || dv < 1 || cols < 1 || cols > omnia_state_max_cols() || (!channel && decay == nullptr) || channel < 0 ||
+      channel > DECAY_TOKEN || qk_heads < 1 || H % qk_heads || (channel != DECAY_TOKEN && (qk_heads != H || skip != nullptr)))
     return (int)cudaErrorInvalidValue;
   const int parts = (dv + cols - 1) / cols;
-  const int row_floats = omnia_state_row_floats(H, dv, channel);
+  const int row_floats = channel == DECAY_TOKEN ? omnia_state_token_row_floats(H, qk_heads, dv)
+                                                : omnia_state_row_floats(H, dv, channel);
   const dim3 grid(H * parts, num_seqs);
-#define OMNIA_STATE_LAUNCH_AS(P, CHANNEL)                                                                       \
+#define OMNIA_STATE_LAUNCH_AS(P, MODE)                                                                       \
   do {                                                                                                          \
     constexpr int R = (STATE_DK + P - 1) / P;                                                                   \
     constexpr int SEG = (R % 4 == 0 && STATE_DK % 4 == 0) ? R + 4 : R + 1;                                      \
-    const size_t smem = sizeof(float) * 2 * STATE_CHUNK * ((size_t)(CHANNEL ? 3 : 2) * P * SEG + ((cols + 3) & ~3)); \
-    if (smem > 48 * 1024 && cudaFuncSetAttribute(state_recurrence_kernel<P, CHANNEL>,                           \
+    const size_t smem = sizeof(float) * 2 * STATE_CHUNK * ((size_t)(MODE == DECAY_CHANNEL ? 3 : 2) * P * SEG +     \
+                                                       ((cols + 3) & ~3) + (MODE == DECAY_TOKEN ? 2 : 0));     \
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(state_recurrence_kernel<P, MODE>,                           \
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) \
       return (int)cudaGetLastError();                                                                           \
     const int column_threads = (cols * P + 31) / 32 * 32;                                                       \
-    launch_pdl(state_recurrence_kernel<P, CHANNEL>, grid, dim3(column_threads + STATE_LOADERS), smem, stream,    \
-               rows, row_floats, H, dv, cols, parts, column_threads, decay, S_state, cu_seqlens, state_slots,   \
+    launch_pdl(state_recurrence_kernel<P, MODE>, grid, dim3(column_threads + STATE_LOADERS), smem, stream,    \
+               rows, row_floats, H, dv, cols, parts, column_threads, decay, qk_heads, skip, S_state, cu_seqlens, state_slots,   \
                o_raw);                                                                                          \
   } while (0)
 #define OMNIA_STATE_LAUNCH(P)                                   \
   do {                                                          \
     if constexpr ((STATE_DK + P - 1) / P <= 32) {               \
-      if (channel) OMNIA_STATE_LAUNCH_AS(P, true);              \
-      else OMNIA_STATE_LAUNCH_AS(P, false);                     \
+      if (channel == DECAY_CHANNEL) OMNIA_STATE_LAUNCH_AS(P, DECAY_CHANNEL); \
+      else if (channel == DECAY_TOKEN) OMNIA_STATE_LAUNCH_AS(P, DECAY_TOKEN); \
+      else OMNIA_STATE_LAUNCH_AS(P, DECAY_CONSTANT);            \
     } else {                                                    \
       return (int)cudaErrorInvalidValue;                        \
     }                                                           \

@@ -227,13 +227,15 @@ def kv_layout(kv: KVView) -> tuple[int, int, int, int, int, int]:
 def qkv_prepare(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, nq: int, dk: int, bias: torch.Tensor | None,
                 q_weight: torch.Tensor | None, k_weight: torch.Tensor | None, eps: float | None,
                 inv_freq: torch.Tensor | None, positions: torch.Tensor, kv: KVView, store: bool,
-                whole: bool = False, interleaved: bool = False) -> torch.Tensor:
+                whole: bool = False, interleaved: bool = False,
+                mix: "tuple[torch.Tensor, int, float] | None" = None) -> torch.Tensor:
     """Per head of the projected rows: bias (the whole row's, [columns]), RMS norm with a weight of the
     head's size (q and k), rotation of the first 2 * len(inv_freq) dims in half-split pairs; q out as
     [tokens, nq, dk], and with `store` the keys and the values (of a width of their own) into the cache.
     `whole`: the norm is one root mean square over all heads of q at once (and one over all heads of k),
     its weights of the whole projection's size ([nq * dk], [nkv * dk]); `interleaved`: the rotation pairs
-    dims (2i, 2i + 1) instead of (i, i + half)."""
+    dims (2i, 2i + 1) instead of (i, i + half). `mix` (rows, col, lam): the values stored are
+    (1 - lam) v + lam (columns from `col` of `rows`, another layer's projected rows of the same tokens)."""
     tokens, stride = proj.shape
     k_ptr, v_ptr, page_stride, nkv, kdim, dv = kv_layout(kv)
     if kdim != dk:
@@ -243,11 +245,17 @@ def qkv_prepare(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, nq: int,
     fn = _function("elementwise", "omnia_qkv_prepare",
                    [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
                     c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int,
-                    c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+                    c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p])
+    other, other_stride, lam = None, 0, 0.0
+    if mix is not None:
+        rows, col, lam = mix
+        if bias is not None or rows.dtype != proj.dtype or rows.shape[0] != tokens:
+            raise KernelError("mixed values take rows of the same tokens and type, and no bias")
+        other, other_stride = rows.data_ptr() + col * rows.element_size(), rows.stride(0)
     _check(fn(_ptr(proj), stride, q_col, k_col, v_col, nq, nkv if store else 0, dk, dv, _ptr(bias), _ptr(q_weight),
               _ptr(k_weight), -1.0 if eps is None else eps, _ptr(inv_freq), rot, _ptr(positions),
               _ptr(kv.slot_mapping) if store else None, _ptr(q), k_ptr, v_ptr, page_stride, kv.page_size,
-              kv.pages.shape[0] * kv.page_size, tokens, int(whole), int(interleaved), _code(proj.dtype),
+              kv.pages.shape[0] * kv.page_size, tokens, int(whole), int(interleaved), other, other_stride, lam, _code(proj.dtype),
               _ptr(error_word(proj.device)), _stream()),
            "qkv_prepare")
     return q
@@ -900,6 +908,21 @@ def begin_pass(step: StepContext) -> None:
         step.workspace.pop("pass", None)
 
 
+def keep_for_pass(step: StepContext, name: str, value) -> None:
+    """Leave `value` (tensors of this step's tokens) for the later layers of this pass."""
+    if step.workspace is None:
+        step.workspace = {}
+    step.workspace.setdefault("pass", {})[name] = value
+
+
+def kept_for_pass(step: StepContext, name: str):
+    """What an earlier layer of this pass left under `name`."""
+    held = (step.workspace or {}).get("pass", {}).get(name)
+    if held is None:
+        raise KernelError(f"no earlier layer of this pass has left {name}")
+    return held
+
+
 def rope_angles(step: StepContext, inv_freq: torch.Tensor) -> torch.Tensor:
     """(cos, sin)(position * inv_freq) for every token of the step, float32 [len(inv_freq), tokens, 2],
     made once per pass and per table of frequencies (layers of one base share it)."""
@@ -1019,7 +1042,7 @@ def residual_after(h, x: torch.Tensor) -> torch.Tensor:
     return h.x_new
 
 
-def _pending_product(step: PendingStep, weight: torch.Tensor, epilogue: int) -> torch.Tensor | None:
+def _pending_product(step: PendingStep, weight: torch.Tensor, epilogue: int, unit: float = 0.0) -> torch.Tensor | None:
     """The product with the pending step in front, or None where the kernel does not take it."""
     if step.x_new is not None or not (weight.dtype == torch.bfloat16 and weight.shape[1] == step.x.shape[1]
                                       and weight.data_ptr() % 16 == 0 and weight.is_contiguous()
@@ -1030,10 +1053,10 @@ def _pending_product(step: PendingStep, weight: torch.Tensor, epilogue: int) -> 
     x_new = torch.empty_like(step.x)
     fn = _function("gemv_stream", "omnia_gemv_stream_pending",
                    [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_float, c_void_p, c_void_p,
-                    c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+                    c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
     _check(fn(_ptr(step.x), _ptr(x_new), _ptr(step.branch), _ptr(step.branch_weight), step.branch_eps or 0.0,
               int(step.branch_eps is not None), _ptr(step.out_weight), step.out_eps, _ptr(weight), _ptr(out), rows, n,
-              weight.shape[1], epilogue, _ptr(error_word(step.x.device)), _stream()), "gemv_stream_pending")
+              weight.shape[1], epilogue, unit, _ptr(error_word(step.x.device)), _stream()), "gemv_stream_pending")
     step.x_new = x_new
     return out
 
@@ -1097,24 +1120,33 @@ def linear_clamped_glu(a: torch.Tensor, gate_up: torch.Tensor, alpha: float, lim
     return clamped_glu(_library_mm(a, gate_up), alpha, limit)
 
 
-def linear_relu_glu(a, gate_up: torch.Tensor) -> torch.Tensor:
-    """relu(a @ gate^T) * (a @ up^T) with gate_up = [gate rows | up rows] -> [rows, inner]. The unit sits
-    where SwiGLU does (the gated epilogues' third form, selected by a negative limit): the
-    weight-streaming kernel up to 16 rows, the tcgen05 kernels from FUSED_GATE_ROWS on; in between,
-    and on the 32-bit path, the library's product and the unit's own kernel. `a` may be a PendingStep."""
-    a = settle(a)
+GATED_UNITS = {"relu": -1.0, "gelu_tanh": -2.0}
+"""The gated epilogues' other units, by the code that takes the place of the clamp's limit."""
+
+
+def linear_glu(a, gate_up: torch.Tensor, kind: str) -> torch.Tensor:
+    """f(a @ gate^T) * (a @ up^T) with gate_up = [gate rows | up rows] -> [rows, inner], f being "relu" or
+    "gelu_tanh" (the tanh form of GELU). The unit sits where SwiGLU does: the weight-streaming kernel up to
+    16 rows (with a pending residual step in front), the tcgen05 kernels from FUSED_GATE_ROWS on; in
+    between, and on the 32-bit path, the library's product and the unit's own kernel."""
+    unit = GATED_UNITS[kind]
+    if isinstance(a, PendingStep):
+        out = _pending_product(a, gate_up, 1, unit)
+        if out is not None:
+            return out
+        a = settle(a)
     if _skinny(a, gate_up):
         out = torch.empty(a.shape[0], gate_up.shape[0] // 2, dtype=a.dtype, device=a.device)
-        return _gemv_stream(a, gate_up, out, 1, 1.0, -1.0)
+        return _gemv_stream(a, gate_up, out, 1, 1.0, unit)
     if _tensor_core(a, gate_up, FUSED_GATE_ROWS):
         out = torch.empty(a.shape[0], gate_up.shape[0] // 2, dtype=a.dtype, device=a.device)
-        return _gemm_tcgen05(a, gate_up, out, 1, 1.0, -1.0)
-    gu = _library_mm(a, gate_up)
-    rows, inner = gu.shape[0], gu.shape[1] // 2
-    act = torch.empty(rows, inner, dtype=gu.dtype, device=gu.device)
-    fn = _function("elementwise", "omnia_clamped_glu", [c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p])
-    _check(fn(_ptr(gu), _ptr(act), rows, inner, 1.0, -1.0, _code(gu.dtype), _stream()), "relu_glu")
-    return act
+        return _gemm_tcgen05(a, gate_up, out, 1, 1.0, unit)
+    return clamped_glu(_library_mm(a, gate_up), 1.0, unit)
+
+
+def linear_relu_glu(a, gate_up: torch.Tensor) -> torch.Tensor:
+    """relu(a @ gate^T) * (a @ up^T) (see `linear_glu`)."""
+    return linear_glu(a, gate_up, "relu")
 
 
 def linear_softcap(a: torch.Tensor, weight: torch.Tensor, multiplier: float, cap: float | None) -> torch.Tensor:
@@ -1217,17 +1249,28 @@ def streams_leave(xs: torch.Tensor, branch: torch.Tensor, mix: torch.Tensor | No
     return h
 
 
-ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "xielu": 3}
+ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "xielu": 3, "gelu_erf": 4}
 
 
 def activation(z: torch.Tensor, kind: str, constants: tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
-    """relu(z)^2, the tanh form of GELU, SiLU, or xIELU with its two constants (`rise` z^2 + z / 2 above
+    """relu(z)^2, the tanh form of GELU, SiLU, the exact GELU, or xIELU with its two constants (`rise` z^2 + z / 2 above
     zero, `fall` (e^z - 1 - z) + z / 2 below), element by element in float32."""
     act = torch.empty_like(z)
     fn = _function("elementwise", "omnia_activation",
                    [c_void_p, c_void_p, c_longlong, c_int, c_float, c_float, c_int, c_void_p])
     _check(fn(_ptr(z), _ptr(act), z.numel(), ACTIVATIONS[kind], *constants, _code(z.dtype), _stream()), "activation")
     return act
+
+
+def gate_rows(out: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """In place: out [tokens, width] times sigmoid(gate), element by element; gate [tokens, >= width] may be columns
+    of wider rows (last dim contiguous)."""
+    tokens, width = out.shape
+    if gate.stride(1) != 1 or gate.shape[1] < width or gate.dtype != out.dtype:
+        raise KernelError("gate_rows takes a gate of the rows' type and width, its last dim contiguous")
+    fn = _function("elementwise", "omnia_gate_rows", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(out), _ptr(gate), gate.stride(0), tokens, width, _code(out.dtype), _stream()), "gate_rows")
+    return out
 
 
 def linear_act(a: torch.Tensor, weight: torch.Tensor, kind: str, constants: tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
@@ -1459,9 +1502,9 @@ def state_attention(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, gate
               tokens, _code(proj.dtype), _stream()), "state_inputs")
     o_raw = torch.empty(tokens, width, dtype=torch.float32, device=proj.device)
     fn = _function("state_recurrence", "omnia_state_recurrence",
-                   [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
-                    c_int, c_void_p], defines)
-    _check(fn(_ptr(rows), heads, dv, cols, int(channel), _ptr(decay), _ptr(S), _ptr(step.cu_seqlens),
+                   [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                    c_void_p, c_int, c_void_p], defines)
+    _check(fn(_ptr(rows), heads, dv, cols, int(channel), _ptr(decay), heads, None, _ptr(S), _ptr(step.cu_seqlens),
               _ptr(step.state_slots), step.num_seqs, _ptr(o_raw), team, _stream()), "state_recurrence")
     out = torch.empty(tokens, width, dtype=proj.dtype, device=proj.device)
     fn = _function("state_recurrence", "omnia_state_heads_out",
@@ -1470,6 +1513,96 @@ def state_attention(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, gate
     _check(fn(_ptr(o_raw), proj.data_ptr() + gate_col * proj.element_size(), stride, _ptr(norm_weight), eps, heads, dv,
               tokens, int(gate == "silu"), _ptr(out), _code(proj.dtype), _stream()), "state_heads_out")
     return out
+
+
+# ------------------------------------------------------------------------------------
+# A state-space recurrence with a decay and a step size per token and head (csrc/ssd.cu, csrc/state_recurrence.cu)
+
+SSD_MAX_TAPS = 16
+SSD_MAX_STATE = 512
+
+
+def ssd_step_columns(requests: int, heads: int, dv: int, sms: int) -> int:
+    """How many value columns of a head a block of the single-token kernel takes: all of them while (request, head)
+    pairs fill the SMs twice, else halves (down to 16 columns, in fours where dv comes in fours)."""
+    cols = dv
+    while cols >= 32 and requests * heads * -(-dv // cols) < 2 * sms:
+        cols = -(-cols // 2)
+        if dv % 4 == 0:
+            cols = -(-cols // 4) * 4
+    return cols
+
+
+@dataclass(frozen=True)
+class SSDWeights:
+    """A state-space mixer's small tensors, all float32: taps [channels, K] (the last column the current token's) and
+    conv_bias [channels] over the channels x | B | C; dt_bias, A_log, D [heads]; norm [heads * dv]."""
+
+    taps: torch.Tensor
+    conv_bias: torch.Tensor
+    dt_bias: torch.Tensor
+    A_log: torch.Tensor
+    D: torch.Tensor
+    norm: torch.Tensor
+
+
+def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N: int, w: SSDWeights, norm_groups: int,
+              eps: float, S: torch.Tensor, conv_state: torch.Tensor, step: StepContext, cols: int | None = None,
+              team: int = 0) -> torch.Tensor:
+    """A state-space mixer from its projected rows (columns from `col0`: z | x | B | C | dt) to what its output
+    projection takes, request by request from `S` [slots, heads, N, dv] and `conv_state` [slots, K - 1, channels]
+    (float32, both moved on): x, B, C = silu(convolution + bias), dt = softplus(dt + dt_bias),
+    S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T, y_t = S_t^T C_t + D x_t per head (its B and C those of its
+    group of neighbouring heads), then RMS norm of y silu(z) over `norm_groups` equal runs, with weight.
+    Everything from the projected rows on is float32. -> [tokens, heads * dv] in proj's type"""
+    tokens, stride = proj.shape
+    inner, channels, K = heads * dv, heads * dv + 2 * groups * N, w.taps.shape[1]
+    if col0 + inner + channels + heads > stride or w.taps.shape[0] != channels or not 1 <= K <= SSD_MAX_TAPS:
+        raise KernelError(f"a state-space mixer of {channels} channels and {K} taps does not fit rows of {stride}")
+    device, code = proj.device, _code(proj.dtype)
+    y = torch.empty(tokens, inner, dtype=torch.float32, device=device)
+    where = (_ptr(step.cu_seqlens), _ptr(step.state_slots), step.num_seqs)
+    if step.decode_only:
+        step_cols = ssd_step_columns(step.num_seqs, heads, dv, sm_count(device))
+        fn = _function("ssd", "omnia_ssd_step",
+                       [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                        c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p])
+        _check(fn(_ptr(proj), stride, col0, heads, dv, groups, N, step_cols, _ptr(w.taps), _ptr(w.conv_bias), K, _ptr(conv_state),
+                  _ptr(w.dt_bias), _ptr(w.A_log), _ptr(w.D), _ptr(S), *where, _ptr(y), code, _stream()), "ssd_step")
+    else:
+        pad4 = lambda n: -(-n // 4) * 4  # noqa: E731
+        at_b = pad4(groups * N)
+        at_x = 2 * at_b
+        at_pairs = at_x + pad4(inner)
+        row = at_pairs + pad4(2 * heads)
+        rows = torch.empty(tokens, row, dtype=torch.float32, device=device)
+        _ssd_inputs(proj, col0, heads, dv, groups, N, w, conv_state, where, rows, row, at_x, at_b, 0, rows[:, at_pairs:], row, True)
+        if cols is None:
+            cols = state_columns(step.num_seqs, heads, N, dv, sm_count(device))
+        fn = _function("state_recurrence", "omnia_state_recurrence",
+                       [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                        c_void_p, c_int, c_void_p], {"STATE_DK": N})
+        _check(fn(_ptr(rows), heads, dv, cols, 2, None, groups, _ptr(w.D), _ptr(S), *where, _ptr(y), team, _stream()),
+               "state_recurrence")
+    out = torch.empty(tokens, inner, dtype=proj.dtype, device=device)
+    fn = _function("ssd", "omnia_ssd_out",
+                   [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p,
+                    c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p])
+    _check(fn(_ptr(y), _ptr(proj), stride, col0, heads, dv, groups, N, norm_groups, eps, _ptr(w.norm), K, _ptr(conv_state),
+              *where, tokens, _ptr(out), code, _stream()), "ssd_out")
+    return out
+
+
+def _ssd_inputs(proj, col0, heads, dv, groups, N, w: SSDWeights, conv_state, where, rows, row_stride, at_x, at_b, at_c, pairs,
+                pair_stride, wide_rows: bool) -> None:
+    """The input step: the convolved x, B and C of every token into `rows`, and its heads' pairs into `pairs`."""
+    fn = _function("ssd", "omnia_ssd_inputs",
+                   [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                    c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int,
+                    c_void_p])
+    _check(fn(_ptr(proj), proj.shape[1], col0, heads, dv, groups, N, _ptr(w.taps), _ptr(w.conv_bias), w.taps.shape[1],
+              _ptr(conv_state), _ptr(w.dt_bias), _ptr(w.A_log), *where, proj.shape[0], _ptr(rows), row_stride, at_x, at_b, at_c,
+              _ptr(pairs), pair_stride, int(wide_rows), _code(proj.dtype), _stream()), "ssd_inputs")
 
 
 # ------------------------------------------------------------------------------------
@@ -1670,26 +1803,34 @@ def batched_mm(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None
 # Routed experts (csrc/moe.cu)
 
 
+ROUTER_SCORING = {"softmax": 0, "sigmoid": 1, "chosen": 2}
+
+
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | None, experts: int, top: int,
               counts: torch.Tensor, scoring: str = "softmax", groups: int = 1, keep_groups: int = 1,
-              normalise: bool = False, weight_scale: float = 1.0) -> tuple[torch.Tensor, torch.Tensor]:
+              normalise: bool = False, weight_scale: float = 1.0, bias: torch.Tensor | None = None,
+              shared_gate: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
     """Per row of `h`: float32 logits against `router` (float32 [outputs, hidden]), softmax over all
     outputs (or, with `scoring` "sigmoid", every output's own sigmoid), the `top` largest of score +
     correction; -> (choice int32 [rows, top], weight float32
     [rows, top]: the chosen outputs' scores; with `normalise` divided by their sum (+ 1e-20); times
     `weight_scale`). With `groups` > 1 the outputs form that many equal runs; a run's score is the sum of its
     two largest choice scores, and only outputs of the `keep_groups` best runs can be chosen. Outputs at or beyond `experts` are identity experts; the
-    others are counted into `counts` (int32 [experts], zero before the call)."""
+    others are counted into `counts` (int32 [experts], zero before the call).
+    `bias` (float32 [outputs]) is added to the logits. `scoring` "chosen": the choice is by the logits (+ correction)
+    and the weights are a softmax over the chosen logits only. `shared_gate` (float32 [rows]) receives the
+    sigmoid of one more row of `router`, its last (a gate for an expert that every row uses)."""
     rows, hidden = h.shape
+    outputs = router.shape[0] - int(shared_gate is not None)
     choice = torch.empty(rows, top, dtype=torch.int32, device=h.device)
     weight = torch.empty(rows, top, dtype=torch.float32, device=h.device)
-    if scoring not in ("softmax", "sigmoid"):
-        raise KernelError(f"router scores are a softmax or sigmoids, not {scoring!r}")
+    if scoring not in ROUTER_SCORING or (scoring == "chosen" and normalise):
+        raise KernelError(f"router scores are a softmax, sigmoids or a softmax of the chosen, not {scoring!r}")
     fn = _function("moe", "omnia_moe_route",
-                   [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                   [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                     c_void_p, c_void_p, c_void_p, c_int, c_void_p])
-    _check(fn(_ptr(h), _ptr(router), _ptr(correction), rows, router.shape[0], experts, hidden, top,
-              int(scoring == "sigmoid"), groups, keep_groups, int(normalise), weight_scale, _ptr(choice), _ptr(weight), _ptr(counts), _code(h.dtype), _stream()), "moe_route")
+    _check(fn(_ptr(h), _ptr(router), _ptr(correction), _ptr(bias), _ptr(shared_gate), rows, outputs, experts, hidden, top,
+              ROUTER_SCORING[scoring], groups, keep_groups, int(normalise), weight_scale, _ptr(choice), _ptr(weight), _ptr(counts), _code(h.dtype), _stream()), "moe_route")
     return choice, weight
 
 
@@ -1723,7 +1864,8 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
                 table: torch.Tensor | None = None, token_ids: torch.Tensor | None = None,
                 alpha: float = 1.0, limit: float = 0.0, scoring: str = "softmax", weigh: str = "output",
                 extra: torch.Tensor | None = None, groups: int = 1, keep_groups: int = 1, normalise: bool = False,
-                weight_scale: float = 1.0, combine: bool = True) -> "torch.Tensor | ExpertRows":
+                weight_scale: float = 1.0, combine: bool = True, bias: torch.Tensor | None = None,
+                activation: str | None = None, shared_gated: bool = False) -> "torch.Tensor | ExpertRows":
     """A routed mixture of gated feed-forward experts over the rows of `h` [rows, hidden]:
     y = sum over a row's `top` choices of score * expert(h), expert e being
     down[e] (silu(gate_e h) * (up_e h)) with gate_up [experts, 2 inner, hidden] (gate rows, then up
@@ -1742,11 +1884,19 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
     `extra` [rows, hidden]: added to y in the same pass (an expert that every row uses).
     `groups`, `keep_groups`, `normalise`, `weight_scale`: how the choice is narrowed and weighted (`moe_route`).
     `combine` False (no `extra`, no identity experts, weights on the outputs): the choices' rows and their
-    weights are returned as they are, for `depth_step` to sum on their way into the residual."""
+    weights are returned as they are, for `depth_step` to sum on their way into the residual.
+    `bias`: added to the router's logits. `activation` "gelu_erf": an expert is down(gelu(up h)) with the exact GELU
+    and no gate, `gate_up` then being [experts, inner, hidden]. `shared_gated`: the router's last row is no
+    output, the sigmoid of its product with a row of h multiplies that row of `extra`."""
     if weigh not in ("output", "input"):
         raise KernelError(f"a choice's weight goes on its expert's output or input, not {weigh!r}")
     rows, hidden = h.shape
-    experts, inner = gate_up.shape[0], gate_up.shape[1] // 2
+    if activation not in (None, "gelu_erf"):
+        raise KernelError(f"ungated experts take the exact GELU, not {activation!r}")
+    dual = activation is None
+    experts, inner = gate_up.shape[0], gate_up.shape[1] // 2 if dual else gate_up.shape[1]
+    if not dual:
+        alpha, limit = 1.0, float(ACTIVATIONS[activation] + 1)
     pairs = rows * top
     device = h.device
     if step is None:
@@ -1761,9 +1911,11 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
                                                    "moe_cursors": (experts, torch.int32, True)})
     if table is not None:
         choice, weight = moe_route_table(token_ids[:rows], table, experts, counts)
+        shared_gate = None
     else:
+        shared_gate = torch.empty(rows, dtype=torch.float32, device=device) if shared_gated else None
         choice, weight = moe_route(h, router, correction, experts, top, counts, scoring, groups, keep_groups, normalise,
-                                   weight_scale)
+                                   weight_scale, bias, shared_gate)
     ints = torch.empty(2 * pairs + experts + 1 + 3 * max_tiles + 1, dtype=torch.int32, device=device)
     place, source = ints[:pairs], ints[pairs: 2 * pairs]
     offsets = ints[2 * pairs: 2 * pairs + experts + 1]
@@ -1794,7 +1946,7 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
                             [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                              c_float, c_float, c_void_p, c_void_p])
         err = _ptr(error_word(device))
-        _check(grouped(_ptr(sorted_rows), _ptr(gate_up), _ptr(act), pairs, 2 * inner, hidden, experts, 1, _ptr(tiles),
+        _check(grouped(_ptr(sorted_rows), _ptr(gate_up), _ptr(act), pairs, gate_up.shape[1], hidden, experts, int(dual), _ptr(tiles),
                        _ptr(tile_count), max_tiles, alpha, limit, err, _stream()), "gemm_tcgen05_grouped")
         _check(grouped(_ptr(act), _ptr(down), _ptr(out), pairs, hidden, inner, experts, 0, _ptr(tiles),
                        _ptr(tile_count), max_tiles, 1.0, 0.0, err, _stream()), "gemm_tcgen05_grouped")
@@ -1804,17 +1956,18 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
                              c_float, c_float, c_int, c_int, c_void_p])
         _check(product(_ptr(h if sorted_rows is None else sorted_rows), _ptr(source) if sorted_rows is None else None,
                        _ptr(gate_up), _ptr(act), _ptr(tiles), _ptr(tile_count), max_tiles, inner,
-                       hidden, 1, alpha, limit, _code(h.dtype), int(tensor_cores), _stream()), "moe_product")
+                       hidden, int(dual), alpha, limit, _code(h.dtype), int(tensor_cores), _stream()), "moe_product")
         _check(product(_ptr(act), None, _ptr(down), _ptr(out), _ptr(tiles), _ptr(tile_count), max_tiles, hidden, inner, 0,
                        1.0, 0.0, _code(h.dtype), int(tensor_cores), _stream()), "moe_product")
     if not combine:
-        if extra is not None or weigh != "output" or (router is not None and router.shape[0] != experts):
+        if extra is not None or shared_gated or weigh != "output" or (router is not None and router.shape[0] != experts):
             raise KernelError("rows that are summed elsewhere have no extra branch, no identity experts and weigh outputs")
         return ExpertRows(out, place, weight, top)
     y = torch.empty_like(h)
     fn = _function("moe", "omnia_moe_combine",
-                   [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check(fn(_ptr(out), _ptr(h), _ptr(place), _ptr(weight) if weigh == "output" else None, _ptr(extra), _ptr(y), rows,
+                   [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(out), _ptr(h), _ptr(place), _ptr(weight) if weigh == "output" else None, _ptr(extra), _ptr(shared_gate),
+              _ptr(y), rows,
               hidden, top, _code(h.dtype), _stream()), "moe_combine")
     return y
 

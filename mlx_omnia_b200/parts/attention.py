@@ -132,7 +132,9 @@ class LatentAttention(Mixer):
               `norm_eps`), and the query heads are uq c_q (tensors `dq` [q_rank, hidden], `dq.norm`, `uq`
               [heads * (dim + rot_dim), q_rank] instead of `q`)
     sink:     the softmax's denominator also holds exp(sink_h) (tensor `sink` [heads], unscaled)
-    gated:    head h's output is multiplied by sigmoid(g(h))_h (tensor `g` [heads, hidden])
+    gated:    True: head h's output is multiplied by sigmoid(g(h))_h (tensor `g` [heads, hidden]); "values": the
+              heads' outputs side by side are multiplied element by element by sigmoid(g(h)) (tensor `g`
+              [heads * vdim, hidden])
     window:   None, or how many latest positions are visible
 
     Tensors: q [heads * (dim + rot_dim), hidden]; dkv [kv_rank + rot_dim, hidden]; dkv.norm [kv_rank];
@@ -142,12 +144,14 @@ class LatentAttention(Mixer):
     graph_safe_mixed = True
 
     def __init__(self, hidden: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float,
-                 norm_eps: float, position: PartSpec, sink: bool = True, gated: bool = True,
+                 norm_eps: float, position: PartSpec, sink: bool = True, gated: "bool | str" = True,
                  window: int | None = None, q_rank: int | None = None) -> None:
         if kv_rank > ops.LATENT_MAX_RANK:
             raise ValueError(f"latent_attention takes a latent of at most {ops.LATENT_MAX_RANK}")
         self.hidden, self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank = hidden, heads, dim, rot_dim, vdim, kv_rank
         self.scale, self.norm_eps, self.sink, self.gated, self.window = float(scale), float(norm_eps), sink, gated, window
+        if gated not in (False, True, "values"):
+            raise ValueError(f"gated is False, True or 'values', not {gated!r}")
         self.position = POSITIONS.build(position)
         self.q_rank = q_rank
         if getattr(self.position, "pairing", None) not in ("interleaved", "half"):
@@ -172,7 +176,7 @@ class LatentAttention(Mixer):
         if self.sink:
             specs["sink"] = TensorSpec((H,), "vector")
         if self.gated:
-            specs["g"] = TensorSpec((H, self.hidden))
+            specs["g"] = TensorSpec((H * self.vdim if self.gated == "values" else H, self.hidden))
         return specs
 
     def load(self, tensors, runtime) -> None:
@@ -189,7 +193,7 @@ class LatentAttention(Mixer):
         total = self.gate_col
         if self.gated:
             rows.append(tensors["g"])
-            total += H
+            total += tensors["g"].shape[0]
         if total % 8:
             rows.append(torch.zeros(8 - total % 8, self.hidden, dtype=rows[0].dtype, device=rows[0].device))
         self.in_proj = torch.cat(rows, dim=0).contiguous()
@@ -217,10 +221,13 @@ class LatentAttention(Mixer):
         q_lat = ops.batched_mm(q[:, :, : self.dim].transpose(0, 1), self.uk)  # [H, tokens, rank]
         o_lat = torch.empty(H, tokens, self.kv_rank, dtype=proj.dtype, device=proj.device)
         ops.latent_attention(q_lat, q[:, :, self.dim:], ctx.kv, step, self.scale, self.sink_logits,
-                             proj[:, self.gate_col:] if self.gated else None, o_lat)
+                             proj[:, self.gate_col:] if self.gated is True else None, o_lat)
         out = torch.empty(tokens, H, self.vdim, dtype=proj.dtype, device=proj.device)
         ops.batched_mm(o_lat, self.uv_t, out=out.transpose(0, 1))
-        return ops.linear(out.view(tokens, H * self.vdim), self.o)
+        out = out.view(tokens, H * self.vdim)
+        if self.gated == "values":
+            ops.gate_rows(out, proj[:, self.gate_col: self.gate_col + H * self.vdim])
+        return ops.linear(out, self.o)
 
 
 @register_mixer("sink_window_attention")
@@ -252,6 +259,9 @@ class SinkWindowAttention(Mixer):
                 [heads * vdim, hidden]) ahead of the output projection; g reads the mixer's own input
     chunk:      None, or the length of the runs that positions are cut into (from the request's
                 position 0): a query sees key j <= i only of its own run
+    value_mix:  None; "source": later layers of the pass mix this layer's projected values into theirs; "mixed":
+                the values kept are (1 - lambda) v + lambda v_first, v_first being the source layer's values of the
+                same tokens. Both have the tensor `vmix` (one number, lambda; unused by the source)
     softcap:    None, or c: a scaled score s becomes c tanh(s / c) ahead of the softmax
     The position part may pair dims half-split (i, i + dims / 2) or interleaved (2i, 2i + 1).
 
@@ -265,7 +275,8 @@ class SinkWindowAttention(Mixer):
                  window: int | None = None, keep_first: int = 0, norm_eps: float | None = None,
                  position: PartSpec | None = None, bias: bool = False, sink: bool = False, own_kv: bool = True,
                  norm_over: str = "head", gated: bool = False, chunk: int | None = None,
-                 softcap: float | None = None, norm_weight: bool = True, values: str = "own") -> None:
+                 softcap: float | None = None, norm_weight: bool = True, values: str = "own",
+                 value_mix: str | None = None) -> None:
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads do not divide into {kv_heads} groups")
         if dim > 256 or vdim > 256:
@@ -282,7 +293,9 @@ class SinkWindowAttention(Mixer):
             raise ValueError(f"sink is False, True or 'zero', not {sink!r}")
         if values not in ("own", "keys") or (values == "keys" and (vdim != dim or bias)):
             raise ValueError("values are 'own' or, without biases and with vdim = dim, 'keys'")
-        self.norm_weight, self.values = bool(norm_weight), values
+        if value_mix not in (None, "source", "mixed") or (value_mix is not None and (bias or not own_kv)):
+            raise ValueError("value_mix is None, 'source' or 'mixed', for a layer with unbiased values of its own")
+        self.norm_weight, self.values, self.value_mix = bool(norm_weight), values, value_mix
         self.hidden, self.heads, self.kv_heads, self.dim, self.vdim = hidden, heads, kv_heads, dim, vdim
         self.scale, self.window, self.keep_first, self.norm_eps = float(scale), window, int(keep_first), norm_eps
         self.bias, self.sink, self.own_kv = bias, sink, own_kv
@@ -313,6 +326,8 @@ class SinkWindowAttention(Mixer):
             specs["k"] = TensorSpec((G * dk, self.hidden))
             if self.values == "own":
                 specs["v"] = TensorSpec((G * dv, self.hidden))
+            if self.value_mix is not None:
+                specs["vmix"] = TensorSpec((), "vector")
             if self.bias:
                 specs["k.b"], specs["v.b"] = TensorSpec((G * dk,)), TensorSpec((G * dv,))
             if self.norm_eps is not None and self.norm_weight:
@@ -345,6 +360,7 @@ class SinkWindowAttention(Mixer):
         weighted = self.norm_eps is not None and self.norm_weight
         self.q_norm = tensors["q.norm"].contiguous() if weighted else None
         self.k_norm = tensors["k.norm"].contiguous() if weighted and self.own_kv else None
+        self.lam = float(tensors["vmix"]) if self.value_mix == "mixed" else 0.0
         self.sink_logits = None
         if self.sink is True:
             self.sink_logits = tensors["sink"].contiguous()
@@ -365,9 +381,14 @@ class SinkWindowAttention(Mixer):
             raise RuntimeError("a mixer without k/v projections cannot own a cache entry")
         if col0 and self.in_bias is not None:
             raise RuntimeError("biased projections start at the projected rows' first column")
+        mix = None
+        if self.value_mix == "source":
+            ops.keep_for_pass(ctx.step, "first_values", (proj, col0 + self.v_col))
+        elif self.value_mix == "mixed":
+            mix = (*ops.kept_for_pass(ctx.step, "first_values"), self.lam)
         q = ops.qkv_prepare(proj, col0, col0 + self.k_col, col0 + self.v_col, self.heads, self.dim, self.in_bias, self.q_norm,
                             self.k_norm, self.norm_eps, self.position.table(), ctx.step.positions, ctx.kv,
-                            store=self.own_kv, whole=self.norm_over == "projection", interleaved=self.interleaved)
+                            store=self.own_kv, whole=self.norm_over == "projection", interleaved=self.interleaved, mix=mix)
         return ops.paged_attention(q, ctx.kv, ctx.step, self.scale, gate=proj if self.gated else None,
                                    gate_col=col0 + self.gate_col, sink=self.sink_logits, window=self.window,
                                    keep_first=self.keep_first, chunk=self.chunk, softcap=self.softcap)

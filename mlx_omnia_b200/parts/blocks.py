@@ -50,13 +50,13 @@ def residual_step(x: torch.Tensor, branch: torch.Tensor, branch_norm: Norm | Non
 class _TwoBranchBlock(Block):
     norm_names: tuple[str, ...] = ()
 
-    def __init__(self, mixer: PartSpec, feed_forward: PartSpec, norms: dict[str, PartSpec],
+    def __init__(self, mixer: PartSpec, feed_forward: PartSpec | None, norms: dict[str, PartSpec],
                  mixer_name: str = "self_attn", feed_forward_name: str = "mlp") -> None:
         missing = set(self.norm_names) - set(norms)
         if missing:
             raise ValueError(f"{type(self).__name__} needs the norms {sorted(missing)}")
         self.mixer = MIXERS.build(mixer)
-        self.feed_forward = FEED_FORWARDS.build(feed_forward)
+        self.feed_forward = FEED_FORWARDS.build(feed_forward) if feed_forward is not None else None
         self.norms = {name: NORMS.build(norms[name]) for name in self.norm_names}
         self.mixer_name, self.feed_forward_name = mixer_name, feed_forward_name
         self.entry_norm = self.norms[self.norm_names[0]]
@@ -68,7 +68,8 @@ class _TwoBranchBlock(Block):
 
     def children(self):
         yield self.mixer_name, self.mixer
-        yield self.feed_forward_name, self.feed_forward
+        if self.feed_forward is not None:
+            yield self.feed_forward_name, self.feed_forward
         yield from self.norms.items()
 
     def tensors(self) -> dict[str, TensorSpec]:
@@ -162,15 +163,21 @@ class ScaledSandwichBlock(Block):
 
 @register_block("pre_norm")
 class PreNormBlock(_TwoBranchBlock):
-    """Two norms, one before each branch; branches are added as they are."""
+    """Two norms, one before each branch; branches are added as they are. The feed-forward may be missing (the
+    block then has one branch and one norm). norm_names: what the two norms' tensors are called."""
 
-    norm_names = ("input_layernorm", "post_attention_layernorm")
+    def __init__(self, mixer: PartSpec, feed_forward: PartSpec | None, norms: dict[str, PartSpec],
+                 mixer_name: str = "self_attn", feed_forward_name: str = "mlp",
+                 norm_names: tuple[str, str] = ("input_layernorm", "post_attention_layernorm")) -> None:
+        self.norm_names = tuple(norm_names) if feed_forward is not None else tuple(norm_names[:1])
+        super().__init__(mixer, feed_forward, norms, mixer_name, feed_forward_name)
 
     def forward(self, x, h, ctx, exit_norm):
         a = self._mix(h, ctx)
         x = ops.residual_after(h, x)
-        h2 = residual_step(x, a, None, self.norms["post_attention_layernorm"],
-                           getattr(self.feed_forward, "takes_pending", False))
+        if self.feed_forward is None:
+            return x, residual_step(x, a, None, exit_norm, ctx.exit_may_pend)
+        h2 = residual_step(x, a, None, self.norms[self.norm_names[1]], getattr(self.feed_forward, "takes_pending", False))
         m = self.feed_forward.forward(h2, ctx)
         x = ops.residual_after(h2, x)
         return x, residual_step(x, m, None, exit_norm, ctx.exit_may_pend)

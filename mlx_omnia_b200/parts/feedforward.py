@@ -101,16 +101,20 @@ class ClampedGLUMLP(FeedForward):
         return ops.linear(ops.linear_clamped_glu(h, self.gate_up, self.alpha, self.limit), self.down)
 
 
-@register_feed_forward("relu_glu_mlp")
-class ReluGLUMLP(FeedForward):
-    """down(relu(gate(h)) * up(h)), no biases.
+@register_feed_forward("glu_mlp")
+class GLUMLP(FeedForward):
+    """down(f(gate(h)) * up(h)), no biases.
 
-    hidden, inner: widths. Tensors: `gate`, `up` [inner, hidden] (stacked into one operand at load),
-    `down` [hidden, inner].
+    hidden, inner: widths; activation: f, "relu" or "gelu_tanh" (the tanh form of GELU).
+    Tensors: `gate`, `up` [inner, hidden] (stacked into one operand at load), `down` [hidden, inner].
     """
 
-    def __init__(self, hidden: int, inner: int) -> None:
-        self.hidden, self.inner = hidden, inner
+    takes_pending = True
+
+    def __init__(self, hidden: int, inner: int, activation: str) -> None:
+        if activation not in ops.GATED_UNITS:
+            raise ValueError(f"glu_mlp activation {activation!r}; known: {sorted(ops.GATED_UNITS)}")
+        self.hidden, self.inner, self.activation = hidden, inner, activation
 
     def tensors(self) -> dict[str, TensorSpec]:
         return {"gate": TensorSpec((self.inner, self.hidden)), "up": TensorSpec((self.inner, self.hidden)),
@@ -122,7 +126,17 @@ class ReluGLUMLP(FeedForward):
         self.down = tensors["down"].contiguous()
 
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
-        return ops.linear(ops.linear_relu_glu(h, self.gate_up), self.down)
+        return ops.linear(ops.linear_glu(h, self.gate_up, self.activation), self.down)
+
+
+@register_feed_forward("relu_glu_mlp")
+class ReluGLUMLP(GLUMLP):
+    """`glu_mlp` with a relu."""
+
+    takes_pending = False
+
+    def __init__(self, hidden: int, inner: int) -> None:
+        super().__init__(hidden, inner, "relu")
 
 
 @register_feed_forward("table_experts")
@@ -185,6 +199,12 @@ class RoutedExperts(FeedForward):
               largest choice scores, and only outputs of the `keep_groups` best runs can be chosen
     normalise: the weights are the chosen scores divided by their sum (+ 1e-20)
     weight_scale: multiplies the weights
+    scoring "chosen": the choice is by the logits, the weights are a softmax over the chosen logits only
+    router_bias: the router's logits have a bias (tensor `router.b` [experts + identity])
+    unit:     "swiglu" (above), or "gelu_erf": an expert is down(gelu(up h)) with the exact GELU and no gate (no
+              `gate` tensors; the shared expert alike)
+    shared_gate: the shared expert's output is multiplied by sigmoid(sg h), one number a token (tensor `shared.sg`
+              [1, hidden], its product taken in float32 beside the router's)
     Tensors: `router` [experts + identity, hidden], `correction` [experts + identity], and per expert i
     `e<i>.gate`, `e<i>.up` [inner, hidden], `e<i>.down` [hidden, inner] (stacked at load).
     """
@@ -192,7 +212,11 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden: int, inner: int, experts: int, top: int, identity: int = 0,
                  correction: bool = True, scoring: str = "softmax", weigh: str = "output",
                  shared_inner: int | None = None, groups: int = 1, keep_groups: int = 1, normalise: bool = False,
-                 weight_scale: float = 1.0) -> None:
+                 weight_scale: float = 1.0, router_bias: bool = False, unit: str = "swiglu",
+                 shared_gate: bool = False) -> None:
+        if unit not in ("swiglu", "gelu_erf") or (shared_gate and shared_inner is None):
+            raise ValueError(f"routed_experts unit {unit!r}; a shared gate needs a shared expert")
+        self.router_bias, self.unit, self.shared_gate = router_bias, unit, shared_gate
         outputs = experts + identity
         if groups < 1 or outputs % groups or not 1 <= keep_groups <= groups or top > keep_groups * (outputs // groups):
             raise ValueError(f"routed_experts: {top} of {outputs} outputs in {groups} groups of which {keep_groups} are kept")
@@ -200,7 +224,7 @@ class RoutedExperts(FeedForward):
         self.normalise, self.weight_scale = bool(normalise), float(weight_scale)
         if experts < 1 or identity < 0 or not 1 <= top <= experts + identity:
             raise ValueError(f"routed_experts of {experts} experts and {identity} identity ones, {top} a token")
-        if scoring not in ("softmax", "sigmoid") or weigh not in ("output", "input"):
+        if scoring not in ops.ROUTER_SCORING or weigh not in ("output", "input"):
             raise ValueError(f"routed_experts scoring {scoring!r}, weigh {weigh!r}")
         self.hidden, self.inner, self.experts, self.identity, self.top = hidden, inner, experts, identity, top
         self.corrected, self.scoring, self.weigh, self.shared_inner = correction, scoring, weigh, shared_inner
@@ -210,32 +234,43 @@ class RoutedExperts(FeedForward):
         specs = {"router": TensorSpec((outputs, self.hidden), "vector")}
         if self.corrected:
             specs["correction"] = TensorSpec((outputs,), "vector")
-        for e in range(self.experts):
-            specs[f"e{e}.gate"] = TensorSpec((self.inner, self.hidden))
-            specs[f"e{e}.up"] = TensorSpec((self.inner, self.hidden))
-            specs[f"e{e}.down"] = TensorSpec((self.hidden, self.inner))
+        if self.router_bias:
+            specs["router.b"] = TensorSpec((outputs,), "vector")
+        units = [(f"e{e}", self.inner) for e in range(self.experts)]
         if self.shared_inner is not None:
-            specs["shared.gate"] = TensorSpec((self.shared_inner, self.hidden))
-            specs["shared.up"] = TensorSpec((self.shared_inner, self.hidden))
-            specs["shared.down"] = TensorSpec((self.hidden, self.shared_inner))
+            units.append(("shared", self.shared_inner))
+        for name, inner in units:
+            if self.unit == "swiglu":
+                specs[f"{name}.gate"] = TensorSpec((inner, self.hidden))
+            specs[f"{name}.up"] = TensorSpec((inner, self.hidden))
+            specs[f"{name}.down"] = TensorSpec((self.hidden, inner))
+        if self.shared_gate:
+            specs["shared.sg"] = TensorSpec((1, self.hidden), "vector")
         return specs
 
     def load(self, tensors, runtime) -> None:
         super().load(tensors, runtime)
-        self.router = tensors["router"].contiguous()
+        # The shared expert's gate is one more row of the router's matrix, behind its outputs.
+        self.router = (torch.cat([tensors["router"], tensors["shared.sg"]]) if self.shared_gate else tensors["router"]).contiguous()
+        self.bias = tensors["router.b"].contiguous() if self.router_bias else None
         self.correction = tensors["correction"].contiguous() if self.corrected else None
-        self.gate_up = torch.stack([torch.cat([tensors[f"e{e}.gate"], tensors[f"e{e}.up"]], dim=0)
-                                    for e in range(self.experts)]).contiguous()
+
+        def first(name: str) -> torch.Tensor:  # what a unit's first product runs on
+            return tensors[name + ".up"] if self.unit == "gelu_erf" else torch.cat([tensors[name + ".gate"], tensors[name + ".up"]])
+
+        self.gate_up = torch.stack([first(f"e{e}") for e in range(self.experts)]).contiguous()
         self.down = torch.stack([tensors[f"e{e}.down"] for e in range(self.experts)]).contiguous()
         self.shared_gate_up = self.shared_down = None
         if self.shared_inner is not None:
-            self.shared_gate_up = torch.cat([tensors["shared.gate"], tensors["shared.up"]], dim=0).contiguous()
-            self.shared_down = tensors["shared.down"].contiguous()
+            self.shared_gate_up, self.shared_down = first("shared").contiguous(), tensors["shared.down"].contiguous()
 
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
         extra = None
         if self.shared_gate_up is not None:
-            extra = ops.linear(ops.linear_swiglu(h, self.shared_gate_up), self.shared_down)
+            if self.unit == "gelu_erf":
+                extra = ops.linear(ops.linear_act(h, self.shared_gate_up, self.unit), self.shared_down)
+            else:
+                extra = ops.linear(ops.linear_swiglu(h, self.shared_gate_up), self.shared_down)
         return self._experts(h, ctx, extra, True)
 
     @property
@@ -252,4 +287,5 @@ class RoutedExperts(FeedForward):
         return ops.moe_experts(h, self.router, self.correction, self.gate_up, self.down, self.top, ctx.step,
                                scoring=self.scoring, weigh=self.weigh, extra=extra, groups=self.groups,
                                keep_groups=self.keep_groups, normalise=self.normalise, weight_scale=self.weight_scale,
-                               combine=combine)
+                               combine=combine, bias=self.bias, activation=None if self.unit == "swiglu" else self.unit,
+                               shared_gated=self.shared_gate)

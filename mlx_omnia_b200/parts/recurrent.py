@@ -23,6 +23,10 @@ a = exp(-c r softplus(lam)), the output multiplied by a tanh-GELU branch.
 `min_gru` is a gated recurrence over channels whose gate and candidate read the current token only:
 S <- (1 - z) S + z cand, the output multiplied by silu(g(h)).
 
+`state_space` is the Mamba-2 form: per head a decay and a step size per token, S <- exp(-exp(A_log) dt) S +
+dt B x^T, y = S^T C + D x, with B and C shared by groups of heads behind a short convolution, y gated by
+silu(z) ahead of an RMS norm over groups of channels.
+
 `side_by_side` runs two mixers on the same input and adds their outputs with a constant each.
 """
 
@@ -367,6 +371,67 @@ class MinGRU(Mixer):
         """S * silu(g) for every channel, ahead of the output projection, from projected rows whose columns
         from `col0` on are this mixer's input projection."""
         return ops.mingru(proj, col0, col0 + self.width, col0 + 2 * self.width, self.z_bias, self.x_bias, ctx.state, ctx.step)
+
+
+@register_mixer("state_space")
+class StateSpace(Mixer):
+    """hidden: model width; heads of `vdim` channels; state: N, the rows of a head's state; groups: sets of B and C,
+    each shared by heads / groups neighbouring heads; conv: taps of the convolution over x, B and C; norm_groups:
+    equal runs of the heads side by side, each normed by its own root mean square; norm_eps: eps under the root.
+
+    The input projection's rows are [z: heads * vdim | x: heads * vdim | B: groups * N | C: groups * N | dt: heads].
+    x, B, C = silu(convolution + conv.b); dt = softplus(dt + dt_bias); per head
+    S <- exp(-exp(A_log) dt) S + dt B x^T from S = 0, y = S^T C + D x; out = o (norm(y silu(z)) norm's weight).
+
+    Tensors: in [2 * heads * vdim + 2 * groups * N + heads, hidden]; conv [channels, taps] (last column: the current
+    token's), conv.b [channels]; dt_bias, A_log, D [heads]; norm [heads * vdim]; o [hidden, heads * vdim].
+    State (float32): S [heads, N, vdim] and the convolution's last taps - 1 inputs."""
+
+    graph_safe = True
+    graph_safe_mixed = True
+    takes_pending = True  # h goes to the in-projection and nowhere else
+
+    def __init__(self, hidden: int, heads: int, vdim: int, state: int, groups: int, conv: int, norm_groups: int,
+                 norm_eps: float) -> None:
+        if groups < 1 or heads % groups:
+            raise ValueError(f"{heads} heads do not divide into {groups} groups")
+        if norm_groups < 1 or heads * vdim % norm_groups:
+            raise ValueError(f"{heads * vdim} channels do not divide into {norm_groups} norm groups")
+        if not 1 <= conv <= ops.SSD_MAX_TAPS or not 1 <= state <= ops.SSD_MAX_STATE:
+            raise ValueError(f"state_space takes 1 to {ops.SSD_MAX_TAPS} taps and a state of 1 to {ops.SSD_MAX_STATE} rows, "
+                             f"got {conv} and {state}")
+        self.hidden, self.heads, self.vdim, self.state, self.groups = hidden, heads, vdim, state, groups
+        self.conv, self.norm_groups, self.norm_eps = conv, norm_groups, float(norm_eps)
+        self.inner = heads * vdim
+        self.channels = self.inner + 2 * groups * state
+
+    def state_spec(self):
+        return {"S": StateSpec((self.heads, self.state, self.vdim), torch.float32),
+                "conv": StateSpec((max(self.conv - 1, 1), self.channels), torch.float32)}
+
+    def tensors(self) -> dict[str, TensorSpec]:
+        H, vector = self.heads, "vector"
+        return {"in": TensorSpec((self.inner + self.channels + H, self.hidden)),
+                "conv": TensorSpec((self.channels, self.conv), vector), "conv.b": TensorSpec((self.channels,), vector),
+                "dt_bias": TensorSpec((H,), vector), "A_log": TensorSpec((H,), vector), "D": TensorSpec((H,), vector),
+                "norm": TensorSpec((self.inner,), vector), "o": TensorSpec((self.hidden, self.inner))}
+
+    def load(self, tensors, runtime) -> None:
+        super().load(tensors, runtime)
+        rows = tensors["in"]  # padded to a multiple of 8 rows, for the kernels that want them so
+        if rows.shape[0] % 8:
+            rows = torch.cat([rows, torch.zeros(8 - rows.shape[0] % 8, self.hidden, dtype=rows.dtype, device=rows.device)])
+        self.in_proj, self.o = rows.contiguous(), tensors["o"].contiguous()
+        self.weights = ops.SSDWeights(*(tensors[name].contiguous() for name in ("conv", "conv.b", "dt_bias", "A_log", "D", "norm")))
+
+    def forward(self, h, ctx) -> torch.Tensor:
+        return ops.linear(self.forward_heads(ops.linear(h, self.in_proj), 0, ctx), self.o)
+
+    def forward_heads(self, proj: torch.Tensor, col0: int, ctx) -> torch.Tensor:
+        """The normed channels, ahead of the output projection, from projected rows whose columns from `col0` on
+        are this mixer's input projection."""
+        return ops.ssd_mixer(proj, col0, self.heads, self.vdim, self.groups, self.state, self.weights, self.norm_groups,
+                             self.norm_eps, ctx.state["S"], ctx.state["conv"], ctx.step)
 
 
 @register_mixer("side_by_side")
