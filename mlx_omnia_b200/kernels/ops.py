@@ -1516,7 +1516,8 @@ def state_attention(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, gate
 
 
 # ------------------------------------------------------------------------------------
-# A state-space recurrence with a decay and a step size per token and head (csrc/ssd.cu, csrc/state_recurrence.cu)
+# A state-space recurrence with a decay and a step size per token and head (csrc/ssd.cu,
+# csrc/ssd_chunk.cu, csrc/state_recurrence.cu)
 
 SSD_MAX_TAPS = 16
 SSD_MAX_STATE = 512
@@ -1533,6 +1534,20 @@ def ssd_step_columns(requests: int, heads: int, dv: int, sms: int) -> int:
     return cols
 
 
+SSD_CHUNK_MAX_STATE = 256
+
+
+def ssd_chunk_columns(requests: int, heads: int, dv: int, N: int, dtype: torch.dtype, sms: int) -> int:
+    """Value columns a block of the chunked kernel takes, or 0 where that kernel does not apply (float32, a state or
+    heads whose widths its tiles do not fit): 32, or 16 where heads are no multiple of 32 wide or 32 would leave half
+    the SMs idle."""
+    if dtype != torch.bfloat16 or N % 16 or N > SSD_CHUNK_MAX_STATE or dv % 16:
+        return 0
+    if dv % 32 or 2 * requests * heads * (dv // 32) <= sms:
+        return 16
+    return 32
+
+
 @dataclass(frozen=True)
 class SSDWeights:
     """A state-space mixer's small tensors, all float32: taps [channels, K] (the last column the current token's) and
@@ -1547,14 +1562,16 @@ class SSDWeights:
 
 
 def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N: int, w: SSDWeights, norm_groups: int,
-              eps: float, S: torch.Tensor, conv_state: torch.Tensor, step: StepContext, cols: int | None = None,
-              team: int = 0) -> torch.Tensor:
+              eps: float, S: torch.Tensor, conv_state: torch.Tensor, step: StepContext,
+              chunked: bool | None = None) -> torch.Tensor:
     """A state-space mixer from its projected rows (columns from `col0`: z | x | B | C | dt) to what its output
     projection takes, request by request from `S` [slots, heads, N, dv] and `conv_state` [slots, K - 1, channels]
     (float32, both moved on): x, B, C = silu(convolution + bias), dt = softplus(dt + dt_bias),
     S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T, y_t = S_t^T C_t + D x_t per head (its B and C those of its
     group of neighbouring heads), then RMS norm of y silu(z) over `norm_groups` equal runs, with weight.
-    Everything from the projected rows on is float32. -> [tokens, heads * dv] in proj's type"""
+    The recurrence runs in float32 token by token, or (`chunked` None: where it applies) in chunks on the tensor
+    cores from x, B and C rounded to bfloat16, everything else of it in float32 or as sums of two bfloat16
+    numbers; a step of single tokens is one kernel. -> [tokens, heads * dv] in proj's type"""
     tokens, stride = proj.shape
     inner, channels, K = heads * dv, heads * dv + 2 * groups * N, w.taps.shape[1]
     if col0 + inner + channels + heads > stride or w.taps.shape[0] != channels or not 1 <= K <= SSD_MAX_TAPS:
@@ -1569,7 +1586,19 @@ def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N
                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p])
         _check(fn(_ptr(proj), stride, col0, heads, dv, groups, N, step_cols, _ptr(w.taps), _ptr(w.conv_bias), K, _ptr(conv_state),
                   _ptr(w.dt_bias), _ptr(w.A_log), _ptr(w.D), _ptr(S), *where, _ptr(y), code, _stream()), "ssd_step")
+    elif chunked is not False and (cols := ssd_chunk_columns(step.num_seqs, heads, dv, N, proj.dtype, sm_count(device))):
+        rows = torch.empty(tokens, channels, dtype=proj.dtype, device=device)
+        pairs = torch.empty(tokens, 2 * heads, dtype=torch.float32, device=device)
+        at_b, at_c = inner, inner + groups * N
+        _ssd_inputs(proj, col0, heads, dv, groups, N, w, conv_state, where, rows, channels, 0, at_b, at_c, pairs, 2 * heads, False)
+        fn = _function("ssd_chunk", "omnia_ssd_chunk",
+                       [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
+                        c_void_p, c_int, c_void_p, c_void_p], {"SSD_N": N, "SSD_COLS": cols})
+        _check(fn(_ptr(rows), channels, 0, at_b, at_c, _ptr(pairs), heads, groups, dv, _ptr(w.D), _ptr(S), *where, _ptr(y),
+                  _stream()), "ssd_chunk")
     else:
+        if chunked:
+            raise KernelError(f"the chunked recurrence does not take a state of {N} rows and heads of {dv} in {proj.dtype}")
         pad4 = lambda n: -(-n // 4) * 4  # noqa: E731
         at_b = pad4(groups * N)
         at_x = 2 * at_b
@@ -1577,12 +1606,11 @@ def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N
         row = at_pairs + pad4(2 * heads)
         rows = torch.empty(tokens, row, dtype=torch.float32, device=device)
         _ssd_inputs(proj, col0, heads, dv, groups, N, w, conv_state, where, rows, row, at_x, at_b, 0, rows[:, at_pairs:], row, True)
-        if cols is None:
-            cols = state_columns(step.num_seqs, heads, N, dv, sm_count(device))
+        cols = state_columns(step.num_seqs, heads, N, dv, sm_count(device))
         fn = _function("state_recurrence", "omnia_state_recurrence",
                        [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                         c_void_p, c_int, c_void_p], {"STATE_DK": N})
-        _check(fn(_ptr(rows), heads, dv, cols, 2, None, groups, _ptr(w.D), _ptr(S), *where, _ptr(y), team, _stream()),
+        _check(fn(_ptr(rows), heads, dv, cols, 2, None, groups, _ptr(w.D), _ptr(S), *where, _ptr(y), 0, _stream()),
                "state_recurrence")
     out = torch.empty(tokens, inner, dtype=proj.dtype, device=device)
     fn = _function("ssd", "omnia_ssd_out",
