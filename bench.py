@@ -34,6 +34,10 @@ stand beside the like kernels of Bobarax. `--only rinirax` is that record for th
 whose residual is averaged over depth, differential attention behind short convolutions, windowed latent
 attention, a gated recurrence over channels, group-limited experts), beside Narezen at equal width, depth,
 heads and experts; its kernels stand beside the like kernels of Narezen and, for latent attention, of Fokalorn.
+`--only gisudra` is that record for the Gisudra design (a state-space recurrence with a decay per token and head,
+windowed attention with kept first tokens and mixed values, gated latent attention, ungated experts with a gated
+shared one), beside Rinirax at equal width, depth, heads, window and experts; its kernels stand beside the like
+kernels of Rinirax and, for the recurrence and the windowed attention, of Narezen and Bobarax.
 """
 
 from __future__ import annotations
@@ -1796,6 +1800,161 @@ def run_rinirax(args) -> dict:
     return record
 
 
+def gisudra_config(size: dict) -> dict:
+    """Layers in fours: a state-space recurrence of twice the width, windowed attention with kept first tokens and
+    mixed values, windowed latent attention, and the recurrence again; ungated experts with a gated shared one
+    everywhere but in the last of four, which has a dense unit."""
+    H, G, d, D, W = size["heads"], size["kv"], size["dim"], size["width"], size["window"]
+    moe = {"kind": "moe", "expert": {"ff": size["eff"]}, "router": {"experts": size["experts"], "top": size["top"]},
+           "shared": {"ff": size["eff"]}}
+    mamba = {"heads": 2 * D // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+    layers = []
+    for i in range(size["layers"]):
+        kind = i % 4
+        if kind in (0, 3):
+            layers.append({"type": "mamba2", "mixer": mamba, "mlp": moe if kind == 0 else {"kind": "dense", "ff": 2 * D}})
+        elif kind == 1:
+            mixer = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": W, "keep_first": 64},
+                     "v_mix": True}
+            layers.append({"type": "attention", "mixer": mixer, "mlp": moe})
+        else:
+            mixer = {"heads": H, "dim": d, "rot_dim": 64, "vdim": d, "kv_rank": 4 * d, "scale": (d + 64) ** -0.5,
+                     "mask": {"size": W}, "rot": {"base": 10000.0, "dims": 64}}
+            layers.append({"type": "latent_attention", "mixer": mixer, "mlp": moe})
+    return {"architecture": "Gisudra", "vocab": DOLUTAR_VOCAB, "width": D, "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def run_gisudra(args) -> dict:
+    """Prefill and decode of Gisudra and of Rinirax at equal sizes, then the new design's kernels alone (each replayed
+    from a CUDA graph), each beside the like kernel of Rinirax, or for the state recurrence and the windowed
+    attention of Narezen, or for the dense unit of Muse-Glimmer."""
+    import torch
+
+    from mlx_omnia_b200.kernels import ops
+    from mlx_omnia_b200.parts.base import KVSpec, KVView
+
+    measured, peak_source = peaks()
+    hbm, flops_peak = measured["hbm_gbs"] * 1e9, measured["bf16_tflops"] * 1e12
+    g = torch.Generator().manual_seed(SEED)
+    batch, context, tokens = args.batch, args.context, args.prefill_tokens
+    dev, bf = torch.device("cuda:0"), torch.bfloat16
+
+    def kernels(size: dict) -> dict:
+        H, G, d, D, W = size["heads"], size["kv"], size["dim"], size["width"], size["window"]
+        E, top, F, keep = size["experts"], size["top"], size["eff"], 64
+        out = {}
+
+        def note(name, fn, count, bytes_=None, flops=None):
+            ms = replayed_ms(fn, count)
+            entry = {"us": round(ms * 1000.0, 2)}
+            if bytes_ is not None:
+                entry.update(gb_s=round(bytes_ / ms / 1e6, 1), frac_hbm=round(bytes_ / (ms / 1e3) / hbm, 4))
+            if flops is not None:
+                entry.update(tflops=round(flops / ms / 1e9, 2), frac_tensor=round(flops / (ms / 1e3) / flops_peak, 4))
+            out[name] = entry
+
+        for mode, lens, starts in (("prefill", [tokens], [0]), ("decode", [1] * batch, [context - 1] * batch)):
+            st = step_alone(lens, starts, dev)
+            n, T, page, reps = len(lens), sum(lens), 16, 5 if mode == "prefill" else 20
+            # the state-space mixer between its two projections, beside Narezen's state recurrence with a decay per
+            # key channel (half the attention's heads); flops: the token-by-token form's two products a head
+            HM, dv, N, K = 2 * D // 64, 64, 128, 4
+            inner, channels = HM * dv, HM * dv + 2 * N
+            mproj = (torch.randn(T, inner + channels + HM, device=dev) * 0.5).to(bf)
+            w = ops.SSDWeights(torch.randn(channels, K, device=dev) * 0.5, torch.zeros(channels, device=dev),
+                               torch.full((HM,), -2.0, device=dev), torch.zeros(HM, device=dev), torch.ones(HM, device=dev),
+                               torch.ones(inner, device=dev))
+            S, conv = torch.zeros(n + 1, HM, N, dv, device=dev), torch.zeros(n + 1, K - 1, channels, device=dev)
+            note(f"ssd_mixer_{mode}", lambda: ops.ssd_mixer(mproj, 0, HM, dv, 1, N, w, 1, 1e-5, S, conv, st), reps,
+                 bytes_=mproj.numel() * 2 + T * inner * 2 + 8 * n * HM * N * dv, flops=4 * T * HM * N * dv)
+            if mode == "prefill":
+                note("ssd_mixer_token_by_token_prefill",
+                     lambda: ops.ssd_mixer(mproj, 0, HM, dv, 1, N, w, 1, 1e-5, S, conv, st, chunked=False), reps,
+                     bytes_=mproj.numel() * 2 + T * inner * 2 + 8 * n * HM * N * dv, flops=4 * T * HM * N * dv)
+            R = max(H // 2, 1)
+            sproj = (torch.randn(T, 4 * R * d, device=dev) * 0.5).to(bf)
+            logits, zb, S2 = torch.randn(T, R * d, device=dev), torch.zeros(R * d, device=dev), torch.zeros(n + 1, R, d, d, device=dev)
+            note(f"like:state_attention_{mode}",
+                 lambda: ops.state_attention(sproj, 0, R * d, 2 * R * d, 3 * R * d, R, d, d, S2, st, 1e-5, decay_logits=logits,
+                                             decay_bias=zb, tau=16.0), reps,
+                 bytes_=sproj.numel() * 2 + T * R * d * 6 + 8 * n * R * d * d, flops=4 * T * R * d * d)
+            del mproj, sproj, S, S2, logits
+            # normed projections into the cache with values mixed, and windowed attention with kept tokens and a gate
+            pages = -(-st.max_seq_len // page)
+            table = torch.arange(n * pages, dtype=torch.int32, device=dev).view(n, pages)
+            slots = torch.cat([table[i].long()[(st.positions[st.cu_seqlens[i]: st.cu_seqlens[i + 1]] // page).long()] * page
+                               + st.positions[st.cu_seqlens[i]: st.cu_seqlens[i + 1]].long() % page for i in range(n)])
+            cache = (torch.randn(n * pages, 2, G, page, d, device=dev) * 0.3).to(bf)
+            kv = KVView(cache, table, slots, page, W, True, KVSpec(((G, d), (G, d)), W, keep_first=keep))
+            like_kv = KVView(cache, table, slots, page, W, True, KVSpec(((G, d), (G, d)), W))
+            cols = (2 * H + 2 * G) * d
+            proj, other = ((torch.randn(T, cols, device=dev) * 0.5).to(bf) for _ in range(2))
+            nw = torch.ones(d, device=dev)
+            moved = T * (H + 2 * G) * d * 4
+            note(f"qkv_prepare_mixed_{mode}",
+                 lambda: ops.qkv_prepare(proj, 0, H * d, (H + G) * d, H, d, None, nw, nw, 1e-5, None, st.positions, kv, True,
+                                         mix=(other, (H + G) * d, 0.4)), 20, bytes_=moved + T * G * d * 2)
+            inv = torch.tensor([100000.0 ** (-4.0 * i / d) for i in range(d // 4)], device=dev)
+            note(f"like:qkv_prepare_{mode}",
+                 lambda: ops.qkv_prepare(proj, 0, H * d, (H + G) * d, H, d, None, None, None, None, inv, st.positions, like_kv, True),
+                 20, bytes_=moved)
+            q = (torch.randn(T, H, d, device=dev) * 0.3).to(bf)
+            spans = [(s + i + 1, min(s + i + 1, W)) for s, count in zip(starts, lens) for i in range(count)]
+            seen = sum(near for _, near in spans)
+            kept = sum(min(all_, W + keep) for all_, _ in spans)
+            held = sum(min(s + count, W + keep) if mode == "decode" else s + count for s, count in zip(starts, lens))
+            io = 6 * T * H * d
+            note(f"window_keep_attention_{mode}", lambda: ops.paged_attention(q, kv, st, 0.1, gate=proj, gate_col=(H + 2 * G) * d), reps,
+                 bytes_=held * 2 * G * d * 2 + io, flops=4 * kept * H * d)
+            note(f"like:window_attention_{mode}", lambda: ops.paged_attention(q, like_kv, st, 0.1, gate=proj, gate_col=(H + 2 * G) * d), reps,
+                 bytes_=held * 2 * G * d * 2 + io, flops=4 * seen * H * d)
+            del q, proj, other, cache
+            # the latent's end: values out of latent space and the gate on every value, beside the values alone
+            rank = 4 * d
+            o_lat, uv = (torch.randn(H, T, rank, device=dev) * 0.1).to(bf), (torch.randn(H, rank, d, device=dev) * 0.1).to(bf)
+            vals, gate = torch.empty(T, H, d, dtype=bf, device=dev), torch.randn(T, H * d, device=dev).to(bf)
+            work = dict(bytes_=o_lat.numel() * 2 + uv.numel() * 2 + vals.numel() * 2, flops=2 * T * H * rank * d)
+            note(f"latent_values_gated_{mode}", lambda: ops.latent_values(o_lat, uv, vals, gate), 10,
+                 **{**work, "bytes_": work["bytes_"] + gate.numel() * 2})
+            note(f"like:latent_values_{mode}", lambda: ops.batched_mm(o_lat, uv, out=vals.transpose(0, 1)), 10, **work)
+            del o_lat, gate, vals
+            # ungated experts with the shared one's gate, beside gated ones chosen within groups
+            h = (torch.randn(T, D, device=dev) * 0.5).to(bf)
+            egu = (torch.randn(E, 2 * F, D, device=dev) * D ** -0.5).to(bf)
+            eup, edn = egu[:, :F].contiguous(), (torch.randn(E, D, F, device=dev) * F ** -0.5).to(bf)
+            router, bias, correction = torch.randn(E + 1, D, device=dev) * 0.05, torch.zeros(E, device=dev), torch.zeros(E, device=dev)
+            shared = torch.randn(T, D, device=dev).to(bf)
+            used = E * (1.0 - (1.0 - top / E) ** T)
+            note(f"ungated_experts_{mode}",
+                 lambda: ops.moe_experts(h, router, None, eup, edn, top, st, scoring="chosen", bias=bias, activation="gelu_erf",
+                                         extra=shared, shared_gated=True), 5,
+                 bytes_=used * 2 * F * D * 2 + T * D * 6, flops=2 * T * top * 2 * F * D)
+            note(f"like:group_limited_experts_{mode}",
+                 lambda: ops.moe_experts(h, router[:E], correction, egu, edn, top, st, scoring="sigmoid", groups=4, keep_groups=2,
+                                         normalise=True, weight_scale=1.5, combine=False), 5,
+                 bytes_=used * 3 * F * D * 2 + T * D * 4, flops=2 * T * top * 3 * F * D)
+            del egu, eup, edn
+            # the dense unit's first product
+            gu = (torch.randn(4 * D, D, device=dev) * D ** -0.5).to(bf)
+            dense = dict(bytes_=gu.numel() * 2 + T * D * 6, flops=2 * T * gu.numel())
+            note(f"gelu_glu_{mode}", lambda: ops.linear_glu(h, gu, "gelu_tanh"), 10, **dense)
+            note(f"like:swiglu_{mode}", lambda: ops.linear_swiglu(h, gu), 10, **dense)
+            del gu
+        ops.raise_on_error(dev)
+        return out
+
+    record = {"metric": "Gisudra beside Rinirax at equal sizes", "unit": "tokens/s", "dtype": "bf16",
+              "data": "synthetic: seeded uniform-random token ids, random weights",
+              "config": {"prefill_tokens": tokens, "decode_batch": batch, "decode_context": context, "vocab": DOLUTAR_VOCAB,
+                         "peaks": peak_source}, "sizes": {}}
+    for name in ([args.size] if args.size else list(BOBARAX_SIZES)):
+        size = BOBARAX_SIZES[name]
+        record["sizes"][name] = {"gisudra": whole_model_ms(gisudra_config(size), args, DOLUTAR_VOCAB, g),
+                                 "rinirax": whole_model_ms(rinirax_config(size), args, DOLUTAR_VOCAB, g),
+                                 "kernels": kernels(size), "layers": size["layers"]}
+    return record
+
+
 def main() -> int:
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
@@ -1808,7 +1967,7 @@ def main() -> int:
                         help="with --only decode|prefill and OMNIA_TIMELINE=1 in the environment: one step's "
                              "kernels with the time each takes in the stream, on stderr")
     parser.add_argument("--only", choices=["all", "decode", "prefill", "mixed", "portions", "sampling", "products", "elementwise", "fokalorn",
-                                           "dolutar", "bobarax", "narezen", "rinirax"], default="all",
+                                           "dolutar", "bobarax", "narezen", "rinirax", "gisudra"], default="all",
                         help="time one part only (small cases for profilers); prints a short record")
     parser.add_argument("--config", type=int, choices=sorted(CONFIGS), default=2,
                         help="with --only: the sizes of another benchmark configuration (3: 36 layers, hidden 4096, "
@@ -1820,7 +1979,7 @@ def main() -> int:
     parser.add_argument("--portion", type=int, default=256,
                         help="--only mixed: tokens of a prompt that run beside --batch decoding requests")
     parser.add_argument("--size", choices=sorted(FOKALORN_SIZES), default=None,
-                        help="--only fokalorn, dolutar, bobarax, narezen or rinirax: one size instead of all")
+                        help="--only fokalorn, dolutar, bobarax, narezen, rinirax or gisudra: one size instead of all")
     args = parser.parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable":
@@ -1845,6 +2004,9 @@ def main() -> int:
         return 0
     if args.only == "rinirax":
         print(json.dumps(run_rinirax(args)))
+        return 0
+    if args.only == "gisudra":
+        print(json.dumps(run_gisudra(args)))
         return 0
     if args.only == "dolutar":
         print(json.dumps(run_dolutar(args)))

@@ -1827,6 +1827,15 @@ def batched_mm(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None
     return torch.bmm(a, b) if out is None else torch.bmm(a, b, out=out)
 
 
+def latent_values(o_lat: torch.Tensor, uv: torch.Tensor, out: torch.Tensor, gate: torch.Tensor | None = None) -> torch.Tensor:
+    """Attention outputs out of latent space: out[t, h] = o_lat[h, t] @ uv[h], with `gate` (columns of projected rows,
+    [tokens, heads * vdim]) times sigmoid(gate), element by element. o_lat [heads, tokens, rank], uv [heads, rank,
+    vdim], out [tokens, heads, vdim]. -> out as [tokens, heads * vdim]"""
+    batched_mm(o_lat, uv, out=out.transpose(0, 1))
+    rows = out.view(out.shape[0], -1)
+    return rows if gate is None else gate_rows(rows, gate)
+
+
 # ------------------------------------------------------------------------------------
 # Routed experts (csrc/moe.cu)
 

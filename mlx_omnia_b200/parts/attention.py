@@ -223,11 +223,8 @@ class LatentAttention(Mixer):
         ops.latent_attention(q_lat, q[:, :, self.dim:], ctx.kv, step, self.scale, self.sink_logits,
                              proj[:, self.gate_col:] if self.gated is True else None, o_lat)
         out = torch.empty(tokens, H, self.vdim, dtype=proj.dtype, device=proj.device)
-        ops.batched_mm(o_lat, self.uv_t, out=out.transpose(0, 1))
-        out = out.view(tokens, H * self.vdim)
-        if self.gated == "values":
-            ops.gate_rows(out, proj[:, self.gate_col: self.gate_col + H * self.vdim])
-        return ops.linear(out, self.o)
+        gate = proj[:, self.gate_col: self.gate_col + H * self.vdim] if self.gated == "values" else None
+        return ops.linear(ops.latent_values(o_lat, self.uv_t, out, gate), self.o)
 
 
 @register_mixer("sink_window_attention")
