@@ -12,13 +12,21 @@
 //
 //   inputs   a thread walks a channel (or a head's dt) over a run of tokens with the taps' window in registers,
 //            so every projected value is read once. Out: float32 rows [C | B | x | (a, dt) a head] for the token-by-
-//            token recurrence (state_recurrence.cu), or for the chunked one (ssd_chunk.cu) rows [x | B | C] in the
-//            element type beside float32 pairs (log a, dt).
+//            token recurrence (state_recurrence.cu), or for the chunked one (ssd_chunk.cu) float16 rows
+//            [x | B | C] beside float32 pairs (log a, dt).
 //   step     a step in which every request brings one token: convolution, step sizes and recurrence in one
 //            kernel, a block per (request, head, run of columns).
 //   out      per token: the skip's y times silu(z), norm and weight, rounded once; and, after the last token,
 //            per request: the convolution's carried inputs moved on.
 #include "common.cuh"
+
+#include <cuda_fp16.h>
+
+// float16 holds the convolution's outputs for the chunked recurrence; what is beyond its range is held at its end.
+template <>
+__device__ __forceinline__ __half from_f32<__half>(float v) {
+  return __float2half_rn(v > 65504.f ? 65504.f : v < -65504.f ? -65504.f : v);
+}
 
 namespace {
 
@@ -143,6 +151,24 @@ ssd_step_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, int c
   float* part = x_s + ((cols + 3) & ~3);        // [teams][mine]
   const T* row = proj + (size_t)t * stride + col0;
   const int slot = state_slots[seq];
+  float* S = S_state + ((size_t)slot * s.H + head) * N * s.dv + j0;
+  const int runs = mine / VEC, teams = max(1, (int)blockDim.x / max(runs, 1));
+  // The first rows of S are asked for ahead of everything else: they come from memory, the rest is arithmetic.
+  constexpr int AHEAD = 8;
+  float ahead[AHEAD][VEC];
+  if ((int)threadIdx.x < teams * runs) {
+    const float* at = S + (size_t)(threadIdx.x / runs) * s.dv + (threadIdx.x % runs) * VEC;
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i)
+      if ((int)threadIdx.x / runs + i * teams < N) {
+        if constexpr (VEC == 4) {
+          const float4 v = *reinterpret_cast<const float4*>(at + (size_t)i * teams * s.dv);
+          ahead[i][0] = v.x, ahead[i][1] = v.y, ahead[i][2] = v.z, ahead[i][3] = v.w;
+        } else {
+          ahead[i][0] = at[(size_t)i * teams * s.dv];
+        }
+      }
+  }
   const float* held = conv_state + (size_t)slot * max(K - 1, 1) * C;
   for (int i = threadIdx.x; i < 2 * N + mine; i += blockDim.x) {
     const int c = i < N ? inner + group * N + i : i < 2 * N ? inner + gn + group * N + (i - N) : head * s.dv + j0 + (i - 2 * N);
@@ -154,29 +180,36 @@ ssd_step_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, int c
   const float dt = softplus(to_f32(row[inner + C + head]) + dt_bias[head]);
   const float a = expf(-expf(A_log[head]) * dt);
   __syncthreads();
-  float* S = S_state + ((size_t)slot * s.H + head) * N * s.dv + j0;
-  const int runs = mine / VEC, teams = max(1, (int)blockDim.x / max(runs, 1));
   for (int item = threadIdx.x; item < teams * runs; item += blockDim.x) {
     const int m = item / runs, j = (item % runs) * VEC;
     float sum[VEC], v[VEC];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) sum[e] = 0.f, v[e] = dt * x_s[j + e];
-#pragma unroll 8
-    for (int r = m; r < N; r += teams) {
-      float* at = S + (size_t)r * s.dv + j;
+    auto move_on = [&](int r, float* st) {
       const float b = b_s[r], c = c_s[r];
+      float* at = S + (size_t)r * s.dv + j;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) st[e] = fmaf(b, v[e], a * st[e]), sum[e] = fmaf(st[e], c, sum[e]);
+      if constexpr (VEC == 4) *reinterpret_cast<float4*>(at) = make_float4(st[0], st[1], st[2], st[3]);
+      else at[0] = st[0];
+    };
+    int r = m;
+    if (item == (int)threadIdx.x) {
+#pragma unroll
+      for (int i = 0; i < AHEAD; ++i, r += teams)
+        if (r < N) move_on(r, ahead[i]);
+    }
+#pragma unroll 8
+    for (; r < N; r += teams) {
+      const float* at = S + (size_t)r * s.dv + j;
+      float st[VEC];
       if constexpr (VEC == 4) {
-        float4 st = *reinterpret_cast<const float4*>(at);
-        st.x = fmaf(b, v[0], a * st.x), st.y = fmaf(b, v[1], a * st.y);
-        st.z = fmaf(b, v[2], a * st.z), st.w = fmaf(b, v[3], a * st.w);
-        *reinterpret_cast<float4*>(at) = st;
-        sum[0] = fmaf(st.x, c, sum[0]), sum[1] = fmaf(st.y, c, sum[1]);
-        sum[2] = fmaf(st.z, c, sum[2]), sum[3] = fmaf(st.w, c, sum[3]);
+        const float4 q = *reinterpret_cast<const float4*>(at);
+        st[0] = q.x, st[1] = q.y, st[2] = q.z, st[3] = q.w;
       } else {
-        const float st = fmaf(b, v[0], a * at[0]);
-        at[0] = st;
-        sum[0] = fmaf(st, c, sum[0]);
+        st[0] = at[0];
       }
+      move_on(r, st);
     }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) part[m * mine + j + e] = sum[e];
@@ -266,8 +299,7 @@ bool sizes_ok(const Sizes& s, int K) {
 
 }  // namespace
 
-// wide_rows != 0: float32 rows (whatever the element type) and (a, dt) pairs; else rows in the element type and
-// (log a, dt) pairs. Places and strides in elements of what they index; pairs must start on 8 bytes in every row.
+// wide_rows != 0: float32 rows and (a, dt) pairs; else float16 rows and (log a, dt) pairs. Places and strides in elements of what they index; pairs must start on 8 bytes in every row.
 extern "C" int omnia_ssd_inputs(const void* proj, int stride, int col0, int H, int dv, int G, int N, const float* taps,
                                 const float* conv_bias, int K, const float* conv_state, const float* dt_bias,
                                 const float* A_log, const int* cu_seqlens, const int* state_slots, int num_seqs, int tokens,
@@ -280,7 +312,7 @@ extern "C" int omnia_ssd_inputs(const void* proj, int stride, int col0, int H, i
     if (wide_rows)
       return launch_inputs<T, float>(proj, stride, col0, s, taps, conv_bias, K, conv_state, dt_bias, A_log, cu_seqlens,
                                      state_slots, num_seqs, tokens, rows, row_stride, at_x, at_b, at_c, pairs, pair_stride, 0, stream);
-    return launch_inputs<T, T>(proj, stride, col0, s, taps, conv_bias, K, conv_state, dt_bias, A_log, cu_seqlens, state_slots,
+    return launch_inputs<T, __half>(proj, stride, col0, s, taps, conv_bias, K, conv_state, dt_bias, A_log, cu_seqlens, state_slots,
                                num_seqs, tokens, rows, row_stride, at_x, at_b, at_c, pairs, pair_stride, 1, stream);
   });
   return (int)cudaErrorInvalidValue;

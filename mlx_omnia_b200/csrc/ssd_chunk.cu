@@ -5,19 +5,22 @@
 //   S  <- e^(l_last) S + sum_s e^(l_last - l_s) dt_s B_s x_s^T
 //
 // Four products a chunk: C B^T, its weighted lower triangle times x, C S, and B^T times the weighted x. B, C and x
-// are bfloat16 as the convolution's output is rounded; everything that float32 makes (the weighted triangle, the
-// weighted x, the state as an operand) is split into the sum of two bfloat16 numbers, so it enters its product with
-// 16 bits of mantissa, and the sums, the decays and the carried state are float32. All exponents are of differences
+// are float16 (three bits more than bfloat16 would keep of what the convolution makes in float32; their size needs
+// no wider exponent); everything else that enters a product (the weighted triangle, the weighted x, the state) is
+// split into the sum of two float16 numbers, 22 bits of mantissa, the state and the triangle after a scaling by a
+// power of two that keeps their largest entries in range. Sums, decays and the carried state are float32. All exponents are of differences
 // that are at most zero.
 //
 // A block owns SSD_COLS value columns of one head of one request and walks its chunks in order; a column of S needs
 // no other column. Warp w has 16 of the chunk's tokens for the first three products (the tokens dealt so that the two
 // warps of a scheduler have equal shares of the triangle) and 16 of the state's rows for the last, whose float32
-// values never leave its registers; the other warps read them as pairs of bfloat16 from shared memory. The next
+// values never leave its registers; the other warps read them as pairs of float16 from shared memory. The next
 // chunk's B, C, x and step sizes come in by asynchronous copies meanwhile.
 //
 // Compiled per state size and columns: -DSSD_N=<N> (a multiple of 16), -DSSD_COLS=<16 or 32>.
 #include "common.cuh"
+
+#include <cuda_fp16.h>
 
 #ifndef SSD_N
 #define SSD_N 128
@@ -28,15 +31,15 @@
 
 namespace {
 
-typedef __nv_bfloat16 bf16;
+typedef __half f16;
 
 constexpr int N = SSD_N, COLS = SSD_COLS;
 static_assert(N % 16 == 0 && (COLS == 16 || COLS == 32), "sizes the tensor cores' tiles fit");
 constexpr int NROW = N + 8, XROW = COLS + 8;  // rows of shared memory in elements: an odd number of 16-byte pieces
 
 constexpr size_t smem_bytes(int L) {
-  return sizeof(bf16) * (2 * (size_t)L * (2 * NROW + XROW) + 2 * N * XROW + 2 * L * XROW) + 2 * sizeof(float2) * L +
-         3 * sizeof(float) * L;
+  return sizeof(f16) * (2 * (size_t)L * (2 * NROW + XROW) + 2 * N * XROW + 2 * L * XROW) + 2 * sizeof(float2) * L +
+         3 * sizeof(float) * L + sizeof(float) * 8;
 }
 constexpr int L = N <= 128 && smem_bytes(128) <= 227 * 1024 ? 128 : 64;
 static_assert(smem_bytes(L) <= 227 * 1024, "a chunk fits shared memory");
@@ -58,26 +61,28 @@ __device__ __forceinline__ void copy8(const void* smem, const void* gmem, bool v
   asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;\n" ::"r"(shared_address(smem)), "l"(gmem), "r"(valid ? 8 : 0)
                : "memory");
 }
-__device__ __forceinline__ void ldmatrix(uint32_t* r, const bf16* p) {
+__device__ __forceinline__ void ldmatrix(uint32_t* r, const f16* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(shared_address(p)) : "memory");
 }
-__device__ __forceinline__ void ldmatrix_t(uint32_t* r, const bf16* p) {
+__device__ __forceinline__ void ldmatrix_t(uint32_t* r, const f16* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(shared_address(p)) : "memory");
 }
 __device__ __forceinline__ void mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
   asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+      "mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-// (u, v) as two pairs of bfloat16 whose sum has 16 bits of mantissa.
+// (u, v) as two pairs of float16 whose sum has 22 bits of mantissa (numbers beyond float16's range are held at its end).
 __device__ __forceinline__ void split(float u, float v, uint32_t& hi, uint32_t& lo) {
-  __nv_bfloat162 h = __floats2bfloat162_rn(u, v);
-  __nv_bfloat162 l = __floats2bfloat162_rn(u - __low2float(h), v - __high2float(h));
-  hi = *reinterpret_cast<uint32_t*>(&h);
-  lo = *reinterpret_cast<uint32_t*>(&l);
+  u = u > 65504.f ? 65504.f : u < -65504.f ? -65504.f : u;
+  v = v > 65504.f ? 65504.f : v < -65504.f ? -65504.f : v;
+  const __half2 h = __floats2half2_rn(u, v);
+  const __half2 l = __floats2half2_rn(u - __low2float(h), v - __high2float(h));
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 __device__ __forceinline__ float power_of_two(float v) {
   float r;
@@ -87,30 +92,31 @@ __device__ __forceinline__ float power_of_two(float v) {
 
 // rows: bfloat16 [tokens, row_stride], x, B and C at their places; pairs: (log a, dt) [tokens, H]; y: float32 [tokens, H * dv].
 __global__ void __launch_bounds__(THREADS, 1)
-ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at_b, int at_c, const float2* __restrict__ pairs,
+ssd_chunk_kernel(const f16* __restrict__ rows, int row_stride, int at_x, int at_b, int at_c, const float2* __restrict__ pairs,
                  int H, int G, int dv, const float* __restrict__ D, float* __restrict__ S_state,
                  const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, float* __restrict__ y) {
   pdl_wait();
   pdl_launch_dependents();
   extern __shared__ __align__(16) unsigned char chunk_smem[];
-  bf16* Bs[2], *Cs[2], *Xs[2];
+  f16* Bs[2], *Cs[2], *Xs[2];
   float2* ps[2];
-  bf16* at = reinterpret_cast<bf16*>(chunk_smem);
+  f16* at = reinterpret_cast<f16*>(chunk_smem);
 #pragma unroll
   for (int b = 0; b < 2; ++b) {
     Bs[b] = at, at += L * NROW;
     Cs[b] = at, at += L * NROW;
     Xs[b] = at, at += L * XROW;
   }
-  bf16* Sh = at;               // [N][XROW] the state's upper halves, then the lower ones
-  bf16* Sl = Sh + N * XROW;
-  bf16* Wh = Sl + N * XROW;    // [L][XROW] the weighted x
-  bf16* Wl = Wh + L * XROW;
+  f16* Sh = at;               // [N][XROW] the state's upper halves, then the lower ones
+  f16* Sl = Sh + N * XROW;
+  f16* Wh = Sl + N * XROW;    // [L][XROW] the weighted x
+  f16* Wl = Wh + L * XROW;
   ps[0] = reinterpret_cast<float2*>(Wl + L * XROW);
   ps[1] = ps[0] + L;
   float* cum = reinterpret_cast<float*>(ps[1] + L);  // running sum of log2 a
   float* dts = cum + L;
   float* wgt = dts + L;                              // what a token's x is weighted with on its way into the state
+  float* peaks = wgt + L;                            // each warp's largest entry of the state
 
   const int parts = dv / COLS, head = blockIdx.x / parts, col0 = (blockIdx.x % parts) * COLS, seq = blockIdx.y;
   const int begin = cu_seqlens[seq], end = cu_seqlens[seq + 1];
@@ -118,9 +124,9 @@ ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at
   const int group = head / (H / G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t4 = lane & 3, mat = lane >> 3, r8 = lane & 7;
   const float skip = D[head];
-  const bf16* b_rows = rows + at_b + group * N;
-  const bf16* c_rows = rows + at_c + group * N;
-  const bf16* x_rows = rows + at_x + head * dv + col0;
+  const f16* b_rows = rows + at_b + group * N;
+  const f16* c_rows = rows + at_c + group * N;
+  const f16* x_rows = rows + at_x + head * dv + col0;
 
   auto fetch = [&](int t0, int n, int b) {
     const int fill = min(L, (n + 31) & ~31);  // rows past the portion's end are zeros, up to a whole block of keys
@@ -147,12 +153,24 @@ ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at
 #pragma unroll
     for (int nt = 0; nt < NTW; ++nt)
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
+      for (int side = 0; side < 2; ++side) {
         float2 v = make_float2(0.f, 0.f);
-        if (m0 + m < MT) v = *reinterpret_cast<const float2*>(mine + (size_t)((m0 + m) * 16 + g + 8 * half) * dv + nt * 8);
-        S[m][nt][2 * half] = v.x, S[m][nt][2 * half + 1] = v.y;
+        if (m0 + m < MT) v = *reinterpret_cast<const float2*>(mine + (size_t)((m0 + m) * 16 + g + 8 * side) * dv + nt * 8);
+        S[m][nt][2 * side] = v.x, S[m][nt][2 * side + 1] = v.y;
       }
 
+  auto note_peak = [&]() {
+    float peak = 0.f;
+#pragma unroll
+    for (int m = 0; m < MPW; ++m)
+#pragma unroll
+      for (int nt = 0; nt < NTW; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) peak = fmaxf(peak, fabsf(S[m][nt][e]));
+    peak = warp_max(peak);
+    if (lane == 0) peaks[warp] = peak;
+  };
+  note_peak();
   const int tile = WARPS == 8 && warp >= 4 ? 11 - warp : warp, row0 = tile * 16;
   const int chunks = (end - begin + L - 1) / L;
   fetch(begin, min(L, end - begin), 0);
@@ -161,17 +179,23 @@ ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at
     asm volatile("cp.async.wait_group 0;\n" ::: "memory");
     __syncthreads();  // the chunk has arrived, and everybody is done with the last one
     if (c + 1 < chunks) fetch(t0 + L, min(L, end - t0 - L), b ^ 1);
-    const bf16 *Bc = Bs[b], *Cc = Cs[b], *Xc = Xs[b];
+    const f16 *Bc = Bs[b], *Cc = Cs[b], *Xc = Xs[b];
+    // A state beyond 2^15 goes down by a power of two on its way into the product, whose result goes up by it.
+    float peak = peaks[0];
+#pragma unroll
+    for (int i = 1; i < WARPS; ++i) peak = fmaxf(peak, peaks[i]);
+    const int shift = max((int)(__float_as_uint(peak) >> 23) - 127 - 14, 0);
+    const float down = __uint_as_float((uint32_t)(127 - shift) << 23), up = __uint_as_float((uint32_t)(127 + shift) << 23);
 #pragma unroll
     for (int m = 0; m < MPW; ++m)
       if (m0 + m < MT)
 #pragma unroll
         for (int nt = 0; nt < NTW; ++nt)
 #pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            const int place = ((m0 + m) * 16 + g + 8 * half) * XROW + c0 + nt * 8 + 2 * t4;
+          for (int side = 0; side < 2; ++side) {
+            const int place = ((m0 + m) * 16 + g + 8 * side) * XROW + c0 + nt * 8 + 2 * t4;
             uint32_t hi, lo;
-            split(S[m][nt][2 * half], S[m][nt][2 * half + 1], hi, lo);
+            split(S[m][nt][2 * side] * down, S[m][nt][2 * side + 1] * down, hi, lo);
             *reinterpret_cast<uint32_t*>(Sh + place) = hi;
             *reinterpret_cast<uint32_t*>(Sl + place) = lo;
           }
@@ -206,7 +230,7 @@ ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at
     for (int i = tid; i < key_rows * (COLS / 2); i += THREADS) {
       const int r = i / (COLS / 2), place = r * XROW + (i % (COLS / 2)) * 2;
       const float w = wgt[r];
-      const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(Xc + place);
+      const __half2 v = *reinterpret_cast<const __half2*>(Xc + place);
       uint32_t hi, lo;
       split(w * __low2float(v), w * __high2float(v), hi, lo);
       *reinterpret_cast<uint32_t*>(Wh + place) = hi;
@@ -233,7 +257,7 @@ ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at
           mma(acc[2 * pair + 1], cf[ks], lo[2], lo[3]);
         }
       const float cum_a = cum[row0 + g], cum_b = cum[row0 + g + 8];
-      const float ea = power_of_two(cum_a), eb = power_of_two(cum_b);
+      const float ea = power_of_two(cum_a) * up, eb = power_of_two(cum_b) * up;
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) acc[nt][0] *= ea, acc[nt][1] *= ea, acc[nt][2] *= eb, acc[nt][3] *= eb;
       // The keys in blocks of 32, up to this warp's last token.
@@ -261,6 +285,28 @@ ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at
             p[j][e] *= key <= row0 + g ? power_of_two(cum_a - ck) * dk : 0.f;
             p[j][2 + e] *= key <= row0 + g + 8 ? power_of_two(cum_b - ck) * dk : 0.f;
           }
+        // Weights beyond 2^15 (a whole warp's matter, and a rare one): they and the sums so far go down by a power of
+        // two, and the sums come up again.
+        float most = 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) most = fmaxf(most, fabsf(p[j][e]));
+        const bool wide = __any_sync(0xffffffffu, most > 32768.f);
+        float raise = 1.f;
+        if (wide) {
+          const int places = max((int)(__float_as_uint(warp_max(most)) >> 23) - 127 - 14, 0);
+          const float lower = __uint_as_float((uint32_t)(127 - places) << 23);
+          raise = __uint_as_float((uint32_t)(127 + places) << 23);
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) p[j][e] *= lower;
+#pragma unroll
+          for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[nt][e] *= lower;
+        }
 #pragma unroll
         for (int kk = 0; kk < 2; ++kk) {
           uint32_t hi[4], lo[4];
@@ -278,17 +324,22 @@ ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at
             mma(acc[2 * pair + 1], lo, xv[2], xv[3]);
           }
         }
+        if (wide)
+#pragma unroll
+          for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[nt][e] *= raise;
       }
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int r = row0 + g + 8 * half;
+      for (int side = 0; side < 2; ++side) {
+        const int r = row0 + g + 8 * side;
         if (r >= n) continue;
         float* out = y + (size_t)(t0 + r) * H * dv + head * dv + col0 + 2 * t4;
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
-          const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(Xc + r * XROW + nt * 8 + 2 * t4);
-          *reinterpret_cast<float2*>(out + nt * 8) = make_float2(fmaf(skip, __low2float(v), acc[nt][2 * half]),
-                                                                 fmaf(skip, __high2float(v), acc[nt][2 * half + 1]));
+          const __half2 v = *reinterpret_cast<const __half2*>(Xc + r * XROW + nt * 8 + 2 * t4);
+          *reinterpret_cast<float2*>(out + nt * 8) = make_float2(fmaf(skip, __low2float(v), acc[nt][2 * side]),
+                                                                 fmaf(skip, __high2float(v), acc[nt][2 * side + 1]));
         }
       }
     }
@@ -308,8 +359,8 @@ ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at
         if constexpr (NTW == 1) {
           // One tile of eight columns: its upper and lower halves in one load.
           uint32_t w[4];
-          const bf16* half = (mat >> 1) ? Wl : Wh;
-          ldmatrix_t(w, half + (ks * 16 + (mat & 1) * 8 + r8) * XROW + c0);
+          const f16* part = (mat >> 1) ? Wl : Wh;
+          ldmatrix_t(w, part + (ks * 16 + (mat & 1) * 8 + r8) * XROW + c0);
           mma(S[m][0], bt, w[0], w[1]);
           mma(S[m][0], bt, w[2], w[3]);
         } else {
@@ -327,6 +378,7 @@ ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at
         }
       }
     }
+    note_peak();
   }
 #pragma unroll
   for (int m = 0; m < MPW; ++m)
@@ -334,9 +386,9 @@ ssd_chunk_kernel(const bf16* __restrict__ rows, int row_stride, int at_x, int at
 #pragma unroll
       for (int nt = 0; nt < NTW; ++nt)
 #pragma unroll
-        for (int half = 0; half < 2; ++half)
-          *reinterpret_cast<float2*>(mine + (size_t)((m0 + m) * 16 + g + 8 * half) * dv + nt * 8) =
-              make_float2(S[m][nt][2 * half], S[m][nt][2 * half + 1]);
+        for (int side = 0; side < 2; ++side)
+          *reinterpret_cast<float2*>(mine + (size_t)((m0 + m) * 16 + g + 8 * side) * dv + nt * 8) =
+              make_float2(S[m][nt][2 * side], S[m][nt][2 * side + 1]);
 }
 
 }  // namespace
@@ -358,7 +410,7 @@ extern "C" int omnia_ssd_chunk(const void* rows, int row_stride, int at_x, int a
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  launch_pdl(ssd_chunk_kernel, dim3(H * (dv / COLS), num_seqs), dim3(THREADS), smem_bytes(L), stream, (const bf16*)rows,
+  launch_pdl(ssd_chunk_kernel, dim3(H * (dv / COLS), num_seqs), dim3(THREADS), smem_bytes(L), stream, (const f16*)rows,
              row_stride, at_x, at_b, at_c, (const float2*)pairs, H, G, dv, D, S_state, cu_seqlens, state_slots, y);
   return OMNIA_LAUNCH_RESULT();
 }

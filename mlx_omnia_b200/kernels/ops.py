@@ -1570,7 +1570,7 @@ def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N
     S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T, y_t = S_t^T C_t + D x_t per head (its B and C those of its
     group of neighbouring heads), then RMS norm of y silu(z) over `norm_groups` equal runs, with weight.
     The recurrence runs in float32 token by token, or (`chunked` None: where it applies) in chunks on the tensor
-    cores from x, B and C rounded to bfloat16, everything else of it in float32 or as sums of two bfloat16
+    cores from x, B and C rounded to float16, everything else of it in float32 or as sums of two float16
     numbers; a step of single tokens is one kernel. -> [tokens, heads * dv] in proj's type"""
     tokens, stride = proj.shape
     inner, channels, K = heads * dv, heads * dv + 2 * groups * N, w.taps.shape[1]
@@ -1587,7 +1587,7 @@ def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N
         _check(fn(_ptr(proj), stride, col0, heads, dv, groups, N, step_cols, _ptr(w.taps), _ptr(w.conv_bias), K, _ptr(conv_state),
                   _ptr(w.dt_bias), _ptr(w.A_log), _ptr(w.D), _ptr(S), *where, _ptr(y), code, _stream()), "ssd_step")
     elif chunked is not False and (cols := ssd_chunk_columns(step.num_seqs, heads, dv, N, proj.dtype, sm_count(device))):
-        rows = torch.empty(tokens, channels, dtype=proj.dtype, device=device)
+        rows = torch.empty(tokens, channels, dtype=torch.float16, device=device)
         pairs = torch.empty(tokens, 2 * heads, dtype=torch.float32, device=device)
         at_b, at_c = inner, inner + groups * N
         _ssd_inputs(proj, col0, heads, dv, groups, N, w, conv_state, where, rows, channels, 0, at_b, at_c, pairs, 2 * heads, False)

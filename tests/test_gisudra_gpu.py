@@ -178,7 +178,7 @@ def ssd_plain(rows, w, H, dv, N, G, groups, eps):
 def test_the_chunked_recurrence_across_its_edges(H, dv, N, G):
     """Two requests in portions that end inside, at and just past chunks of 64 and 128 tokens, from slots that others
     used, decays from nearly none to a tenth a token. The plain recurrence on x, B and C rounded as the kernel's
-    operands are: the carried state must agree to what sums of two bfloat16 numbers hold, far inside one rounding."""
+    operands are: the carried state must agree to what sums of two float16 numbers hold, far inside one rounding."""
     g = torch.Generator().manual_seed(N + H)
     inner, C, K, eps = H * dv, H * dv + 2 * G * N, 3, 1e-6
     w = ops.SSDWeights(torch.randn(C, K, generator=g) * 0.6, 0.2 * torch.randn(C, generator=g), torch.randn(H, generator=g) - 2.0,
@@ -202,7 +202,7 @@ def test_the_chunked_recurrence_across_its_edges(H, dv, N, G):
         z, xbc, dt = torch.split(rows[r].to(F64), [inner, C, H], -1)
         xbc = plain.silu(plain.causal_conv(xbc, w.taps, w.conv_bias))
         dt = plain.softplus(dt + w.dt_bias.to(F64))
-        for values, state, out, tolerances in ((xbc.float().to(torch.bfloat16).to(F64), S, got, (1e-4, 6e-3)),
+        for values, state, out, tolerances in ((xbc.float().to(torch.float16).to(F64), S, got, (5e-5, 6e-3)),
                                                (xbc, exact[0], sequential, (2e-5, 6e-3))):
             x, B, Cc = torch.split(values, [inner, G * N, G * N], -1)
             T = len(values)
@@ -212,6 +212,25 @@ def test_the_chunked_recurrence_across_its_edges(H, dv, N, G):
             assert rel(torch.cat(out[r]), want) < tolerances[1], r
     assert float((S[[0, 2, 4]] - 3.0).abs().max()) == 0.0
     ops.raise_on_error(CUDA)
+
+
+def test_a_state_beyond_sixteen_bits_of_exponent():
+    """Inputs so large that the state passes float16's range by far: the chunked kernel scales it on its way into the
+    product, so its outputs agree with the token-by-token kernel's."""
+    T, H, dv, N, G, eps = 300, 2, 32, 16, 1, 1e-6
+    rows, w = ssd_rows(T, H, dv, N, G, 5)
+    rows[:, H * dv: -H] = rows[:, H * dv: -H].abs() * 120.0
+    rows = rows.to(torch.bfloat16).to(CUDA)
+    w = ops.SSDWeights(w.taps, w.conv_bias, w.dt_bias, torch.full((H,), -5.0), w.D, w.norm)
+    dev = ops.SSDWeights(*(t.to(CUDA) for t in (w.taps, w.conv_bias, w.dt_bias, w.A_log, w.D, w.norm)))
+    out, states = [], []
+    for chunked in (True, False):
+        S, conv = torch.zeros(1, H, N, dv, device=CUDA), torch.zeros(1, 1, H * dv + 2 * G * N, device=CUDA)
+        out.append(torch.cat([ops.ssd_mixer(rows[a:b], 0, H, dv, G, N, dev, 2, eps, S, conv, Batch([b - a], [a], [0]), chunked=chunked)
+                              for a, b in ((0, 150), (150, 300))]))
+        states.append(S)
+    assert float(states[1].abs().max()) > 2e5
+    assert rel(states[0], states[1]) < 1e-3 and rel(out[0], out[1]) < 8e-3
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
