@@ -53,9 +53,40 @@ struct Sizes {
   __host__ __device__ int channels() const { return H * dv + 2 * G * N; }
 };
 
-// grid (ceil((channels + H) / 128), ceil(tokens / RUN)), 128 threads. KT: taps held in registers (>= taps).
-// Places of x, B and C in an output row are at_x, at_b, at_c; the pairs' rows are pair_stride floats apart.
-template <typename T, typename O, int KT>
+// VC neighbouring elements as float32, or as O.
+template <int VC>
+__device__ __forceinline__ void load_vec(const float* p, float* v) {
+  if constexpr (VC == 2) {
+    const float2 q = *reinterpret_cast<const float2*>(p);
+    v[0] = q.x, v[1] = q.y;
+  } else {
+    v[0] = p[0];
+  }
+}
+template <int VC>
+__device__ __forceinline__ void load_vec(const __nv_bfloat16* p, float* v) {
+  if constexpr (VC == 2) {
+    const __nv_bfloat162 q = *reinterpret_cast<const __nv_bfloat162*>(p);
+    v[0] = __low2float(q), v[1] = __high2float(q);
+  } else {
+    v[0] = to_f32(p[0]);
+  }
+}
+template <int VC>
+__device__ __forceinline__ void store_vec(float* p, const float* v) {
+  if constexpr (VC == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+  else p[0] = v[0];
+}
+template <int VC>
+__device__ __forceinline__ void store_vec(__half* p, const float* v) {
+  if constexpr (VC == 2) *reinterpret_cast<__half2*>(p) = __halves2half2(from_f32<__half>(v[0]), from_f32<__half>(v[1]));
+  else p[0] = from_f32<__half>(v[0]);
+}
+
+// grid (ceil((channels / VC + H) / 128), ceil(tokens / RUN)), 128 threads. KT: taps held in registers (>= taps); VC:
+// channels a thread walks (2 where every width and place is even). Places of x, B and C in an output row are at_x,
+// at_b, at_c; the pairs' rows are pair_stride floats apart.
+template <typename T, typename O, int KT, int VC>
 __global__ void __launch_bounds__(128)
 ssd_inputs_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, const float* __restrict__ taps,
                   const float* __restrict__ conv_bias, int K, const float* __restrict__ conv_state,
@@ -65,12 +96,13 @@ ssd_inputs_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, con
   pdl_wait();
   pdl_launch_dependents();
   const int C = s.channels(), inner = s.inner(), gn = s.G * s.N;
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c >= C + s.H) return;
+  const int unit = blockIdx.x * blockDim.x + threadIdx.x;
+  if (unit >= C / VC + s.H) return;
   const int t0 = blockIdx.y * RUN, t1 = min(tokens, t0 + RUN);
-  if (c >= C) {
-    const int h = c - C;
+  if (unit >= C / VC) {
+    const int h = unit - C / VC;
     const float bias = dt_bias[h], rate = expf(A_log[h]);
+#pragma unroll 8
     for (int t = t0; t < t1; ++t) {
       const float dt = softplus(to_f32(proj[(size_t)t * stride + col0 + inner + C + h]) + bias);
       float2* pair = reinterpret_cast<float2*>(pairs + (size_t)t * pair_stride) + h;
@@ -78,15 +110,19 @@ ssd_inputs_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, con
     }
     return;
   }
+  const int c = unit * VC;
   // taps [C, K]: w[KT - 1] the current token's, zeros ahead of the first.
-  float w[KT], u[KT];
+  float w[KT][VC], u[KT][VC], bias[VC];
 #pragma unroll
-  for (int j = 0; j < KT; ++j) {
-    const int tap = j - (KT - K);
-    w[j] = tap >= 0 ? taps[(size_t)c * K + tap] : 0.f;
-    u[j] = 0.f;
+  for (int e = 0; e < VC; ++e) {
+    bias[e] = conv_bias[c + e];
+#pragma unroll
+    for (int j = 0; j < KT; ++j) {
+      const int tap = j - (KT - K);
+      w[j][e] = tap >= 0 ? taps[(size_t)(c + e) * K + tap] : 0.f;
+      u[j][e] = 0.f;
+    }
   }
-  const float bias = conv_bias[c];
   const T* column = proj + col0 + inner + c;
   O* out = rows + (c < inner ? at_x + c : c < inner + gn ? at_b + (c - inner) : at_c + (c - inner - gn));
   int seq = request_of(cu_seqlens, num_seqs, t0);
@@ -98,18 +134,40 @@ ssd_inputs_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, con
     for (int j = 0; j < KT - 1; ++j) {
       const int back = KT - 1 - j;  // how many tokens before t
       if (back > K - 1) {
-        u[j + 1] = 0.f;
+#pragma unroll
+        for (int e = 0; e < VC; ++e) u[j + 1][e] = 0.f;
         continue;
       }
       const int at = t - back;
-      u[j + 1] = at >= begin ? to_f32(column[(size_t)at * stride]) : held[(size_t)(K - 1 + at - begin) * C];
+      if (at >= begin) load_vec<VC>(column + (size_t)at * stride, u[j + 1]);
+      else load_vec<VC>(held + (size_t)(K - 1 + at - begin) * C, u[j + 1]);
     }
   };
+  // One token: u[1 .. KT - 1] are the inputs before it, oldest first.
+  auto token = [&](int t, const float* now) {
+    float y[VC];
+#pragma unroll
+    for (int e = 0; e < VC; ++e) {
+      y[e] = bias[e];
+#pragma unroll
+      for (int j = 0; j < KT - 1; ++j) u[j][e] = u[j + 1][e], y[e] = fmaf(w[j][e], u[j][e], y[e]);
+      u[KT - 1][e] = now[e];
+      y[e] = silu(fmaf(w[KT - 1][e], now[e], y[e]));
+    }
+    store_vec<VC>(out + (size_t)t * row_stride, y);
+  };
+  if (t1 - t0 == RUN && t1 <= end) {
+    // The whole run in one request: all its inputs asked for at once.
+    float now[RUN][VC];
+#pragma unroll
+    for (int i = 0; i < RUN; ++i) load_vec<VC>(column + (size_t)(t0 + i) * stride, now[i]);
+    window(t0);
+#pragma unroll
+    for (int i = 0; i < RUN; ++i) token(t0 + i, now[i]);
+    return;
+  }
   window(t0);
-  T next = column[(size_t)t0 * stride];
   for (int t = t0; t < t1; ++t) {
-    const float now = to_f32(next);
-    if (t + 1 < t1) next = column[(size_t)(t + 1) * stride];
     if (t >= end) {
       do {
         ++seq;
@@ -117,13 +175,9 @@ ssd_inputs_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, con
       } while (t >= end && seq + 1 < num_seqs);
       window(t);
     }
-    // u[1 .. KT - 1] are the inputs before this token, oldest first.
-    float y = bias;
-#pragma unroll
-    for (int j = 0; j < KT - 1; ++j) u[j] = u[j + 1], y = fmaf(w[j], u[j], y);
-    u[KT - 1] = now;
-    y = fmaf(w[KT - 1], now, y);
-    out[(size_t)t * row_stride] = from_f32<O>(silu(y));
+    float now[VC];
+    load_vec<VC>(column + (size_t)t * stride, now);
+    token(t, now);
   }
 }
 
@@ -222,9 +276,30 @@ ssd_step_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, int c
   }
 }
 
-// Blocks 0 .. tokens - 1: a token each; the others: a request's carried inputs each.
-template <typename T>
-__global__ void __launch_bounds__(256)
+constexpr int OUT_ITEMS = 4;  // runs of four channels a thread of the output step keeps in registers
+
+// Four neighbouring elements of the gate's columns as float32.
+__device__ __forceinline__ void load_four(const float* p, float* v) {
+  const float4 q = *reinterpret_cast<const float4*>(p);
+  v[0] = q.x, v[1] = q.y, v[2] = q.z, v[3] = q.w;
+}
+__device__ __forceinline__ void load_four(const __nv_bfloat16* p, float* v) {
+  const uint2 q = *reinterpret_cast<const uint2*>(p);
+  const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&q.x), b = *reinterpret_cast<const __nv_bfloat162*>(&q.y);
+  v[0] = __low2float(a), v[1] = __high2float(a), v[2] = __low2float(b), v[3] = __high2float(b);
+}
+__device__ __forceinline__ void store_four(float* p, const float* v) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void store_four(__nv_bfloat16* p, const float* v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
+// Blocks 0 .. tokens - 1: a token each; the others: blockDim channels of a request's carried inputs each.
+// WHOLE: one norm group, its channels in fours and in the threads' registers.
+template <typename T, bool WHOLE>
+__global__ void __launch_bounds__(1024)
 ssd_out_kernel(const float* __restrict__ y, const T* __restrict__ proj, int stride, int col0, Sizes s, int norm_groups,
                float eps, const float* __restrict__ norm_w, int K, float* __restrict__ conv_state,
                const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, int tokens, T* __restrict__ out) {
@@ -234,21 +309,53 @@ ssd_out_kernel(const float* __restrict__ y, const T* __restrict__ proj, int stri
   __shared__ float red[33];
   const int inner = s.inner(), C = s.channels();
   if ((int)blockIdx.x >= tokens) {
-    const int seq = blockIdx.x - tokens, begin = cu_seqlens[seq], n = cu_seqlens[seq + 1] - begin;
-    if (n <= 0 || K < 2) return;
-    float* held = conv_state + (size_t)state_slots[seq] * (K - 1) * C;
-    for (int c = threadIdx.x; c < C; c += blockDim.x)
-      // Place j of the new window is n tokens further on than place j of the old one; ascending, so that a
-      // place is read before it is written.
-      for (int j = 0; j < K - 1; ++j)
-        held[(size_t)j * C + c] = j + n < K - 1 ? held[(size_t)(j + n) * C + c]
-                                                : to_f32(proj[(size_t)(begin + j + n - (K - 1)) * stride + col0 + inner + c]);
+    const int blocks = (C + blockDim.x - 1) / blockDim.x, item = blockIdx.x - tokens;
+    const int seq = item / blocks, c = (item % blocks) * blockDim.x + threadIdx.x;
+    const int begin = cu_seqlens[seq], n = cu_seqlens[seq + 1] - begin;
+    if (n <= 0 || K < 2 || c >= C) return;
+    float* held = conv_state + (size_t)state_slots[seq] * (K - 1) * C + c;
+    // Place j of the new window is n tokens further on than place j of the old one.
+    float v[MAX_TAPS - 1];
+#pragma unroll
+    for (int j = 0; j < MAX_TAPS - 1; ++j)
+      if (j < K - 1)
+        v[j] = j + n < K - 1 ? held[(size_t)(j + n) * C] : to_f32(proj[(size_t)(begin + j + n - (K - 1)) * stride + col0 + inner + c]);
+#pragma unroll
+    for (int j = 0; j < MAX_TAPS - 1; ++j)
+      if (j < K - 1) held[(size_t)j * C] = v[j];
     return;
   }
   const size_t t = blockIdx.x;
   const float* yt = y + t * inner;
   const T* z = proj + t * stride + col0;
   const int run = inner / norm_groups;
+  if constexpr (WHOLE) {
+    float v[OUT_ITEMS][4], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < OUT_ITEMS; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 4;
+      if (c < inner) {
+        float gate[4];
+        load_four(yt + c, v[i]);
+        load_four(z + c, gate);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[i][e] *= silu(gate[e]), ss += v[i][e] * v[i][e];
+      }
+    }
+    const float r = 1.f / sqrtf(block_sum(ss, red) / (float)inner + eps);
+#pragma unroll
+    for (int i = 0; i < OUT_ITEMS; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 4;
+      if (c < inner) {
+        float w[4];
+        load_four(norm_w + c, w);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[i][e] *= r * w[e];
+        store_four(out + t * inner + c, v[i]);
+      }
+    }
+    return;
+  }
   if (norm_groups == 1) {
     float ss = 0.f;
     for (int c = threadIdx.x; c < inner; c += blockDim.x) {
@@ -265,6 +372,7 @@ ssd_out_kernel(const float* __restrict__ y, const T* __restrict__ proj, int stri
   for (int g = threadIdx.x >> 5; g < norm_groups; g += warps) {
     const int c0 = g * run;
     float ss = 0.f;
+#pragma unroll 4
     for (int i = lane; i < run; i += 32) {
       const float v = yt[c0 + i] * silu(to_f32(z[c0 + i]));
       out_s[c0 + i] = v;
@@ -272,6 +380,7 @@ ssd_out_kernel(const float* __restrict__ y, const T* __restrict__ proj, int stri
     }
     const float r = 1.f / sqrtf(warp_sum(ss) / (float)run + eps);
     __syncwarp();
+#pragma unroll 4
     for (int i = lane; i < run; i += 32) out[t * inner + c0 + i] = from_f32<T>(out_s[c0 + i] * r * norm_w[c0 + i]);
   }
 }
@@ -281,15 +390,25 @@ int launch_inputs(const void* proj, int stride, int col0, const Sizes& s, const 
                   const float* conv_state, const float* dt_bias, const float* A_log, const int* cu_seqlens,
                   const int* state_slots, int num_seqs, int tokens, void* rows, int row_stride, int at_x, int at_b, int at_c,
                   float* pairs, int pair_stride, int log_decay, cudaStream_t stream) {
-  const dim3 grid((s.channels() + s.H + 127) / 128, (tokens + RUN - 1) / RUN);
-#define OMNIA_SSD_INPUTS(KT)                                                                                              \
-  launch_pdl(ssd_inputs_kernel<T, O, KT>, grid, dim3(128), 0, stream, (const T*)proj, stride, col0, s, taps, conv_bias, K, \
+  // Two channels a thread where every width, place and stride is even and every base on two elements.
+  const bool even = ((s.inner() | (s.G * s.N) | stride | col0 | row_stride | at_x | at_b | at_c) & 1) == 0 &&
+                    ((uintptr_t)proj % (2 * sizeof(T))) == 0 && ((uintptr_t)rows % (2 * sizeof(O))) == 0 &&
+                    ((uintptr_t)conv_state & 7) == 0;
+  const dim3 grid((s.channels() / (even ? 2 : 1) + s.H + 127) / 128, (tokens + RUN - 1) / RUN);
+#define OMNIA_SSD_INPUTS_AS(KT, VC)                                                                                       \
+  launch_pdl(ssd_inputs_kernel<T, O, KT, VC>, grid, dim3(128), 0, stream, (const T*)proj, stride, col0, s, taps, conv_bias, K, \
              conv_state, dt_bias, A_log, cu_seqlens, state_slots, num_seqs, tokens, (O*)rows, row_stride, at_x, at_b, at_c,  \
              pairs, pair_stride, log_decay)
+#define OMNIA_SSD_INPUTS(KT)                 \
+  do {                                       \
+    if (even) OMNIA_SSD_INPUTS_AS(KT, 2);    \
+    else OMNIA_SSD_INPUTS_AS(KT, 1);         \
+  } while (0)
   if (K <= 4) OMNIA_SSD_INPUTS(4);
   else if (K <= 8) OMNIA_SSD_INPUTS(8);
   else OMNIA_SSD_INPUTS(MAX_TAPS);
 #undef OMNIA_SSD_INPUTS
+#undef OMNIA_SSD_INPUTS_AS
   return OMNIA_LAUNCH_RESULT();
 }
 
@@ -355,14 +474,26 @@ extern "C" int omnia_ssd_out(const float* y, const void* proj, int stride, int c
   if (tokens == 0) return 0;
   const Sizes s{H, dv, G, N};
   if (!sizes_ok(s, K) || norm_groups < 1 || s.inner() % norm_groups) return (int)cudaErrorInvalidValue;
-  const size_t smem = (size_t)s.inner() * sizeof(float);
+  // One norm group in fours: from registers, as many threads as hold it. Anything else: through shared memory.
+  const int quads = s.inner() / 4, whole_threads = ((quads + OUT_ITEMS - 1) / OUT_ITEMS + 31) / 32 * 32;
+  const bool whole = norm_groups == 1 && s.inner() % 4 == 0 && whole_threads <= 1024 && stride % 4 == 0 && col0 % 4 == 0 &&
+                     (((uintptr_t)y | (uintptr_t)proj | (uintptr_t)norm_w | (uintptr_t)out) & 15) == 0;
+  const size_t smem = whole ? 0 : (size_t)s.inner() * sizeof(float);
   if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+  const int threads = whole ? (whole_threads < 128 ? 128 : whole_threads) : 256;
+  const dim3 grid(tokens + (K > 1 ? num_seqs * ((s.channels() + threads - 1) / threads) : 0));
+#define OMNIA_SSD_OUT(WHOLE)                                                                                                 \
+  do {                                                                                                                       \
+    if (smem > 47 * 1024 && cudaFuncSetAttribute(ssd_out_kernel<T, WHOLE>, cudaFuncAttributeMaxDynamicSharedMemorySize,         \
+                                                 (int)smem) != cudaSuccess)                                                  \
+      return (int)cudaGetLastError();                                                                                        \
+    launch_pdl(ssd_out_kernel<T, WHOLE>, grid, dim3(threads), smem, stream, y, (const T*)proj, stride, col0, s, norm_groups,    \
+               eps, norm_w, K, conv_state, cu_seqlens, state_slots, tokens, (T*)out);                                         \
+  } while (0)
   OMNIA_DISPATCH_DTYPE(dtype, {
-    if (smem > 47 * 1024 &&
-        cudaFuncSetAttribute(ssd_out_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
-      return (int)cudaGetLastError();
-    launch_pdl(ssd_out_kernel<T>, dim3(tokens + num_seqs), dim3(256), smem, stream, y, (const T*)proj, stride, col0, s,
-               norm_groups, eps, norm_w, K, conv_state, cu_seqlens, state_slots, tokens, (T*)out);
+    if (whole) OMNIA_SSD_OUT(true);
+    else OMNIA_SSD_OUT(false);
   });
+#undef OMNIA_SSD_OUT
   return OMNIA_LAUNCH_RESULT();
 }

@@ -63,14 +63,14 @@ __device__ __forceinline__ void copy8(const void* smem, const void* gmem, bool v
 }
 __device__ __forceinline__ void ldmatrix(uint32_t* r, const f16* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(shared_address(p)) : "memory");
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(shared_address(p)));
 }
 __device__ __forceinline__ void ldmatrix_t(uint32_t* r, const f16* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(shared_address(p)) : "memory");
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(shared_address(p)));
 }
 __device__ __forceinline__ void mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm volatile(
+  asm(
       "mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
@@ -98,22 +98,14 @@ ssd_chunk_kernel(const f16* __restrict__ rows, int row_stride, int at_x, int at_
   pdl_wait();
   pdl_launch_dependents();
   extern __shared__ __align__(16) unsigned char chunk_smem[];
-  f16* Bs[2], *Cs[2], *Xs[2];
-  float2* ps[2];
-  f16* at = reinterpret_cast<f16*>(chunk_smem);
-#pragma unroll
-  for (int b = 0; b < 2; ++b) {
-    Bs[b] = at, at += L * NROW;
-    Cs[b] = at, at += L * NROW;
-    Xs[b] = at, at += L * XROW;
-  }
-  f16* Sh = at;               // [N][XROW] the state's upper halves, then the lower ones
+  f16* stage0 = reinterpret_cast<f16*>(chunk_smem);  // two stages of [L][NROW] B, [L][NROW] C, [L][XROW] x
+  constexpr int STAGE = L * (2 * NROW + XROW);
+  f16* Sh = stage0 + 2 * STAGE;  // [N][XROW] the state's upper halves, then the lower ones
   f16* Sl = Sh + N * XROW;
   f16* Wh = Sl + N * XROW;    // [L][XROW] the weighted x
   f16* Wl = Wh + L * XROW;
-  ps[0] = reinterpret_cast<float2*>(Wl + L * XROW);
-  ps[1] = ps[0] + L;
-  float* cum = reinterpret_cast<float*>(ps[1] + L);  // running sum of log2 a
+  float2* ps = reinterpret_cast<float2*>(Wl + L * XROW);  // [2][L] (log a, dt)
+  float* cum = reinterpret_cast<float*>(ps + 2 * L);  // running sum of log2 a
   float* dts = cum + L;
   float* wgt = dts + L;                              // what a token's x is weighted with on its way into the state
   float* peaks = wgt + L;                            // each warp's largest entry of the state
@@ -129,18 +121,21 @@ ssd_chunk_kernel(const f16* __restrict__ rows, int row_stride, int at_x, int at_
   const f16* x_rows = rows + at_x + head * dv + col0;
 
   auto fetch = [&](int t0, int n, int b) {
+    f16* Bd = stage0 + b * STAGE;
+    f16* Cd = Bd + L * NROW;
+    f16* Xd = Cd + L * NROW;
     const int fill = min(L, (n + 31) & ~31);  // rows past the portion's end are zeros, up to a whole block of keys
     for (int i = tid; i < fill * (N / 8); i += THREADS) {
       const int r = i / (N / 8), c = (i % (N / 8)) * 8;
       const size_t from = (size_t)(t0 + (r < n ? r : 0)) * row_stride + c;
-      copy16(Bs[b] + r * NROW + c, b_rows + from, r < n);
-      copy16(Cs[b] + r * NROW + c, c_rows + from, r < n);
+      copy16(Bd + r * NROW + c, b_rows + from, r < n);
+      copy16(Cd + r * NROW + c, c_rows + from, r < n);
     }
     for (int i = tid; i < fill * (COLS / 8); i += THREADS) {
       const int r = i / (COLS / 8), c = (i % (COLS / 8)) * 8;
-      copy16(Xs[b] + r * XROW + c, x_rows + (size_t)(t0 + (r < n ? r : 0)) * row_stride + c, r < n);
+      copy16(Xd + r * XROW + c, x_rows + (size_t)(t0 + (r < n ? r : 0)) * row_stride + c, r < n);
     }
-    for (int r = tid; r < L; r += THREADS) copy8(ps[b] + r, pairs + (size_t)(t0 + (r < n ? r : 0)) * H + head, r < n);
+    for (int r = tid; r < L; r += THREADS) copy8(ps + b * L + r, pairs + (size_t)(t0 + (r < n ? r : 0)) * H + head, r < n);
     asm volatile("cp.async.commit_group;\n" ::: "memory");
   };
 
@@ -179,7 +174,7 @@ ssd_chunk_kernel(const f16* __restrict__ rows, int row_stride, int at_x, int at_
     asm volatile("cp.async.wait_group 0;\n" ::: "memory");
     __syncthreads();  // the chunk has arrived, and everybody is done with the last one
     if (c + 1 < chunks) fetch(t0 + L, min(L, end - t0 - L), b ^ 1);
-    const f16 *Bc = Bs[b], *Cc = Cs[b], *Xc = Xs[b];
+    const f16 *Bc = stage0 + b * STAGE, *Cc = Bc + L * NROW, *Xc = Cc + L * NROW;
     // A state beyond 2^15 goes down by a power of two on its way into the product, whose result goes up by it.
     float peak = peaks[0];
 #pragma unroll
@@ -205,7 +200,7 @@ ssd_chunk_kernel(const f16* __restrict__ rows, int row_stride, int at_x, int at_
       float sum[PER], dt[PER], total = 0.f;
 #pragma unroll
       for (int i = 0; i < PER; ++i) {
-        const float2 pair = ps[b][lane * PER + i];  // zeros past the portion's end
+        const float2 pair = ps[b * L + lane * PER + i];  // zeros past the portion's end
         total += pair.x * 1.4426950408889634f;
         sum[i] = total, dt[i] = pair.y;
       }
