@@ -185,7 +185,7 @@ ssd_inputs_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, con
 // convolution, then S moved on in place, four columns and every `teams`-th row a thread, the teams' sums added in
 // their order. y float32 [tokens, inner].
 template <typename T, int VEC>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 4)
 ssd_step_kernel(const T* __restrict__ proj, int stride, int col0, Sizes s, int cols, const float* __restrict__ taps,
                 const float* __restrict__ conv_bias, int K, const float* __restrict__ conv_state,
                 const float* __restrict__ dt_bias, const float* __restrict__ A_log, const float* __restrict__ D,

@@ -222,6 +222,7 @@ ssd_chunk_kernel(const f16* __restrict__ rows, int row_stride, int at_x, int at_
     }
     __syncthreads();
     const int key_rows = (n + 15) & ~15;
+#pragma unroll 8
     for (int i = tid; i < key_rows * (COLS / 2); i += THREADS) {
       const int r = i / (COLS / 2), place = r * XROW + (i % (COLS / 2)) * 2;
       const float w = wgt[r];

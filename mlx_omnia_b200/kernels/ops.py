@@ -15,6 +15,7 @@ from ctypes import c_float, c_int, c_longlong, c_void_p
 
 import dataclasses
 from dataclasses import dataclass
+from typing import Callable
 
 import numpy as np
 import torch
@@ -874,6 +875,9 @@ def _gemm_tcgen05(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epil
               _ptr(error_word(a.device)), _stream()), library)
     return out
 
+
+SIDE_BY_SIDE_ROWS = 256
+"""Up to this many rows, two branches of a captured step are recorded side by side."""
 
 _side_streams: dict[int, "torch.cuda.Stream"] = {}
 
@@ -1900,7 +1904,7 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
                 tensor_cores: bool | None = None, tcgen05: bool | None = None,
                 table: torch.Tensor | None = None, token_ids: torch.Tensor | None = None,
                 alpha: float = 1.0, limit: float = 0.0, scoring: str = "softmax", weigh: str = "output",
-                extra: torch.Tensor | None = None, groups: int = 1, keep_groups: int = 1, normalise: bool = False,
+                extra: "torch.Tensor | Callable[[], torch.Tensor] | None" = None, groups: int = 1, keep_groups: int = 1, normalise: bool = False,
                 weight_scale: float = 1.0, combine: bool = True, bias: torch.Tensor | None = None,
                 activation: str | None = None, shared_gated: bool = False) -> "torch.Tensor | ExpertRows":
     """A routed mixture of gated feed-forward experts over the rows of `h` [rows, hidden]:
@@ -1918,7 +1922,8 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
     `scoring`: the router's scores are a "softmax" over all outputs or every output's own "sigmoid".
     `weigh` "input": y = sum of expert(score * h) instead: a choice's score multiplies what its expert
     is given (the product in float32, rounded once), and the experts' outputs are added as they are.
-    `extra` [rows, hidden]: added to y in the same pass (an expert that every row uses).
+    `extra` [rows, hidden]: added to y in the same pass (an expert that every row uses), or a function that makes it
+    (called where it can run beside the chosen experts).
     `groups`, `keep_groups`, `normalise`, `weight_scale`: how the choice is narrowed and weighted (`moe_route`).
     `combine` False (no `extra`, no identity experts, weights on the outputs): the choices' rows and their
     weights are returned as they are, for `depth_step` to sum on their way into the residual.
@@ -1944,58 +1949,70 @@ def moe_experts(h: torch.Tensor, router: torch.Tensor | None, correction: torch.
         tcgen05 = tensor_cores and pairs >= MOE_TCGEN05_PAIRS and pairs >= 64 * experts
     tile_rows = 128 if tcgen05 else MOE_TILE_ROWS
     max_tiles = min(pairs, -(-pairs // tile_rows) + experts)
-    counts, cursors = _step_buffers(step, device, {"moe_counts": (experts, torch.int32, True),
-                                                   "moe_cursors": (experts, torch.int32, True)})
-    if table is not None:
-        choice, weight = moe_route_table(token_ids[:rows], table, experts, counts)
-        shared_gate = None
-    else:
-        shared_gate = torch.empty(rows, dtype=torch.float32, device=device) if shared_gated else None
-        choice, weight = moe_route(h, router, correction, experts, top, counts, scoring, groups, keep_groups, normalise,
-                                   weight_scale, bias, shared_gate)
-    ints = torch.empty(2 * pairs + experts + 1 + 3 * max_tiles + 1, dtype=torch.int32, device=device)
-    place, source = ints[:pairs], ints[pairs: 2 * pairs]
-    offsets = ints[2 * pairs: 2 * pairs + experts + 1]
-    tiles = ints[2 * pairs + experts + 1: 2 * pairs + experts + 1 + 3 * max_tiles]
-    tile_count = ints[-1:]
-    fn = _function("moe", "omnia_moe_plan",
-                   [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                    c_int, c_int, c_void_p])
-    _check(fn(_ptr(choice), _ptr(counts), _ptr(cursors), _ptr(offsets), _ptr(tiles), _ptr(tile_count), _ptr(place),
-              _ptr(source), rows, top, experts, max_tiles, tile_rows, _stream()), "moe_plan")
-    act = torch.empty(pairs, inner, dtype=h.dtype, device=device)
-    out = torch.empty(pairs, hidden, dtype=h.dtype, device=device)
-    sorted_rows = None
-    if weigh == "input":
-        # The weighted rows in sorted order; rows past the last sorted one (identity choices) stay unread.
-        sorted_rows = torch.empty(pairs, hidden, dtype=h.dtype, device=device)
-        fn = _function("moe", "omnia_moe_weighted_rows",
-                       [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-        _check(fn(_ptr(h), _ptr(place), _ptr(weight), _ptr(sorted_rows), pairs, hidden, top, _code(h.dtype), _stream()),
-               "moe_weighted_rows")
-    if tcgen05:
-        if sorted_rows is None:
+    def chosen() -> tuple:
+        """The choices, and every chosen expert's output."""
+        counts, cursors = _step_buffers(step, device, {"moe_counts": (experts, torch.int32, True),
+                                                       "moe_cursors": (experts, torch.int32, True)})
+        if table is not None:
+            choice, weight = moe_route_table(token_ids[:rows], table, experts, counts)
+            shared_gate = None
+        else:
+            shared_gate = torch.empty(rows, dtype=torch.float32, device=device) if shared_gated else None
+            choice, weight = moe_route(h, router, correction, experts, top, counts, scoring, groups, keep_groups, normalise,
+                                       weight_scale, bias, shared_gate)
+        ints = torch.empty(2 * pairs + experts + 1 + 3 * max_tiles + 1, dtype=torch.int32, device=device)
+        place, source = ints[:pairs], ints[pairs: 2 * pairs]
+        offsets = ints[2 * pairs: 2 * pairs + experts + 1]
+        tiles = ints[2 * pairs + experts + 1: 2 * pairs + experts + 1 + 3 * max_tiles]
+        tile_count = ints[-1:]
+        fn = _function("moe", "omnia_moe_plan",
+                       [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                        c_int, c_int, c_void_p])
+        _check(fn(_ptr(choice), _ptr(counts), _ptr(cursors), _ptr(offsets), _ptr(tiles), _ptr(tile_count), _ptr(place),
+                  _ptr(source), rows, top, experts, max_tiles, tile_rows, _stream()), "moe_plan")
+        act = torch.empty(pairs, inner, dtype=h.dtype, device=device)
+        out = torch.empty(pairs, hidden, dtype=h.dtype, device=device)
+        sorted_rows = None
+        if weigh == "input":
+            # The weighted rows in sorted order; rows past the last sorted one (identity choices) stay unread.
             sorted_rows = torch.empty(pairs, hidden, dtype=h.dtype, device=device)
-            fn = _function("moe", "omnia_moe_gather", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
-            _check(fn(_ptr(h), _ptr(source), _ptr(offsets[experts:]), _ptr(sorted_rows), pairs, hidden, _code(h.dtype),
-                      _stream()), "moe_gather")
-        grouped = _function("gemm_tcgen05", "omnia_gemm_tcgen05_grouped",
-                            [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
-                             c_float, c_float, c_void_p, c_void_p])
-        err = _ptr(error_word(device))
-        _check(grouped(_ptr(sorted_rows), _ptr(gate_up), _ptr(act), pairs, gate_up.shape[1], hidden, experts, int(dual), _ptr(tiles),
-                       _ptr(tile_count), max_tiles, alpha, limit, err, _stream()), "gemm_tcgen05_grouped")
-        _check(grouped(_ptr(act), _ptr(down), _ptr(out), pairs, hidden, inner, experts, 0, _ptr(tiles),
-                       _ptr(tile_count), max_tiles, 1.0, 0.0, err, _stream()), "gemm_tcgen05_grouped")
+            fn = _function("moe", "omnia_moe_weighted_rows",
+                           [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+            _check(fn(_ptr(h), _ptr(place), _ptr(weight), _ptr(sorted_rows), pairs, hidden, top, _code(h.dtype), _stream()),
+                   "moe_weighted_rows")
+        if tcgen05:
+            if sorted_rows is None:
+                sorted_rows = torch.empty(pairs, hidden, dtype=h.dtype, device=device)
+                fn = _function("moe", "omnia_moe_gather", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+                _check(fn(_ptr(h), _ptr(source), _ptr(offsets[experts:]), _ptr(sorted_rows), pairs, hidden, _code(h.dtype),
+                          _stream()), "moe_gather")
+            grouped = _function("gemm_tcgen05", "omnia_gemm_tcgen05_grouped",
+                                [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+                                 c_float, c_float, c_void_p, c_void_p])
+            err = _ptr(error_word(device))
+            _check(grouped(_ptr(sorted_rows), _ptr(gate_up), _ptr(act), pairs, gate_up.shape[1], hidden, experts, int(dual), _ptr(tiles),
+                           _ptr(tile_count), max_tiles, alpha, limit, err, _stream()), "gemm_tcgen05_grouped")
+            _check(grouped(_ptr(act), _ptr(down), _ptr(out), pairs, hidden, inner, experts, 0, _ptr(tiles),
+                           _ptr(tile_count), max_tiles, 1.0, 0.0, err, _stream()), "gemm_tcgen05_grouped")
+        else:
+            product = _function("moe", "omnia_moe_product",
+                                [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                 c_float, c_float, c_int, c_int, c_void_p])
+            _check(product(_ptr(h if sorted_rows is None else sorted_rows), _ptr(source) if sorted_rows is None else None,
+                           _ptr(gate_up), _ptr(act), _ptr(tiles), _ptr(tile_count), max_tiles, inner,
+                           hidden, int(dual), alpha, limit, _code(h.dtype), int(tensor_cores), _stream()), "moe_product")
+            _check(product(_ptr(act), None, _ptr(down), _ptr(out), _ptr(tiles), _ptr(tile_count), max_tiles, hidden, inner, 0,
+                           1.0, 0.0, _code(h.dtype), int(tensor_cores), _stream()), "moe_product")
+        return out, place, weight, shared_gate
+
+    if callable(extra):
+        # What every row uses needs no choice: in a captured step of few rows it runs beside the chosen experts.
+        if rows <= SIDE_BY_SIDE_ROWS:
+            (out, place, weight, shared_gate), extra = side_by_side(chosen, extra, device)
+        else:
+            (out, place, weight, shared_gate), extra = chosen(), extra()
     else:
-        product = _function("moe", "omnia_moe_product",
-                            [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                             c_float, c_float, c_int, c_int, c_void_p])
-        _check(product(_ptr(h if sorted_rows is None else sorted_rows), _ptr(source) if sorted_rows is None else None,
-                       _ptr(gate_up), _ptr(act), _ptr(tiles), _ptr(tile_count), max_tiles, inner,
-                       hidden, int(dual), alpha, limit, _code(h.dtype), int(tensor_cores), _stream()), "moe_product")
-        _check(product(_ptr(act), None, _ptr(down), _ptr(out), _ptr(tiles), _ptr(tile_count), max_tiles, hidden, inner, 0,
-                       1.0, 0.0, _code(h.dtype), int(tensor_cores), _stream()), "moe_product")
+        out, place, weight, shared_gate = chosen()
     if not combine:
         if extra is not None or shared_gated or weigh != "output" or (router is not None and router.shape[0] != experts):
             raise KernelError("rows that are summed elsewhere have no extra branch, no identity experts and weigh outputs")

@@ -355,10 +355,6 @@ class BranchNormBlock(Block):
         return x, self._step(x, m, self.norms["norm2"], exit_norm, True)
 
 
-SIDE_BY_SIDE_ROWS = 256
-"""Up to this many rows a parallel block's two branches are captured side by side."""
-
-
 @register_block("parallel")
 class ParallelBlock(Block):
     """One norm whose output both branches read: r = x + mixer(norm(x)) + feed_forward(norm(x)). The
@@ -413,7 +409,7 @@ class ParallelBlock(Block):
             ff = self.feed_forward
             rows = getattr(ff, "gives_rows", False)
             feed = lambda: ff.forward_rows(h, ctx) if rows else ff.forward(h, ctx)  # noqa: E731
-            if h.shape[0] <= SIDE_BY_SIDE_ROWS:
+            if h.shape[0] <= ops.SIDE_BY_SIDE_ROWS:
                 branch, second = ops.side_by_side(mix, feed, h.device)
             else:
                 branch, second = mix(), feed()

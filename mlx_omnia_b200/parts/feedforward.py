@@ -267,10 +267,10 @@ class RoutedExperts(FeedForward):
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
         extra = None
         if self.shared_gate_up is not None:
-            if self.unit == "gelu_erf":
-                extra = ops.linear(ops.linear_act(h, self.shared_gate_up, self.unit), self.shared_down)
-            else:
-                extra = ops.linear(ops.linear_swiglu(h, self.shared_gate_up), self.shared_down)
+            def extra() -> torch.Tensor:
+                if self.unit == "gelu_erf":
+                    return ops.linear(ops.linear_act(h, self.shared_gate_up, self.unit), self.shared_down)
+                return ops.linear(ops.linear_swiglu(h, self.shared_gate_up), self.shared_down)
         return self._experts(h, ctx, extra, True)
 
     @property
