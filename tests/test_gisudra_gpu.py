@@ -260,7 +260,7 @@ def test_a_far_token_shows_through_a_slow_decay(dtype):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("H,G,dk,dv,size,keep,page", [(4, 2, 64, 64, 25, 7, 16), (6, 2, 16, 24, 11, 5, 4), (3, 3, 5, 7, 1, 2, 8),
-                                                      (8, 2, 128, 128, 40, 20, 16), (2, 2, 32, 32, None, 0, 16), (4, 1, 96, 96, 33, 16, 16),
+                                                      (8, 2, 128, 128, 45, 18, 16), (2, 2, 32, 32, None, 0, 16), (4, 1, 96, 96, 33, 16, 16),
                                                       (4, 4, 64, 64, 3, 0, 4), (20, 1, 8, 8, 17, 1, 16), (5, 1, 64, 96, 50, 32, 16)])
 def test_windowed_attention_with_kept_tokens_and_mixed_values(dtype, H, G, dk, dv, size, keep, page):
     """Two layers in one pass, the second mixing the first one's values into its own: two requests in portions and
