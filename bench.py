@@ -1860,17 +1860,17 @@ def run_gisudra(args) -> dict:
             # key channel (half the attention's heads); flops: the token-by-token form's two products a head
             HM, dv, N, K = 2 * D // 64, 64, 128, 4
             inner, channels = HM * dv, HM * dv + 2 * N
-            mproj = (torch.randn(T, inner + channels + HM, device=dev) * 0.5).to(bf)
+            mproj = torch.randn(T, inner + channels + HM, device=dev) * 0.5
             w = ops.SSDWeights(torch.randn(channels, K, device=dev) * 0.5, torch.zeros(channels, device=dev),
                                torch.full((HM,), -2.0, device=dev), torch.zeros(HM, device=dev), torch.ones(HM, device=dev),
                                torch.ones(inner, device=dev))
             S, conv = torch.zeros(n + 1, HM, N, dv, device=dev), torch.zeros(n + 1, K - 1, channels, device=dev)
-            note(f"ssd_mixer_{mode}", lambda: ops.ssd_mixer(mproj, 0, HM, dv, 1, N, w, 1, 1e-5, S, conv, st), reps,
-                 bytes_=mproj.numel() * 2 + T * inner * 2 + 8 * n * HM * N * dv, flops=4 * T * HM * N * dv)
+            note(f"ssd_mixer_{mode}", lambda: ops.ssd_mixer(mproj, 0, HM, dv, 1, N, w, 1, 1e-5, S, conv, st, dtype=bf), reps,
+                 bytes_=mproj.numel() * 4 + T * inner * 2 + 8 * n * HM * N * dv, flops=4 * T * HM * N * dv)
             if mode == "prefill":
                 note("ssd_mixer_token_by_token_prefill",
-                     lambda: ops.ssd_mixer(mproj, 0, HM, dv, 1, N, w, 1, 1e-5, S, conv, st, chunked=False), reps,
-                     bytes_=mproj.numel() * 2 + T * inner * 2 + 8 * n * HM * N * dv, flops=4 * T * HM * N * dv)
+                     lambda: ops.ssd_mixer(mproj, 0, HM, dv, 1, N, w, 1, 1e-5, S, conv, st, chunked=False, dtype=bf), reps,
+                     bytes_=mproj.numel() * 4 + T * inner * 2 + 8 * n * HM * N * dv, flops=4 * T * HM * N * dv)
             R = max(H // 2, 1)
             sproj = (torch.randn(T, 4 * R * d, device=dev) * 0.5).to(bf)
             logits, zb, S2 = torch.randn(T, R * d, device=dev), torch.zeros(R * d, device=dev), torch.zeros(n + 1, R, d, d, device=dev)

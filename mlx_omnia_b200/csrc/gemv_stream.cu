@@ -438,7 +438,8 @@ gemv_stream_kernel(const bf16* __restrict__ a, const __grid_constant__ CUtensorM
           const int col = tile * TILE_ROWS + r;
           if (col >= n) continue;
           if (EPI == EPI_SOFTCAP) {
-            const float z = __bfloat162float(__float2bfloat16_rn(v)) * multiplier;
+            // cap < 0: the float32 product as it is, for a reader that goes on in float32.
+            const float z = (cap < 0.f ? v : __bfloat162float(__float2bfloat16_rn(v))) * multiplier;
             reinterpret_cast<float*>(out)[(size_t)token * n + col] = cap > 0.f ? cap * tanhf(z / cap) : z;
           } else {
             // cap selects an activation of the stored product (0 none, 1 relu^2, 2 tanh-GELU, 3 SiLU, 4 xIELU
@@ -543,7 +544,7 @@ int launch_rows(const bf16* a, const bf16* w, void* out, int m, int n, int k, in
 }  // namespace
 
 // epilogue: 0 store bfloat16 [m, n] (cap 1, 2, 3: relu^2, tanh-GELU or SiLU of the product, 4: xIELU with the constants `multiplier` and `second`, 5: exact GELU; 0: as it is); 1 SwiGLU, w = [gate rows | up rows] with n = 2 * inner,
-// out bfloat16 [m, inner] (cap > 0: the clamped unit min(gate, cap) * sigmoid(multiplier * min(gate, cap)) * (clamp(up, +-cap) + 1); cap -1: relu(gate) * up, -2: tanh-GELU(gate) * up); 2 soft cap, out float32 [m, n]. err: the device error word.
+// out bfloat16 [m, inner] (cap > 0: the clamped unit min(gate, cap) * sigmoid(multiplier * min(gate, cap)) * (clamp(up, +-cap) + 1); cap -1: relu(gate) * up, -2: tanh-GELU(gate) * up); 2 soft cap, out float32 [m, n] (cap < 0: no cap, and the product not rounded). err: the device error word.
 extern "C" int omnia_gemv_stream(const void* a, const void* w, void* out, int m, int n, int k, int epilogue,
                                  float multiplier, float cap, float second, int* err, cudaStream_t stream) {
   if (m == 0 || n == 0) return 0;
@@ -564,7 +565,7 @@ extern "C" int omnia_gemv_stream(const void* a, const void* w, void* out, int m,
 
 extern "C" int omnia_gemv_stream_pending_max_k(void) { return PENDING_MAX_K; }
 
-// The same product with a pending residual step in front of it (epilogues 0 and 1):
+// The same product with a pending residual step in front of it (epilogues 0, 1, and 2 with cap < 0):
 //   x_out = x + (norm_branch ? rms(branch, eps_b) * wb : branch),  a = bfloat16(rms(x_out, eps_o) * wo),
 // x, x_out float32 [m, k] (different buffers, m <= 8), branch bfloat16 [m, k], wb, wo float32 [k] or null.
 extern "C" int omnia_gemv_stream_pending(const float* x, float* x_out, const void* branch, const float* wb,
@@ -582,6 +583,8 @@ extern "C" int omnia_gemv_stream_pending(const float* x, float* x_out, const voi
     if (n % 2 || cap > 0.f) return (int)cudaErrorInvalidValue;
     return launch_rows<EPI_SWIGLU, true>(nullptr, wp, out, m, n, k, n / 2, 1.f, cap, 0.f, pending, err, stream);
   }
+  if (epilogue == EPI_SOFTCAP && cap < 0.f)
+    return launch_rows<EPI_SOFTCAP, true>(nullptr, wp, out, m, n, k, 0, 1.f, cap, 0.f, pending, err, stream);
   if (epilogue != EPI_STORE) return (int)cudaErrorInvalidValue;
   return launch_rows<EPI_STORE, true>(nullptr, wp, out, m, n, k, 0, 1.f, 0.f, 0.f, pending, err, stream);
 }

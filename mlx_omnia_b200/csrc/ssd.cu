@@ -16,8 +16,10 @@
 //            [x | B | C] beside float32 pairs (log a, dt).
 //   step     a step in which every request brings one token: convolution, step sizes and recurrence in one
 //            kernel, a block per (request, head, run of columns).
-//   out      per token: the skip's y times silu(z), norm and weight, rounded once; and, after the last token,
+//   out      per token: y (the skip in it) times silu(z), norm and weight, rounded once; and, after the last token,
 //            per request: the convolution's carried inputs moved on.
+//
+// The projected rows may be float32 where the rest of the model is bfloat16.
 #include "common.cuh"
 
 #include <cuda_fp16.h>
@@ -298,11 +300,11 @@ __device__ __forceinline__ void store_four(__nv_bfloat16* p, const float* v) {
 
 // Blocks 0 .. tokens - 1: a token each; the others: blockDim channels of a request's carried inputs each.
 // WHOLE: one norm group, its channels in fours and in the threads' registers.
-template <typename T, bool WHOLE>
+template <typename T, typename O, bool WHOLE>
 __global__ void __launch_bounds__(1024)
 ssd_out_kernel(const float* __restrict__ y, const T* __restrict__ proj, int stride, int col0, Sizes s, int norm_groups,
                float eps, const float* __restrict__ norm_w, int K, float* __restrict__ conv_state,
-               const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, int tokens, T* __restrict__ out) {
+               const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, int tokens, O* __restrict__ out) {
   pdl_wait();
   pdl_launch_dependents();
   extern __shared__ __align__(16) float out_s[];
@@ -364,7 +366,7 @@ ssd_out_kernel(const float* __restrict__ y, const T* __restrict__ proj, int stri
       ss += v * v;
     }
     const float r = 1.f / sqrtf(block_sum(ss, red) / (float)run + eps);
-    for (int c = threadIdx.x; c < inner; c += blockDim.x) out[t * inner + c] = from_f32<T>(out_s[c] * r * norm_w[c]);
+    for (int c = threadIdx.x; c < inner; c += blockDim.x) out[t * inner + c] = from_f32<O>(out_s[c] * r * norm_w[c]);
     return;
   }
   // A warp takes a group at a time.
@@ -381,7 +383,7 @@ ssd_out_kernel(const float* __restrict__ y, const T* __restrict__ proj, int stri
     const float r = 1.f / sqrtf(warp_sum(ss) / (float)run + eps);
     __syncwarp();
 #pragma unroll 4
-    for (int i = lane; i < run; i += 32) out[t * inner + c0 + i] = from_f32<T>(out_s[c0 + i] * r * norm_w[c0 + i]);
+    for (int i = lane; i < run; i += 32) out[t * inner + c0 + i] = from_f32<O>(out_s[c0 + i] * r * norm_w[c0 + i]);
   }
 }
 
@@ -470,7 +472,7 @@ extern "C" int omnia_ssd_step(const void* proj, int stride, int col0, int H, int
 extern "C" int omnia_ssd_out(const float* y, const void* proj, int stride, int col0, int H, int dv, int G, int N,
                              int norm_groups, float eps, const float* norm_w, int K, float* conv_state,
                              const int* cu_seqlens, const int* state_slots, int num_seqs, int tokens, void* out, int dtype,
-                             cudaStream_t stream) {
+                             int out_dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
   const Sizes s{H, dv, G, N};
   if (!sizes_ok(s, K) || norm_groups < 1 || s.inner() % norm_groups) return (int)cudaErrorInvalidValue;
@@ -484,16 +486,27 @@ extern "C" int omnia_ssd_out(const float* y, const void* proj, int stride, int c
   const dim3 grid(tokens + (K > 1 ? num_seqs * ((s.channels() + threads - 1) / threads) : 0));
 #define OMNIA_SSD_OUT(WHOLE)                                                                                                 \
   do {                                                                                                                       \
-    if (smem > 47 * 1024 && cudaFuncSetAttribute(ssd_out_kernel<T, WHOLE>, cudaFuncAttributeMaxDynamicSharedMemorySize,         \
+    if (smem > 47 * 1024 && cudaFuncSetAttribute(ssd_out_kernel<T, O, WHOLE>, cudaFuncAttributeMaxDynamicSharedMemorySize,         \
                                                  (int)smem) != cudaSuccess)                                                  \
       return (int)cudaGetLastError();                                                                                        \
-    launch_pdl(ssd_out_kernel<T, WHOLE>, grid, dim3(threads), smem, stream, y, (const T*)proj, stride, col0, s, norm_groups,    \
-               eps, norm_w, K, conv_state, cu_seqlens, state_slots, tokens, (T*)out);                                         \
+    launch_pdl(ssd_out_kernel<T, O, WHOLE>, grid, dim3(threads), smem, stream, y, (const T*)proj, stride, col0, s, norm_groups,    \
+               eps, norm_w, K, conv_state, cu_seqlens, state_slots, tokens, (O*)out);                                         \
   } while (0)
-  OMNIA_DISPATCH_DTYPE(dtype, {
+  // The output in the projected rows' type, or bfloat16 from float32 rows.
+  if (dtype == OMNIA_F32 && out_dtype == OMNIA_BF16) {
+    using T = float;
+    using O = __nv_bfloat16;
     if (whole) OMNIA_SSD_OUT(true);
     else OMNIA_SSD_OUT(false);
-  });
+  } else if (dtype == out_dtype) {
+    OMNIA_DISPATCH_DTYPE(dtype, {
+      using O = T;
+      if (whole) OMNIA_SSD_OUT(true);
+      else OMNIA_SSD_OUT(false);
+    });
+  } else {
+    return (int)cudaErrorInvalidValue;
+  }
 #undef OMNIA_SSD_OUT
   return OMNIA_LAUNCH_RESULT();
 }

@@ -1053,7 +1053,8 @@ def _pending_product(step: PendingStep, weight: torch.Tensor, epilogue: int, uni
                                       and pending_supported(step.x, step.branch)):
         return None
     rows, n = step.x.shape[0], weight.shape[0]
-    out = torch.empty(rows, n // 2 if epilogue == 1 else n, dtype=torch.bfloat16, device=step.x.device)
+    out = torch.empty(rows, n // 2 if epilogue == 1 else n, dtype=torch.float32 if epilogue == 2 else torch.bfloat16,
+                      device=step.x.device)
     x_new = torch.empty_like(step.x)
     fn = _function("gemv_stream", "omnia_gemv_stream_pending",
                    [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_float, c_void_p, c_void_p,
@@ -1079,6 +1080,23 @@ def linear(a, weight: torch.Tensor) -> torch.Tensor:
     if _skinny(a, weight):
         return _gemv_stream(a, weight, torch.empty(a.shape[0], weight.shape[0], dtype=a.dtype, device=a.device), 0)
     return _library_mm(a, weight)
+
+
+def linear_wide(a, weight: torch.Tensor) -> torch.Tensor:
+    """a @ weight^T as float32, the products' accumulators unrounded, for a reader that goes on in float32. A few
+    bfloat16 rows (a decode step, with the pending residual step in front) on the weight-streaming kernel, otherwise
+    the vendor library's product with a float32 result. `a` may be a PendingStep."""
+    if isinstance(a, PendingStep):
+        out = _pending_product(a, weight, 2, -1.0)
+        if out is not None:
+            return out
+        a = settle(a)
+    if a.dtype == torch.float32:
+        return _library_mm(a, weight)
+    if _skinny(a, weight):
+        out = torch.empty(a.shape[0], weight.shape[0], dtype=torch.float32, device=a.device)
+        return _gemv_stream(a, weight, out, 2, 1.0, -1.0)
+    return torch.mm(a, weight.t(), out_dtype=torch.float32)
 
 
 def linear_add(a: torch.Tensor, weight: torch.Tensor, alpha: float, other: torch.Tensor, beta: float) -> torch.Tensor:
@@ -1567,7 +1585,7 @@ class SSDWeights:
 
 def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N: int, w: SSDWeights, norm_groups: int,
               eps: float, S: torch.Tensor, conv_state: torch.Tensor, step: StepContext,
-              chunked: bool | None = None) -> torch.Tensor:
+              chunked: bool | None = None, dtype: torch.dtype | None = None) -> torch.Tensor:
     """A state-space mixer from its projected rows (columns from `col0`: z | x | B | C | dt) to what its output
     projection takes, request by request from `S` [slots, heads, N, dv] and `conv_state` [slots, K - 1, channels]
     (float32, both moved on): x, B, C = silu(convolution + bias), dt = softplus(dt + dt_bias),
@@ -1575,8 +1593,9 @@ def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N
     group of neighbouring heads), then RMS norm of y silu(z) over `norm_groups` equal runs, with weight.
     The recurrence runs in float32 token by token, or (`chunked` None: where it applies) in chunks on the tensor
     cores from x, B and C rounded to float16, everything else of it in float32 or as sums of two float16
-    numbers; a step of single tokens is one kernel. -> [tokens, heads * dv] in proj's type"""
+    numbers; a step of single tokens is one kernel. -> [tokens, heads * dv] in `dtype` (None: proj's)"""
     tokens, stride = proj.shape
+    dtype = dtype or proj.dtype
     inner, channels, K = heads * dv, heads * dv + 2 * groups * N, w.taps.shape[1]
     if col0 + inner + channels + heads > stride or w.taps.shape[0] != channels or not 1 <= K <= SSD_MAX_TAPS:
         raise KernelError(f"a state-space mixer of {channels} channels and {K} taps does not fit rows of {stride}")
@@ -1590,7 +1609,7 @@ def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N
                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p])
         _check(fn(_ptr(proj), stride, col0, heads, dv, groups, N, step_cols, _ptr(w.taps), _ptr(w.conv_bias), K, _ptr(conv_state),
                   _ptr(w.dt_bias), _ptr(w.A_log), _ptr(w.D), _ptr(S), *where, _ptr(y), code, _stream()), "ssd_step")
-    elif chunked is not False and (cols := ssd_chunk_columns(step.num_seqs, heads, dv, N, proj.dtype, sm_count(device))):
+    elif chunked is not False and (cols := ssd_chunk_columns(step.num_seqs, heads, dv, N, dtype, sm_count(device))):
         rows = torch.empty(tokens, channels, dtype=torch.float16, device=device)
         pairs = torch.empty(tokens, 2 * heads, dtype=torch.float32, device=device)
         at_b, at_c = inner, inner + groups * N
@@ -1602,7 +1621,7 @@ def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N
                   _stream()), "ssd_chunk")
     else:
         if chunked:
-            raise KernelError(f"the chunked recurrence does not take a state of {N} rows and heads of {dv} in {proj.dtype}")
+            raise KernelError(f"the chunked recurrence does not take a state of {N} rows and heads of {dv} in {dtype}")
         pad4 = lambda n: -(-n // 4) * 4  # noqa: E731
         at_b = pad4(groups * N)
         at_x = 2 * at_b
@@ -1616,12 +1635,12 @@ def ssd_mixer(proj: torch.Tensor, col0: int, heads: int, dv: int, groups: int, N
                         c_void_p, c_int, c_void_p], {"STATE_DK": N})
         _check(fn(_ptr(rows), heads, dv, cols, 2, None, groups, _ptr(w.D), _ptr(S), *where, _ptr(y), 0, _stream()),
                "state_recurrence")
-    out = torch.empty(tokens, inner, dtype=proj.dtype, device=device)
+    out = torch.empty(tokens, inner, dtype=dtype, device=device)
     fn = _function("ssd", "omnia_ssd_out",
                    [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p,
-                    c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p])
+                    c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p])
     _check(fn(_ptr(y), _ptr(proj), stride, col0, heads, dv, groups, N, norm_groups, eps, _ptr(w.norm), K, _ptr(conv_state),
-              *where, tokens, _ptr(out), code, _stream()), "ssd_out")
+              *where, tokens, _ptr(out), code, _code(dtype), _stream()), "ssd_out")
     return out
 
 

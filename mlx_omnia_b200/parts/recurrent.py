@@ -425,13 +425,15 @@ class StateSpace(Mixer):
         self.weights = ops.SSDWeights(*(tensors[name].contiguous() for name in ("conv", "conv.b", "dt_bias", "A_log", "D", "norm")))
 
     def forward(self, h, ctx) -> torch.Tensor:
-        return ops.linear(self.forward_heads(ops.linear(h, self.in_proj), 0, ctx), self.o)
+        # The input projection stays in float32: where the gated y is nearly zero, the norm behind it magnifies
+        # whatever the projection was rounded by.
+        return ops.linear(self.forward_heads(ops.linear_wide(h, self.in_proj), 0, ctx), self.o)
 
     def forward_heads(self, proj: torch.Tensor, col0: int, ctx) -> torch.Tensor:
         """The normed channels, ahead of the output projection, from projected rows whose columns from `col0` on
         are this mixer's input projection."""
         return ops.ssd_mixer(proj, col0, self.heads, self.vdim, self.groups, self.state, self.weights, self.norm_groups,
-                             self.norm_eps, ctx.state["S"], ctx.state["conv"], ctx.step)
+                             self.norm_eps, ctx.state["S"], ctx.state["conv"], ctx.step, dtype=self.runtime.dtype)
 
 
 @register_mixer("side_by_side")

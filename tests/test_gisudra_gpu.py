@@ -447,6 +447,23 @@ def test_a_pending_residual_step_in_front_of_the_gated_unit(rows):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("rows", [1, 8, 16, 50, 400])
+def test_a_product_that_stays_in_float32(dtype, rows):
+    """Unrounded on every path, also with a pending residual step in front: far closer than one bfloat16 rounding."""
+    g = torch.Generator().manual_seed(rows)
+    h, w = torch.randn(rows, 128, generator=g).to(DTYPES[dtype]), (torch.randn(72, 128, generator=g) * 128 ** -0.5).to(DTYPES[dtype])
+    got = ops.linear_wide(h.to(CUDA), w.to(CUDA))
+    assert got.dtype == torch.float32 and rel(got, h.double() @ w.double().T) < 1e-5
+    if dtype == "bfloat16" and rows <= 8:
+        x, nw = torch.randn(rows, 128, generator=g), 1 + 0.1 * torch.randn(128, generator=g)
+        pending = ops.PendingStep(x.to(CUDA), h.to(CUDA), None, None, nw.to(CUDA), 1e-5)
+        got = ops.linear_wide(pending, w.to(CUDA))
+        normed = plain.rms(x.double() + h.double(), 1e-5, nw).float().to(torch.bfloat16).double()
+        assert got.dtype == torch.float32 and rel(got, normed @ w.double().T) < 2e-3
+        assert rel(ops.residual_after(pending, None), x.double() + h.double()) < 1e-6
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("tokens,width,stride", [(3, 64, 64), (5, 130, 139), (1, 7, 9), (40, 1024, 1200)])
 def test_gating_rows_in_place(dtype, tokens, width, stride):
     g = torch.Generator().manual_seed(width)
