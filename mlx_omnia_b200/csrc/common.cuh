@@ -67,13 +67,12 @@ __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + er
 #define OMNIA_UNIT_RELU (-1.f)
 #define OMNIA_UNIT_GELU_TANH (-2.f)
 __device__ __forceinline__ float gated_unit(float gate, float up, float slope, float cap) {
+  if (cap == 0.f) return gate / (1.f + expf(-gate)) * up;
   if (cap > 0.f) {
     const float g = fminf(gate, cap), u = fminf(fmaxf(up, -cap), cap);
     return g / (1.f + expf(-slope * g)) * (u + 1.f);
   }
-  if (cap <= OMNIA_UNIT_GELU_TANH) return gelu_tanh(gate) * up;
-  if (cap < 0.f) return fmaxf(gate, 0.f) * up;
-  return gate / (1.f + expf(-gate)) * up;
+  return cap <= OMNIA_UNIT_GELU_TANH ? gelu_tanh(gate) * up : fmaxf(gate, 0.f) * up;
 }
 
 // Attention whose heads are the difference of two softmax maps (query heads 2 h and 2 h + 1): a head's output
